@@ -29,6 +29,7 @@
 #include "dsk_kernels.cuh"
 #include "dsk_mega.cuh"
 #include "dsk_hybrid.cuh"
+#include "dsk_linattn.cuh"
 
 using namespace dsk;
 

@@ -72,15 +72,17 @@ __device__ __forceinline__ float block_sum(float v, float* red) {   // red: 33 f
 
 // ---------------------------------------------------------------------------------------------------------------------
 // conversions at upload: src (fp32 | bf16, row-major rows x cols, pitch src_ld) -> dst (fp32 | bf16).  `tr` > 0 writes the
-// per-head transpose of a (heads*tr) x cols matrix: dst[h][c][d] = src[h*tr + d][c] (absorbed key up-projection).
+// per-head transpose of a (heads*tr) x cols matrix: dst[h][c][d] = src[h*tr + d][c] (absorbed key up-projection); otherwise rows
+// are written `ld` elements apart (a block of columns of a wider matrix).
 // ---------------------------------------------------------------------------------------------------------------------
 template <typename ST, typename DT>
-__global__ void convert_kernel(const ST* __restrict__ src, DT* __restrict__ dst, long long rows, long long cols, int tr) {
+__global__ void convert_kernel(const ST* __restrict__ src, DT* __restrict__ dst, long long rows, long long cols, int tr, long long ld) {
   const long long n = rows * cols;
   for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
-    long long o = i;
+    const long long r = i / cols, c = i - r * cols;
+    long long o = r * ld + c;
     if (tr > 0) {
-      const long long r = i / cols, c = i - r * cols, h = r / tr, d = r - h * tr;
+      const long long h = r / tr, d = r - h * tr;
       o = (h * cols + c) * tr + d;
     }
     dst[o] = from_f<DT>(to_f<ST>(src[i]));
@@ -96,15 +98,20 @@ __global__ void advance_ctl(int* ctl, int by) { ctl[0] += by; }
 
 // x[t] = scale * table[tok[t]] (+ bigram[row]).  The second table is indexed by the pair (previous token, token): row
 // (prev * mul_prev + tok * mul_cur) mod buckets, and row `buckets` for the first token of a sequence (position ctl[0] + t == 0).
-// The token before the step's first one is carried[0]; carry_token stores the step's last token there afterwards.
+// The token before the step's first one is carried[0]; carry_token stores the step's last token there afterwards.  x_keep
+// (nullable) receives a copy (a layer loop may add the embedding again).
 template <typename WT>
 __global__ void embed_rows(const int* __restrict__ tok, const WT* __restrict__ table, int width, float* __restrict__ x, float scale,
                            const WT* __restrict__ bigram, int buckets, int mul_prev, int mul_cur, const int* __restrict__ ctl,
-                           const int* __restrict__ carried) {
+                           const int* __restrict__ carried, float* __restrict__ x_keep = nullptr) {
   const int t = blockIdx.x;
   const WT* row = table + (size_t)tok[t] * width;
   if (!bigram) {
-    for (int c = threadIdx.x; c < width; c += blockDim.x) x[(size_t)t * width + c] = scale * to_f<WT>(row[c]);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+      const float v = scale * to_f<WT>(row[c]);
+      x[(size_t)t * width + c] = v;
+      if (x_keep) x_keep[(size_t)t * width + c] = v;
+    }
     return;
   }
   long long r = buckets;
@@ -113,7 +120,11 @@ __global__ void embed_rows(const int* __restrict__ tok, const WT* __restrict__ t
     r = (prev * mul_prev + (long long)tok[t] * mul_cur) % buckets;
   }
   const WT* brow = bigram + (size_t)r * width;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) x[(size_t)t * width + c] = fmaf(scale, to_f<WT>(row[c]), to_f<WT>(brow[c]));
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    const float v = fmaf(scale, to_f<WT>(row[c]), to_f<WT>(brow[c]));
+    x[(size_t)t * width + c] = v;
+    if (x_keep) x_keep[(size_t)t * width + c] = v;
+  }
 }
 // the ring rows of the last taps - 1 positions of a step of T >= taps - 1 tokens (see canon_conv)
 __global__ void canon_history(const float* __restrict__ x, int ld, float* __restrict__ hist, int T, int ch, int taps, const int* __restrict__ ctl) {
@@ -181,11 +192,13 @@ __global__ void __launch_bounds__(128) canon_conv(const float* __restrict__ x, i
 // RMS norm in groups.  Row t of `in` (n values) is cut into `groups` equal consecutive parts; each part is divided by
 // sqrt(mean(part^2) + eps) and the row is multiplied by w.  mode 0: out[row] = result, where row = (ctl ? ctl[0] : 0) + t,
 // taken modulo `ring` (a ring cache of latents; ring = 0 means rows are not wrapped).  mode 1: out[t] += alpha * result.
+// gate (nullable, row pitch ld_gate): the result is multiplied by it entry by entry.
 // ---------------------------------------------------------------------------------------------------------------------
 template <typename OT>
 __global__ void __launch_bounds__(256) group_rmsnorm(const float* __restrict__ in, int ld_in, const float* __restrict__ w,
                                                      OT* __restrict__ out, int ld_out, int n, int groups, float eps, int mode,
-                                                     float alpha, const int* __restrict__ ctl, int ring) {
+                                                     float alpha, const int* __restrict__ ctl, int ring,
+                                                     const float* __restrict__ gate = nullptr, int ld_gate = 0) {
   __shared__ float red[33];
   const int t = blockIdx.x;
   const float* x = in + (size_t)t * ld_in;
@@ -201,7 +214,8 @@ __global__ void __launch_bounds__(256) group_rmsnorm(const float* __restrict__ i
     const float sc = 1.f / sqrtf(ss / (float)gs + eps);
     for (int i = threadIdx.x; i < gs; i += blockDim.x) {
       const int c = g * gs + i;
-      const float v = x[c] * sc * w[c];
+      float v = x[c] * sc * w[c];
+      if (gate) v *= gate[(size_t)t * ld_gate + c];
       if (mode == 0) o[c] = from_f<OT>(v);
       else o[c] = from_f<OT>(to_f<OT>(o[c]) + alpha * v);
     }
@@ -211,7 +225,8 @@ __global__ void __launch_bounds__(256) group_rmsnorm(const float* __restrict__ i
 // ---------------------------------------------------------------------------------------------------------------------
 // matrix products
 // ---------------------------------------------------------------------------------------------------------------------
-enum { HEPI_STORE = 0, HEPI_ADD = 1, HEPI_GLU = 2, HEPI_GELU_MUL = 3, HEPI_XIELU = 4, HEPI_GEGLU = 5, HEPI_SIGMUL = 6, HEPI_RELU2 = 7, HEPI_LINGATE = 8 };
+enum { HEPI_STORE = 0, HEPI_ADD = 1, HEPI_GLU = 2, HEPI_GELU_MUL = 3, HEPI_XIELU = 4, HEPI_GEGLU = 5, HEPI_SIGMUL = 6, HEPI_RELU2 = 7, HEPI_LINGATE = 8,
+       HEPI_SILU_SIG = 9, HEPI_SOFTCAP = 10 };
 __host__ __device__ constexpr bool epi_dual(int epi) { return epi == HEPI_GLU || epi == HEPI_GEGLU; }   // two weight matrices per output
 
 struct GemmP {
@@ -234,7 +249,8 @@ struct GemmP {
   float lim;               // GLU: g = min(gate, lim), u = clamp(up, -lim, lim), C = g sigmoid(1.702 g) (u + 1)
                            // GEGLU: C = gelu_tanh(gate) * up;  SIGMUL: C *= sigmoid(acc) (a gate on what C already holds);
                            // RELU2: C = max(acc, 0)^2;  LINGATE (the stacked [q | f | v] projection of a gated linear recurrence, aux_off
-                           // columns of q and of f): q columns silu(acc), f columns l + (1 - l) sigmoid(acc) with l = aux[n - aux_off] (fp32), v columns acc
+                           // columns of q and of f): q columns silu(acc), f columns l + (1 - l) sigmoid(acc) with l = aux[n - aux_off] (fp32), v columns acc;
+                           // SILU_SIG: columns below aux_off silu(acc), the others sigmoid(acc);  SOFTCAP: C = lim tanh(alpha acc / lim)
   const void* aux;         // GELU_MUL: C = gelu_tanh(acc) * aux[aux_row[row] * aux_ld + aux_off + n]
   const int* aux_row;
   int aux_ld, aux_off;
@@ -251,6 +267,8 @@ __device__ __forceinline__ void gemm_epilogue(const GemmP& P, float* __restrict_
   else if (EPI == HEPI_GEGLU) crow[n] = gelu_tanh_f(v) * v2;
   else if (EPI == HEPI_SIGMUL) crow[n] *= sigmoid_f(v);
   else if (EPI == HEPI_RELU2) { const float r = fmaxf(v, 0.f); crow[n] = r * r; }
+  else if (EPI == HEPI_SILU_SIG) crow[n] = n < P.aux_off ? silu_f(v) : sigmoid_f(v);
+  else if (EPI == HEPI_SOFTCAP) crow[n] = P.lim * tanhf(P.alpha * v / P.lim);
   else if (EPI == HEPI_LINGATE) {
     const int hn = P.aux_off;
     if (n < hn) crow[n] = silu_f(v);
@@ -1149,7 +1167,8 @@ __global__ void __launch_bounds__(256) latent_swa_attn(const float* __restrict__
 // merges the NS partial softmax results of one (token, head): out = sum_s e^(m_s - m) acc_s / sum_s e^(m_s - m) l_s.
 // Grid (token x head, blocks of 128 columns): a thread owns one column and reads its NS partial values with independent loads.
 __global__ void __launch_bounds__(128) latent_swa_merge(const float* __restrict__ part, float* __restrict__ out, int R, int NS,
-                                                        const float* __restrict__ gate = nullptr, int ld_gate = 0, int H = 1) {
+                                                        const float* __restrict__ gate = nullptr, int ld_gate = 0, int H = 1,
+                                                        int gate_head = 0, int ld_out = 0, float alpha = 1.f) {
   __shared__ float wts[64], ms[64];   // NS <= 64 (kAttnSplitMax)
   const size_t th = blockIdx.x;
   const float* pp = part + th * NS * (R + 2);
@@ -1172,16 +1191,18 @@ __global__ void __launch_bounds__(128) latent_swa_merge(const float* __restrict_
     a0 = fmaf(wts[s], v0, a0); a1 = fmaf(wts[s + 1], v1, a1); a2 = fmaf(wts[s + 2], v2, a2); a3 = fmaf(wts[s + 3], v3, a3);
   }
   for (; s < NS; s++) a0 = fmaf(wts[s], pp[(size_t)s * (R + 2) + 2 + r], a0);
-  // gate (nullable): row th = token * H + head is multiplied by sigmoid(gate[token][head * R + r])
-  const float gt = gate ? sigmoid_f(gate[(th / H) * (size_t)ld_gate + (th % H) * (size_t)R + r]) : 1.f;
-  out[th * R + r] = ((a0 + a1) + (a2 + a3)) * inv * gt;
+  // gate (nullable): row th = token * H + head is multiplied by sigmoid(gate[token][head * R + r]), with gate_head by sigmoid(gate[token][head]);
+  // ld_out > 0: pitch of a token's output row (otherwise H * R); every result is multiplied by alpha
+  const float gt = gate ? sigmoid_f(gate[(th / H) * (size_t)ld_gate + (gate_head ? th % H : (th % H) * (size_t)R + r)]) : 1.f;
+  out[(ld_out > 0 ? (th / H) * (size_t)ld_out + (th % H) * (size_t)R : th * R) + r] = ((a0 + a1) + (a2 + a3)) * inv * gt * alpha;
 }
 
-// out[t][c] *= sigmoid(gate[t][c]) for the n columns of T rows (an output gate whose raw values came out of a stacked projection)
-__global__ void gate_rows(float* __restrict__ out, int ld_out, const float* __restrict__ gate, int ld_gate, int n) {
+// out[t][c] *= sigmoid(gate[t][c / per]) for the n columns of T rows (an output gate whose raw values came out of a stacked
+// projection; per: columns that share a gate)
+__global__ void gate_rows(float* __restrict__ out, int ld_out, const float* __restrict__ gate, int ld_gate, int n, int per) {
   float* o = out + (size_t)blockIdx.x * ld_out;
   const float* g = gate + (size_t)blockIdx.x * ld_gate;
-  for (int c = threadIdx.x; c < n; c += blockDim.x) o[c] *= sigmoid_f(g[c]);
+  for (int c = threadIdx.x; c < n; c += blockDim.x) o[c] *= sigmoid_f(g[per == 1 ? c : c / per]);
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -1327,10 +1348,42 @@ __global__ void __launch_bounds__(256) layer_norm_add_norm(const float* __restri
   }
 }
 
+// Opening of a pre-norm sublayer:  x += e + row (both nullable: the embedding and the vector of a loop pass that starts here);
+// h = x / sqrt(mean(x^2) + eps) * w.  The row stays in registers up to 256 * kLnRegs values.
+__global__ void __launch_bounds__(256) rms_open(float* __restrict__ x, const float* __restrict__ e, const float* __restrict__ row,
+                                                const float* __restrict__ w, float* __restrict__ h, int n, float eps) {
+  __shared__ float red[33];
+  float* xr = x + (size_t)blockIdx.x * n;
+  const float* er = e ? e + (size_t)blockIdx.x * n : nullptr;
+  float* hr = h + (size_t)blockIdx.x * n;
+  const bool add = e || row;
+  float v[kLnRegs], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < kLnRegs; k++) {
+    const int i = threadIdx.x + 256 * k;
+    v[k] = 0.f;
+    if (i < n) {
+      v[k] = xr[i];
+      if (add) { if (er) v[k] += er[i]; if (row) v[k] += row[i]; xr[i] = v[k]; }
+    }
+    ss = fmaf(v[k], v[k], ss);
+  }
+  for (int i = threadIdx.x + 256 * kLnRegs; i < n; i += 256) {
+    float u = xr[i];
+    if (add) { if (er) u += er[i]; if (row) u += row[i]; xr[i] = u; }
+    ss = fmaf(u, u, ss);
+  }
+  const float sc = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+#pragma unroll
+  for (int k = 0; k < kLnRegs; k++) { const int i = threadIdx.x + 256 * k; if (i < n) hr[i] = v[k] * sc * w[i]; }
+  for (int i = threadIdx.x + 256 * kLnRegs; i < n; i += 256) hr[i] = xr[i] * sc * w[i];
+}
+
 // RMS norm of every head of a row with one weight vector shared by the heads: out[t][h][:] = in[t][h][:] / rms(in[t][h][:]) * w[:].
-// One warp per (token, head) of P values.
+// One warp per (token, head) of P values.  gate (nullable, row pitch ld_gate): the result is multiplied by alpha silu(gate[t][h * P + i]).
 __global__ void __launch_bounds__(256) head_rmsnorm(const float* __restrict__ in, int ld_in, const float* __restrict__ w, float* __restrict__ out,
-                                                    int ld_out, int T, int H, int P, float eps) {
+                                                    int ld_out, int T, int H, int P, float eps, const float* __restrict__ gate = nullptr,
+                                                    int ld_gate = 0, float alpha = 1.f) {
   const int lane = threadIdx.x & 31;
   const long long id = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   if (id >= (long long)T * H) return;
@@ -1340,7 +1393,11 @@ __global__ void __launch_bounds__(256) head_rmsnorm(const float* __restrict__ in
   float ss = 0.f;
   for (int i = lane; i < P; i += 32) ss = fmaf(x[i], x[i], ss);
   const float sc = 1.f / sqrtf(warp_sum(ss) / (float)P + eps);
-  for (int i = lane; i < P; i += 32) o[i] = x[i] * sc * w[i];
+  if (gate) {
+    const float* g = gate + (size_t)t * ld_gate + (size_t)h * P;
+    for (int i = lane; i < P; i += 32) o[i] = x[i] * sc * w[i] * (alpha * silu_f(g[i]));
+  } else
+    for (int i = lane; i < P; i += 32) o[i] = x[i] * sc * w[i];
 }
 
 // x[t][:] += row[:] for the T rows of a step (the per-pass vector of a layer loop)
@@ -1353,6 +1410,7 @@ __global__ void add_row(float* __restrict__ x, int ld, const float* __restrict__
 // Query / key preparation of grouped-query attention, one CTA per token of the step (position ctl[0] + t).
 // head_norm == 0:  q <- rot(q / rms(q) * qw),  k <- rot(k / rms(k) * kw)   with the RMS taken over the whole projection (all heads at once);
 // head_norm == 1:  q <- rot(q) / rms_head(rot(q)),  k likewise: every head is divided by its own RMS after the rotation, without a weight.
+// head_norm == 2:  q <- rot(q / rms_head(q) * qw),  k likewise: per head, before the rotation, with one weight of D entries for all heads.
 //   rot acts on the first rot_dims dimensions of every head: with layout 0 the pair (2i, 2i + 1) turns by the angle pos * freq[i], with
 //   layout 1 the pair (i, i + rot_dims / 2); cos / sin are multiplied by `mag`.  Positions and angles are fp32.
 // q (row pitch ld_q; k: ld_k, v_src: ld_v) goes to q_out; the prepared key goes to row cache_row(pos, keep, ring) of kcache.  Values:
@@ -1399,6 +1457,12 @@ __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q,
       const float* src = isq ? qr : kr;
       float* dst = isq ? q_out + (size_t)t * HD + c0 : kcache + row * GD + c0;
       float ss = 0.f;
+      if (head_norm == 2) {
+        for (int d = lane; d < D; d += 32) ss = fmaf(src[c0 + d], src[c0 + d], ss);
+        const float sc = 1.f / sqrtf(warp_sum(ss) / (float)D + eps);
+        for (int d = lane; d < D; d += 32) dst[d] = rot_entry(src + c0, d, d, rot_dims, layout, sc, isq ? qw : kw, fpos, freq, mag);
+        continue;
+      }
       for (int d = lane; d < D; d += 32) {
         const float v = rot_entry(src, c0 + d, d, rot_dims, layout, 1.f, nullptr, fpos, freq, mag);
         dst[d] = v;
@@ -1441,7 +1505,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q,
 // softmax, fp32).  NS > 1: the key range is cut into NS shares over blockIdx.y, partial results {m, l, acc[Dv]} go to `part`
 // in the layout latent_swa_merge reads.  Without score mixing the key heads may be dealt over gridDim.z CTAs (G / gridDim.z key
 // heads with their query heads each), which stage only their own slice of the key rows.  gate (nullable, row pitch ld_gate):
-// the output is multiplied by sigmoid(gate[t][h * Dv + r]) (an output gate on the concatenated heads; with NS > 1 the merge does it).
+// the output is multiplied by sigmoid(gate[t][h * Dv + r]), with gate_head by sigmoid(gate[t][h]) (an output gate on the concatenated
+// heads; with NS > 1 the merge does it), and by alpha; ld_out: pitch of a token's output row.
 // ---------------------------------------------------------------------------------------------------------------------
 __host__ __device__ inline size_t gqa_attn_smem_floats(int H, int G, int D, int Dv) {
   return (size_t)H * D + (size_t)H * 32 + (size_t)32 * (G * D + 1) + 2 * (size_t)H + (size_t)H * Dv + (size_t)H * H + 8 * 32 + 32 + 32;
@@ -1449,7 +1514,8 @@ __host__ __device__ inline size_t gqa_attn_smem_floats(int H, int G, int D, int 
 __global__ void __launch_bounds__(256) gqa_attn(const float* __restrict__ q, const float* __restrict__ kc, const float* __restrict__ vc,
                                                 float* __restrict__ out, const float* __restrict__ talk, int T, int H, int G, int D,
                                                 int Dv, const int* __restrict__ ctl, int mask, int span, int ring, float scale, int NS,
-                                                float* __restrict__ part, ScoreMods mods, const float* __restrict__ gate, int ld_gate) {
+                                                float* __restrict__ part, ScoreMods mods, const float* __restrict__ gate, int ld_gate, int gate_head,
+                                                int ld_out, float alpha) {
   extern __shared__ float sm[];
   const int GD = G * D, GV = G * Dv, rep = H / G;
   const int GL = G / (int)gridDim.z, g0 = (int)blockIdx.z * GL, h0 = g0 * rep, HL = GL * rep, GDl = GL * D;   // this CTA's key heads and query heads
@@ -1576,10 +1642,10 @@ __global__ void __launch_bounds__(256) gqa_attn(const float* __restrict__ q, con
       if (lane == 0) { pp[0] = m; pp[1] = l; }
       for (int r = lane; r < Dv; r += 32) pp[2 + r] = accs[h * Dv + r] * corr;
     } else {
-      const float inv = corr / l;
+      const float inv = corr / l * alpha;
       for (int r = lane; r < Dv; r += 32) {
-        const float gt = gate ? sigmoid_f(gate[(size_t)t * ld_gate + (size_t)hg * Dv + r]) : 1.f;
-        out[((size_t)t * H + hg) * Dv + r] = accs[h * Dv + r] * inv * gt;
+        const float gt = gate ? sigmoid_f(gate[(size_t)t * ld_gate + (gate_head ? (size_t)hg : (size_t)hg * Dv + r)]) : 1.f;
+        out[(size_t)t * ld_out + (size_t)hg * Dv + r] = accs[h * Dv + r] * inv * gt;
       }
     }
   }

@@ -15,11 +15,14 @@
 //   shift (token shift), norm1.b / norm2.b / final.norm.b (layer norms with a bias)
 //         | mix.q, mix.f, mix.f.b, mix.lower, mix.v, mix.norm, mix.o                                   (gated linear recurrence)
 //   mlp.router, mlp.router.b, mlp.e<j>.up|down                                                        (routed feed-forward, top-softmax router)
+//   mix.q|k|v (+ .conv), mix.b, mix.a, mix.A_log, mix.dt_bias, mix.norm, mix.g, mix.o                 (gated delta rule)
+//   mix.q|k|v|g, mix.norm, mix.o                                                                      (lightning attention)
+// Two mixers side by side name theirs mix.left.* and mix.right.*.
 // Grouped-query attention with its switches on adds mix.v, mix.q.b / k.b / v.b, mix.rel, mix.sink, mix.vmix; latent attention with a
 // rotated key part (DSK_MIX_MLA) has mix.dq, dq.norm, uq, dkv, dkv.norm, uk, uv, g, o; a gated dense feed-forward mlp.gate / up / down;
 // DSK_BLOCK_POST layers norm1 / norm2, ls1 / ls2, canon1 / canon2, rg1 / rg2 (+ .b); the model "bigram" beside "embed".
 // A parallel block computes, with h = norm1(x):  x += m (mixer(h) + ff(h));  a sandwich block  x += norm1b(mixer(norm1(x))),
-// x += norm2b(ff(norm2(x))).  Then, when the model has a per-layer token table,
+// x += norm2b(ff(norm2(x)));  a pre-norm block  x += m mixer(norm1(x)), x += m ff(norm2(x)).  Then, when the model has a per-layer token table,
 // g = gelu_tanh(side.gate x) * side.embed[token][i*sd : (i+1)*sd],  y = side.proj g,  x += m * rmsnorm(y) * side.norm.
 // A layer loop repeats a range of layers with the same weights; each repetition ("layer run") keeps a separate cache / state.
 #pragma once
@@ -84,7 +87,12 @@ struct HLayer {
   // (zeros elsewhere), lower bounds, and the output norm's weight (one vector for all heads)
   HTensor lin_in;
   float *lin_bias = nullptr, *lower = nullptr, *lin_norm = nullptr;
-  char have_lin[3] = {0, 0, 0}, have_linb = 0;
+  char have_lin[4] = {0, 0, 0, 0}, have_linb = 0;   // lightning attention: [q | k | v | g]
+  float *decay = nullptr, *log_decay = nullptr;     // lightning attention: one number per head
+  // gated delta rule: its projections ride in qkv (att_layout), convolution taps of the [q | k | v] channels in one array; A_log, dt_bias
+  // and lin_norm as above.  Side by side with attention, o holds both output matrices column by column: [left | right]
+  float* gdn_conv_w = nullptr;
+  char have_gdn[6] = {0, 0, 0, 0, 0, 0}, have_conv[3] = {0, 0, 0}, have_o[2] = {0, 0};
 };
 
 // one execution of a layer: layers inside the loop range run once per pass, each time with a state of their own
@@ -112,6 +120,7 @@ struct LayerState {
   float* canon = nullptr;           // DSK_BLOCK_POST: [2][taps - 1][width] rings of the two input convolutions
   float* shift = nullptr;           // token shift: the mixer input of the sequence's last token [width]
   float* lin = nullptr;             // gated linear recurrence: [heads][dim][vdim]
+  // gated delta rule: state in lin, the convolutions' inputs in hist, a ring over positions of taps - 1 + kConvSpare rows
   size_t ssm_bytes = 0, hist_bytes = 0, cache_bytes = 0, vcache_bytes = 0, canon_bytes = 0, shift_bytes = 0, lin_bytes = 0;
 };
 
@@ -130,6 +139,9 @@ struct State {
   int* d_rows = nullptr;
   int prefill_keys = 0;                      // keys a block of queries can see at most; 0: the matrix path is off
   float* y = nullptr;                        // a sublayer's output before its closing norm (sandwich and post blocks)
+  float* emb = nullptr;                      // the step's embedding output (a layer loop that adds it again)
+  // linear attention: prepared q, k and v rows, per-block records, outputs ahead of their norm
+  float *lq = nullptr, *lk = nullptr, *lv = nullptr, *lrec = nullptr, *lout = nullptr;
   float* hs = nullptr;                       // the token-shifted mixer input of the step
   float* vfirst = nullptr;                   // [chunk][kv_heads * vdim] values of the step's tokens in the first value-mixing layer
   int* d_prev = nullptr;                     // the sequence's last token (bigram embedding)
@@ -153,13 +165,41 @@ static long long ssd_inner(const dsk_layer_spec& s) { return (long long)s.ssm_he
 static long long ssd_channels(const dsk_layer_spec& s) { return ssd_inner(s) + 2LL * s.ssm_groups * s.ssm_state; }
 static long long ssd_proj(const dsk_layer_spec& s) { return ssd_inner(s) + ssd_channels(s) + s.ssm_heads; }
 
+static bool has_gdn(const dsk_layer_spec& s) { return s.mixer == DSK_MIX_GDN || s.mixer2 == DSK_MIX_GDN; }
+static long long gdn_qk(const dsk_layer_spec& s) { return has_gdn(s) ? (long long)s.gdn_kv_heads * s.gdn_dim : 0; }
+static long long gdn_v(const dsk_layer_spec& s) { return has_gdn(s) ? (long long)s.gdn_heads * s.gdn_vdim : 0; }
+
+// Columns of the stacked projection of attention with a value matrix and of the delta rule:  [q | k | v | gate], or, with a delta
+// rule beside it (or alone),  [q | k | v | dq | dk | dv | dg | gate | db | da], padded with zero rows to a multiple of 8.
+struct AttLayout {
+  long long k = 0, v = 0, gate = 0, gate_rows = 0, dq = 0, dk = 0, dv = 0, dg = 0, db = 0, da = 0, total = 0;
+};
+static AttLayout att_layout(const dsk_layer_spec& s) {
+  AttLayout a;
+  long long n = 0;
+  if (s.mixer == DSK_MIX_GQA) {
+    a.k = (long long)s.att_heads * s.att_dim; a.v = a.k + (long long)s.att_kv_heads * s.att_dim; n = a.v + (long long)s.att_kv_heads * s.att_vdim;
+    a.gate_rows = s.att_out_gate == DSK_GATE_ENTRY ? (long long)s.att_heads * s.att_vdim : s.att_out_gate == DSK_GATE_HEAD ? s.att_heads : 0;
+  }
+  if (has_gdn(s)) { a.dq = n; a.dk = a.dq + gdn_qk(s); a.dv = a.dk + gdn_qk(s); a.dg = a.dv + gdn_v(s); n = a.dg + gdn_v(s); }
+  a.gate = n; n += a.gate_rows;
+  if (has_gdn(s)) { a.db = n; a.da = n + s.gdn_heads; n = (a.da + s.gdn_heads + 7) / 8 * 8; }
+  a.total = n;
+  return a;
+}
+
 static int validate(const dsk_hybrid_config& c, const dsk_layer_spec* L) {
   if (c.dim <= 0 || c.vocab_size <= 0 || c.n_layers <= 0 || c.max_seq_len <= 0) return fail(-1, "hybrid model: bad dimensions");
   if (c.quant != DSK_F32 && c.quant != DSK_BF16) return fail(-1, "hybrid models run with quant fp32 or bf16");
   if (c.norm_groups <= 0 || c.dim % c.norm_groups != 0) return fail(-1, "norm groups %d do not divide width %d", c.norm_groups, c.dim);
   if (c.chunk < 1 || c.chunk > 4096) return fail(-1, "chunk %d out of range (1..4096)", c.chunk);
   if (c.side_dim < 0) return fail(-1, "negative side_dim");
-  if (c.block != DSK_BLOCK_PARALLEL && c.block != DSK_BLOCK_SANDWICH && c.block != DSK_BLOCK_POST) return fail(-1, "unknown block kind %d", c.block);
+  if (c.block != DSK_BLOCK_PARALLEL && c.block != DSK_BLOCK_SANDWICH && c.block != DSK_BLOCK_POST && c.block != DSK_BLOCK_PRE) return fail(-1, "unknown block kind %d", c.block);
+  if (c.block == DSK_BLOCK_PRE && (c.norm_kind != DSK_NORM_RMS || c.norm_groups != 1 || c.token_shift || c.side_dim > 0))
+    return fail(-1, "pre-norm blocks run with ungrouped RMS norms, without a token shift and without the per-layer token input");
+  if (c.norm_one_plus && (c.norm_kind != DSK_NORM_RMS || c.norm_scalar)) return fail(-1, "norm weights stored around zero belong to RMS norms with a weight vector");
+  if (c.loop_embed && c.block != DSK_BLOCK_PRE) return fail(-1, "a layer loop that adds the embedding again belongs to pre-norm blocks");
+  if (!(c.logit_softcap >= 0.f)) return fail(-1, "negative logit cap");
   if (c.block == DSK_BLOCK_POST && (c.norm_groups != 1 || c.loop_times >= 1))
     return fail(-1, "post-norm blocks run with ungrouped norms and without a layer loop");
   if (c.block == DSK_BLOCK_POST && c.norm_kind == DSK_NORM_LAYER && c.norm_scalar) return fail(-1, "single-number norm weights belong to RMS norms");
@@ -174,6 +214,13 @@ static int validate(const dsk_hybrid_config& c, const dsk_layer_spec* L) {
     return fail(-1, "layer loop %d..%d outside the %d layers", c.loop_start, c.loop_stop, c.n_layers);
   for (int i = 0; i < c.n_layers; i++) {
     const dsk_layer_spec& s = L[i];
+    if (s.mixer2 != 0 && !(s.mixer2 == DSK_MIX_GDN && s.mixer == DSK_MIX_GQA && s.att_value_proj && s.att_kv_from < 0 && !s.att_vmix))
+      return fail(-1, "layer %d: two mixers side by side are attention with its own value matrix and the delta rule", i);
+    if (has_gdn(s)) {
+      if (s.gdn_heads <= 0 || s.gdn_kv_heads <= 0 || s.gdn_dim <= 0 || s.gdn_vdim <= 0 || s.gdn_conv < 1) return fail(-1, "layer %d: bad delta-rule sizes", i);
+      if (s.gdn_heads % s.gdn_kv_heads != 0) return fail(-1, "layer %d: delta-rule heads %d not a multiple of its key heads %d", i, s.gdn_heads, s.gdn_kv_heads);
+      if (s.gdn_dim > 256) return fail(-1, "layer %d: key size %d > 256 unsupported (the recurrence keeps the state in registers)", i, s.gdn_dim);
+    }
     if (s.mixer == DSK_MIX_SSD) {
       if (s.ssm_heads <= 0 || s.ssm_vdim <= 0 || s.ssm_state <= 0 || s.ssm_groups <= 0 || s.ssm_conv < 1 || s.ssm_norm_groups <= 0)
         return fail(-1, "layer %d: bad state-space mixer sizes", i);
@@ -200,16 +247,18 @@ static int validate(const dsk_hybrid_config& c, const dsk_layer_spec* L) {
       if (s.rot_dims < 0 || s.rot_dims > s.att_dim || s.rot_dims % 2 != 0) return fail(-1, "layer %d: rot dims %d must be even and at most dim %d", i, s.rot_dims, s.att_dim);
       if (s.rot_dims > 0 && !(s.rot_base > 0.f)) return fail(-1, "layer %d: bad rotation base", i);
       if ((s.rot_layout != DSK_ROT_PAIRS && s.rot_layout != DSK_ROT_HALF) || (s.rot_scale != DSK_ROTSCALE_YARN && s.rot_scale != DSK_ROTSCALE_BANDS) ||
-          (s.att_qk_norm != DSK_QKNORM_WHOLE && s.att_qk_norm != DSK_QKNORM_HEAD))
+          (s.att_qk_norm != DSK_QKNORM_WHOLE && s.att_qk_norm != DSK_QKNORM_HEAD && s.att_qk_norm != DSK_QKNORM_HEAD_WEIGHT))
         return fail(-1, "layer %d: unknown rotation layout, rotation scaling or query / key norm", i);
       if (s.rot_scale == DSK_ROTSCALE_BANDS && s.rot_factor > 0.f && (!(s.rot_fast > s.rot_slow) || s.rot_original <= 0))
         return fail(-1, "layer %d: wavelength-band rotation scaling needs high > low and a positive original length", i);
+      if (s.att_out_gate < DSK_GATE_NONE || s.att_out_gate > DSK_GATE_HEAD) return fail(-1, "layer %d: unknown output gate %d", i, s.att_out_gate);
       if (s.att_out_gate && !s.att_value_proj) return fail(-1, "layer %d: the output gate's rows ride in the stacked q / k / v projection (att_value_proj)", i);
       if (s.att_kv_from >= 0) {
         const int j = s.att_kv_from;
         if (j >= i || L[j].mixer != DSK_MIX_GQA || L[j].att_kv_from >= 0)
           return fail(-1, "layer %d: kv_from %d must name an earlier attention layer that projects its own keys and values", i, j);
         const dsk_layer_spec& o = L[j];
+        if (s.att_out_gate == DSK_GATE_HEAD) return fail(-1, "layer %d: a per-head output gate belongs to a layer with its own keys and values", i);
         if (o.att_kv_heads != s.att_kv_heads || o.att_dim != s.att_dim || o.att_vdim != s.att_vdim || o.att_keep_first != s.att_keep_first || !o.att_value_proj ||
             !s.att_value_proj || s.att_vmix || s.att_bias)
           return fail(-1, "layer %d: a layer that reads layer %d's keys and values needs its key heads, sizes and kept positions, a value matrix there, and no biases or value mixing of its own", i, j);
@@ -225,11 +274,15 @@ static int validate(const dsk_hybrid_config& c, const dsk_layer_spec* L) {
     } else if (s.mixer == DSK_MIX_HGRN2) {
       if (s.lin_heads <= 0 || s.lin_dim <= 0 || s.lin_vdim <= 0) return fail(-1, "layer %d: bad linear-recurrence sizes", i);
       if (s.lin_dim > 256) return fail(-1, "layer %d: key size %d > 256 unsupported (the recurrence keeps the state in registers)", i, s.lin_dim);
-    } else return fail(-1, "layer %d: unknown mixer %d", i, s.mixer);
-    if (s.mixer != DSK_MIX_SSD && s.mixer != DSK_MIX_HGRN2 && s.att_mask != DSK_MASK_WINDOW && s.att_mask != DSK_MASK_CHUNK) return fail(-1, "layer %d: unknown mask %d", i, s.att_mask);
+    } else if (s.mixer == DSK_MIX_LIGHTNING) {
+      if (s.lin_heads <= 0 || s.lin_dim <= 0 || s.lin_vdim <= 0 || !s.lin_decay) return fail(-1, "layer %d: bad lightning-attention sizes or no decays", i);
+      if (s.lin_dim > 256) return fail(-1, "layer %d: key size %d > 256 unsupported (the recurrence keeps the state in registers)", i, s.lin_dim);
+      for (int h = 0; h < s.lin_heads; h++) if (!(s.lin_decay[h] >= 0.f && s.lin_decay[h] <= 1.f)) return fail(-1, "layer %d: decay %g of head %d outside 0..1", i, (double)s.lin_decay[h], h);
+    } else if (s.mixer != DSK_MIX_GDN) return fail(-1, "layer %d: unknown mixer %d", i, s.mixer);
+    if (s.mixer != DSK_MIX_SSD && s.mixer != DSK_MIX_HGRN2 && s.mixer != DSK_MIX_GDN && s.mixer != DSK_MIX_LIGHTNING && s.att_mask != DSK_MASK_WINDOW && s.att_mask != DSK_MASK_CHUNK) return fail(-1, "layer %d: unknown mask %d", i, s.att_mask);
     if (s.ff_kind == DSK_FF_DENSE) {
       if (s.ff_hidden <= 0) return fail(-1, "layer %d: bad feed-forward size", i);
-      if (s.ff_act != DSK_ACT_XIELU && s.ff_act != DSK_ACT_GEGLU) return fail(-1, "layer %d: unknown activation %d", i, s.ff_act);
+      if (s.ff_act != DSK_ACT_XIELU && s.ff_act != DSK_ACT_GEGLU && s.ff_act != DSK_ACT_GLU_CLAMPED) return fail(-1, "layer %d: unknown activation %d", i, s.ff_act);
     } else if (s.ff_kind == DSK_FF_MOE) {
       if (s.ff_experts <= 0 || s.ff_top <= 0 || s.ff_top > s.ff_experts || s.ff_hidden <= 0) return fail(-1, "layer %d: bad routed feed-forward sizes", i);
       if (s.ff_experts > 4096) return fail(-1, "layer %d: more than 4096 experts unsupported", i);
@@ -266,6 +319,13 @@ static void set_kernel_attrs() {
   cudaFuncSetAttribute(hgrn2_scan<1, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(hgrn2_scan<2, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   cudaFuncSetAttribute(hgrn2_scan<3, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(hgrn2_scan<4, 16>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   cudaFuncSetAttribute(hgrn2_scan<1, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(hgrn2_scan<2, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
+  cudaFuncSetAttribute(gemm_mma<HEPI_SILU_SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMmaSmem);
+  cudaFuncSetAttribute(gemm_mma<HEPI_SOFTCAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMmaSmem);
+  cudaFuncSetAttribute(lin_scan<true, 8, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 8, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
+  cudaFuncSetAttribute(lin_scan<true, 16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
+  cudaFuncSetAttribute(lin_scan<true, 32, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 32, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
+  cudaFuncSetAttribute(lin_scan<true, 16, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 16, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
+  cudaFuncSetAttribute(lin_scan<true, 32, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 32, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   cudaFuncSetAttribute(gqa_attn, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   cudaFuncSetAttribute(mix_heads, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   done = true;
@@ -289,6 +349,16 @@ static dsk_model* model_create(const dsk_hybrid_config* cfg, const dsk_layer_spe
   for (int i = 0; i < cfg->n_layers; i++) {
     HLayer& L = M->L[i];
     L.sp = layers[i];
+    if (L.sp.mixer == DSK_MIX_LIGHTNING) {   // the decays and their logarithms (taken in double, rounded once)
+      const size_t n = (size_t)L.sp.lin_heads * 4;
+      std::vector<float> lg(L.sp.lin_heads);
+      for (int h = 0; h < L.sp.lin_heads; h++) lg[h] = L.sp.lin_decay[h] > 0.f ? (float)std::log((double)L.sp.lin_decay[h]) : -1e30f;
+      if (dmalloc(m, (void**)&L.decay, n) || dmalloc(m, (void**)&L.log_decay, n) || cudaMemcpy(L.decay, L.sp.lin_decay, n, cudaMemcpyHostToDevice) != cudaSuccess ||
+          cudaMemcpy(L.log_decay, lg.data(), n, cudaMemcpyHostToDevice) != cudaSuccess) {
+        fail(-2, "decay table allocation failed"); dsk_model_destroy(m); return nullptr;
+      }
+    }
+    L.sp.lin_decay = nullptr;   // the caller's array
     if (L.sp.ff_kind == DSK_FF_MOE) L.have.assign(3 * (size_t)L.sp.ff_experts, 0);
     if (L.sp.mixer == DSK_MIX_LATENT_SWA) L.owner = L.sp.att_kv_from >= 0 ? L.sp.att_kv_from : i;
     if (L.sp.mixer == DSK_MIX_GQA) L.owner = L.sp.att_kv_from >= 0 ? L.sp.att_kv_from : i;
@@ -365,17 +435,17 @@ static dsk_model* model_create(const dsk_hybrid_config* cfg, const dsk_layer_spe
 static void model_free(dsk_model* m) { delete m->hy; m->hy = nullptr; }
 
 template <typename ST>
-static void launch_convert(const void* src, void* dst, long long rows, long long cols, int tr, bool to_bf16) {
+static void launch_convert(const void* src, void* dst, long long rows, long long cols, int tr, bool to_bf16, long long ld) {
   const long long n = rows * cols;
   const unsigned grid = (unsigned)std::max<long long>(1, std::min<long long>((n + 255) / 256, 1 << 16));
-  if (to_bf16) convert_kernel<ST, __nv_bfloat16><<<grid, 256>>>((const ST*)src, (__nv_bfloat16*)dst, rows, cols, tr);
-  else convert_kernel<ST, float><<<grid, 256>>>((const ST*)src, (float*)dst, rows, cols, tr);
+  if (to_bf16) convert_kernel<ST, __nv_bfloat16><<<grid, 256>>>((const ST*)src, (__nv_bfloat16*)dst, rows, cols, tr, ld);
+  else convert_kernel<ST, float><<<grid, 256>>>((const ST*)src, (float*)dst, rows, cols, tr, ld);
 }
 
 // payload (BF16 or F32; host or device) of logical shape rows x cols (cols == 0: a vector) -> dst (fp32 or bf16), optionally
-// transposed per head (tr)
+// transposed per head (tr), or with its rows `ld` elements apart (0: packed)
 static int put(const char* name, int dtype, const int64_t shape[4], const void* data, size_t nbytes, int on_dev, long long rows,
-               long long cols, void* dst, bool to_bf16, int tr) {
+               long long cols, void* dst, bool to_bf16, int tr, long long ld = 0) {
   if (dtype != DSK_DT_BF16 && dtype != DSK_DT_F32) return fail(-4, "tensor %s: dtype %s unsupported (BF16 or F32)", name, dtype_name(dtype));
   const size_t es = dtype == DSK_DT_BF16 ? 2 : 4;
   const long long n = rows * std::max<long long>(cols, 1);
@@ -389,8 +459,8 @@ static int put(const char* name, int dtype, const int64_t shape[4], const void* 
     CK(cudaMemcpy(staging, data, nbytes, cudaMemcpyHostToDevice));
     src = staging;
   }
-  if (dtype == DSK_DT_BF16) launch_convert<__nv_bfloat16>(src, dst, rows, std::max<long long>(cols, 1), tr, to_bf16);
-  else launch_convert<float>(src, dst, rows, std::max<long long>(cols, 1), tr, to_bf16);
+  if (dtype == DSK_DT_BF16) launch_convert<__nv_bfloat16>(src, dst, rows, std::max<long long>(cols, 1), tr, to_bf16, ld ? ld : std::max<long long>(cols, 1));
+  else launch_convert<float>(src, dst, rows, std::max<long long>(cols, 1), tr, to_bf16, ld ? ld : std::max<long long>(cols, 1));
   CK(cudaGetLastError());
   if (staging) { CK(cudaDeviceSynchronize()); CK(cudaFree(staging)); }
   return 0;
@@ -430,6 +500,26 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
     *have = 1;
     return put(name, dtype, shape, data, nbytes, on_dev, n, 0, *dst + off, false, 0);
   };
+  // columns [col0, col0 + cols) of a matrix that holds two output matrices side by side
+  auto COLS = [&](HTensor& st, long long rows, long long total, long long col0, long long cols, char* have) -> int {
+    if (*have) return fail(-4, "tensor %s uploaded twice", name);
+    if (!st.p) {
+      if (dmalloc(m, &st.p, (size_t)rows * total * M->wsize + 16)) return -2;
+      st.rows = rows; st.cols = total;
+    }
+    *have = 1;
+    return put(name, dtype, shape, data, nbytes, on_dev, rows, cols, (char*)st.p + (size_t)col0 * M->wsize, bf, 0, total);
+  };
+  // weight of a norm outside the mixers, as it multiplies (1 + the stored one when weights are stored around zero)
+  auto NORMW = [&](float** dst) -> int {
+    if (int rc = F32(dst, c.dim, 0)) return rc;
+    if (!c.norm_one_plus) return 0;
+    std::vector<float> v((size_t)c.dim);
+    CK(cudaMemcpy(v.data(), *dst, v.size() * 4, cudaMemcpyDeviceToHost));
+    for (float& x : v) x += 1.f;
+    CK(cudaMemcpy(*dst, v.data(), v.size() * 4, cudaMemcpyHostToDevice));
+    return 0;
+  };
   // a single number (shape []) -> host float
   auto SCALAR = [&](float* dst, char* have) -> int {
     if (*have) return fail(-4, "tensor %s uploaded twice", name);
@@ -455,7 +545,7 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
     CK(cudaMemcpy(M->final_norm, v.data(), (size_t)c.dim * 4, cudaMemcpyHostToDevice));
     return 0;
   }
-  if (nm == "final.norm") return F32(&M->final_norm, c.dim, 0);
+  if (nm == "final.norm") return NORMW(&M->final_norm);
   if (nm == "final.norm.b" && c.norm_bias) return F32(&M->final_norm_b, c.dim, 0);
   if (nm == "head") {
     if (c.tie_head) return fail(-4, "tensor %s: this model's LM head is its embedding table", name);
@@ -499,15 +589,51 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
       if (rest == "rg2" && ff) return MAT(L.rg2, c.dim, c.dim);
       if (rest == "rg2.b" && ff) return F32(&L.rg2_b, c.dim, 0);
     }
-  } else if (rest == "norm1") return F32(&L.norm1, c.dim, 0);
+  } else if (rest == "norm1") return NORMW(&L.norm1);
+  if (c.block == DSK_BLOCK_PRE && rest == "norm2" && s.ff_kind != DSK_FF_NONE) return NORMW(&L.norm2);
   if (c.block == DSK_BLOCK_SANDWICH) {
     if (rest == "norm1b") return F32(&L.norm1b, c.dim, 0);
     if (rest == "norm2" && s.ff_kind != DSK_FF_NONE) return F32(&L.norm2, c.dim, 0);
     if (rest == "norm2b" && s.ff_kind != DSK_FF_NONE) return F32(&L.norm2b, c.dim, 0);
   }
   if (rest.rfind("mix.", 0) == 0) {
-    const std::string k = rest.substr(4);
-    if (is_ssd(s)) {
+    std::string k = rest.substr(4);
+    bool right = s.mixer == DSK_MIX_GDN;
+    if (s.mixer2) {
+      if (k.rfind("left.", 0) == 0) k = k.substr(5);
+      else if (k.rfind("right.", 0) == 0) { k = k.substr(6); right = true; }
+      else return fail(-4, "unknown tensor name %s for two mixers side by side (mix.left.*, mix.right.*)", name);
+    }
+    if (right) {
+      const AttLayout a = att_layout(s);
+      const long long KD = gdn_qk(s), RV = gdn_v(s), HV = s.mixer2 ? (long long)s.att_heads * s.att_vdim : 0;
+      if (!L.qkv.p) { if (dmalloc(m, &L.qkv.p, (size_t)a.total * c.dim * M->wsize + 16)) return -2; CK(cudaMemset(L.qkv.p, 0, (size_t)a.total * c.dim * M->wsize)); L.qkv.rows = a.total; L.qkv.cols = c.dim; }
+      if (k == "q") return STACK(L.qkv, a.total, c.dim, a.dq, KD, &L.have_gdn[0]);
+      if (k == "k") return STACK(L.qkv, a.total, c.dim, a.dk, KD, &L.have_gdn[1]);
+      if (k == "v") return STACK(L.qkv, a.total, c.dim, a.dv, RV, &L.have_gdn[2]);
+      if (k == "g") return STACK(L.qkv, a.total, c.dim, a.dg, RV, &L.have_gdn[3]);
+      if (k == "b") return STACK(L.qkv, a.total, c.dim, a.db, s.gdn_heads, &L.have_gdn[4]);
+      if (k == "a") return STACK(L.qkv, a.total, c.dim, a.da, s.gdn_heads, &L.have_gdn[5]);
+      for (int n = 0; n < 3; n++)
+        if (k == std::string(1, "qkv"[n]) + ".conv") {   // taps of the stacked [q | k | v] channels
+          if (L.have_conv[n]) return fail(-4, "tensor %s uploaded twice", name);
+          if (!L.gdn_conv_w && dmalloc(m, (void**)&L.gdn_conv_w, (size_t)(2 * KD + RV) * s.gdn_conv * 4)) return -2;
+          L.have_conv[n] = 1;
+          return put(name, dtype, shape, data, nbytes, on_dev, n < 2 ? KD : RV, s.gdn_conv, L.gdn_conv_w + (size_t)n * KD * s.gdn_conv, false, 0);
+        }
+      if (k == "A_log") return F32(&L.A_log, s.gdn_heads, 0);
+      if (k == "dt_bias") return F32(&L.dt_bias, s.gdn_heads, 0);
+      if (k == "norm") return F32(&L.lin_norm, s.gdn_vdim, 0);   // one weight vector for all heads
+      if (k == "o") return COLS(L.o, c.dim, HV + RV, HV, RV, &L.have_o[1]);
+    } else if (s.mixer == DSK_MIX_LIGHTNING) {
+      const long long HN = (long long)s.lin_heads * s.lin_dim, HP = (long long)s.lin_heads * s.lin_vdim, tot = 2 * HN + 2 * HP;
+      if (k == "q") return STACK(L.lin_in, tot, c.dim, 0, HN, &L.have_lin[0]);
+      if (k == "k") return STACK(L.lin_in, tot, c.dim, HN, HN, &L.have_lin[1]);
+      if (k == "v") return STACK(L.lin_in, tot, c.dim, 2 * HN, HP, &L.have_lin[2]);
+      if (k == "g") return STACK(L.lin_in, tot, c.dim, 2 * HN + HP, HP, &L.have_lin[3]);
+      if (k == "norm") return F32(&L.mnorm, HP, 0);
+      if (k == "o") return MAT(L.o, c.dim, HP);
+    } else if (is_ssd(s)) {
       const long long inner = ssd_inner(s), ch = ssd_channels(s);
       if (k == "in") return MAT(L.in, ssd_proj(s), c.dim);
       if (k == "conv") return F32(&L.conv_w, ch, s.ssm_conv);
@@ -542,18 +668,20 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
       if (k == "o") return MAT(L.o, c.dim, H * s.att_vdim);
     } else if (s.mixer == DSK_MIX_GQA) {
       const long long HD = (long long)s.att_heads * s.att_dim, GD = (long long)s.att_kv_heads * s.att_dim, GV = (long long)s.att_kv_heads * s.att_vdim;
-      const long long HV = s.att_out_gate ? (long long)s.att_heads * s.att_vdim : 0;
+      const AttLayout a = att_layout(s);
+      const long long HV = a.gate_rows;
       if (s.att_kv_from >= 0) {   // reads another layer's keys and values: only the query projection (and gate) of its own
         if (k == "q") return STACK(L.qkv, HD + HV, c.dim, 0, HD, &L.have_qkv[0]);
         if (k == "g" && s.att_out_gate) return STACK(L.qkv, HD + HV, c.dim, HD, HV, &L.have_qkv[3]);
       } else if (s.att_value_proj) {
-        const long long tot = HD + GD + GV + HV;
-        if (k == "g" && s.att_out_gate) return STACK(L.qkv, tot, c.dim, HD + GD + GV, HV, &L.have_qkv[3]);
+        const long long tot = a.total;
+        if (s.mixer2 && !L.qkv.p) { if (dmalloc(m, &L.qkv.p, (size_t)tot * c.dim * M->wsize + 16)) return -2; CK(cudaMemset(L.qkv.p, 0, (size_t)tot * c.dim * M->wsize)); L.qkv.rows = tot; L.qkv.cols = c.dim; }
+        if (k == "g" && s.att_out_gate) return STACK(L.qkv, tot, c.dim, a.gate, HV, &L.have_qkv[3]);
         if (k == "q") return STACK(L.qkv, tot, c.dim, 0, HD, &L.have_qkv[0]);
         if (k == "k") return STACK(L.qkv, tot, c.dim, HD, GD, &L.have_qkv[1]);
         if (k == "v") return STACK(L.qkv, tot, c.dim, HD + GD, GV, &L.have_qkv[2]);
         if (s.att_bias) {
-          if (!L.qkv_b && HV > 0) { if (dmalloc(m, (void**)&L.qkv_b, (size_t)tot * 4)) return -2; CK(cudaMemset(L.qkv_b, 0, (size_t)tot * 4)); }   // no bias on the gate's rows
+          if (!L.qkv_b && (HV > 0 || s.mixer2)) { if (dmalloc(m, (void**)&L.qkv_b, (size_t)tot * 4)) return -2; CK(cudaMemset(L.qkv_b, 0, (size_t)tot * 4)); }   // no bias on the gate's rows
           if (k == "q.b") return STACKV(&L.qkv_b, tot, 0, HD, &L.have_qkvb[0]);
           if (k == "k.b") return STACKV(&L.qkv_b, tot, HD, GD, &L.have_qkvb[1]);
           if (k == "v.b") return STACKV(&L.qkv_b, tot, HD + GD, GV, &L.have_qkvb[2]);
@@ -569,9 +697,12 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
       if (k == "vmix" || (k == "rel" && s.att_rel_max <= 0)) return 0;   // a checkpoint may carry them for layers that do not use them
       if (k == "q" && !s.att_value_proj) return MAT(L.q, HD, c.dim);
       if (k == "k" && !s.att_value_proj) return MAT(L.kproj, GD, c.dim);
+      if (k == "q.norm" && s.att_qk_norm == DSK_QKNORM_HEAD_WEIGHT) return F32(&L.q_norm, s.att_dim, 0);
+      if (k == "k.norm" && s.att_qk_norm == DSK_QKNORM_HEAD_WEIGHT) return F32(&L.k_norm, s.att_dim, 0);
       if (k == "q.norm" && s.att_qk_norm == DSK_QKNORM_WHOLE) return F32(&L.q_norm, HD, 0);
       if (k == "k.norm" && s.att_qk_norm == DSK_QKNORM_WHOLE) return F32(&L.k_norm, GD, 0);
       if (k == "talk" && s.att_talk) return F32(&L.talk, s.att_heads, s.att_heads);
+      if (k == "o" && s.mixer2) return COLS(L.o, c.dim, (long long)s.att_heads * s.att_vdim + gdn_v(s), 0, (long long)s.att_heads * s.att_vdim, &L.have_o[0]);
       if (k == "o") return MAT(L.o, c.dim, (long long)s.att_heads * s.att_vdim);
     } else {
       const long long H = s.att_heads;
@@ -586,7 +717,7 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
     }
     return fail(-4, "unknown tensor name %s for this layer's mixer", name);
   }
-  if (rest.rfind("mlp.", 0) == 0 && s.ff_kind == DSK_FF_DENSE && s.ff_act == DSK_ACT_GEGLU) {
+  if (rest.rfind("mlp.", 0) == 0 && s.ff_kind == DSK_FF_DENSE && s.ff_act != DSK_ACT_XIELU) {
     const std::string k = rest.substr(4);
     if (k == "gate") return MAT(L.gate_d, s.ff_hidden, c.dim);
     if (k == "up") return MAT(L.up, s.ff_hidden, c.dim);
@@ -679,9 +810,21 @@ static int finalize(dsk_model* m) {
     } else if (!L.norm1) return fail(-5, "missing tensor l%d.norm1", i);
     if (c.token_shift && !L.shift) return fail(-5, "missing tensor l%d.shift", i);
     if (c.norm_bias && (!L.norm1_bias || (s.ff_kind != DSK_FF_NONE && !L.norm2_bias))) return fail(-5, "layer %d: missing norm biases (norm1.b, norm2.b)", i);
+    if (c.block == DSK_BLOCK_PRE && s.ff_kind != DSK_FF_NONE && !L.norm2) return fail(-5, "missing tensor l%d.norm2", i);
+    if (has_gdn(s)) {
+      bool all = L.have_conv[0] && L.have_conv[1] && L.have_conv[2] && L.A_log && L.dt_bias && L.lin_norm && L.have_o[1];
+      for (char h : L.have_gdn) all = all && h;
+      if (!all) return fail(-5, "layer %d: missing delta-rule tensors (q, k, v and their conv, b, a, A_log, dt_bias, g, norm, o)", i);
+      L.qkv.present = true;
+      L.o.present = s.mixer == DSK_MIX_GDN || L.have_o[0];
+    }
     if (c.block == DSK_BLOCK_SANDWICH && (!L.norm1b || (s.ff_kind != DSK_FF_NONE && (!L.norm2 || !L.norm2b))))
       return fail(-5, "layer %d: missing norm tensors (norm1b, norm2, norm2b)", i);
-    if (s.mixer == DSK_MIX_HGRN2) {
+    if (s.mixer == DSK_MIX_GDN) {
+    } else if (s.mixer == DSK_MIX_LIGHTNING) {
+      L.lin_in.present = L.have_lin[0] && L.have_lin[1] && L.have_lin[2] && L.have_lin[3];
+      if (!L.lin_in.present || !L.mnorm || !L.o.present) return fail(-5, "layer %d: missing lightning-attention tensors (mix.q, k, v, g, norm, o)", i);
+    } else if (s.mixer == DSK_MIX_HGRN2) {
       L.lin_in.present = L.have_lin[0] && L.have_lin[1] && L.have_lin[2];
       if (!L.lin_in.present || !L.have_linb || !L.lower || !L.lin_norm || !L.o.present)
         return fail(-5, "layer %d: missing linear-recurrence tensors (mix.q, f, f.b, lower, v, norm, o)", i);
@@ -694,7 +837,7 @@ static int finalize(dsk_model* m) {
         L.qkv.present = L.have_qkv[0] && L.have_qkv[1] && L.have_qkv[2];
         if (!L.qkv.present || (s.att_bias && !(L.have_qkvb[0] && L.have_qkvb[1] && L.have_qkvb[2]))) return fail(-5, "layer %d: missing attention projections (mix.q, k, v and their biases)", i);
       } else if (!L.q.present || !L.kproj.present) return fail(-5, "layer %d: missing attention tensors (mix.q, k)", i);
-      if (!L.o.present || (s.att_qk_norm == DSK_QKNORM_WHOLE && (!L.q_norm || !L.k_norm)) || (s.att_talk && !L.talk))
+      if (!L.o.present || (s.att_qk_norm != DSK_QKNORM_HEAD && (!L.q_norm || !L.k_norm)) || (s.att_talk && !L.talk))
         return fail(-5, "layer %d: missing attention tensors (mix.q.norm, k.norm, talk, o)", i);
       if ((s.att_sink && !L.sink) || (s.att_rel_max > 0 && !L.rel) || (s.att_vmix && !L.have_vmix && i != M->vmix_first))
         return fail(-5, "layer %d: missing attention tensors (mix.sink, rel, vmix)", i);
@@ -718,7 +861,7 @@ static int finalize(dsk_model* m) {
       if (!L.q.present || !L.ukT.present || !L.uk.present || !L.uv.present || !L.o.present) return fail(-5, "layer %d: missing latent-attention tensors (mix.q, uk, uv, o)", i);
       if (s.att_kv_from < 0 && (!L.dkv.present || !L.dkv_norm)) return fail(-5, "layer %d: missing mix.dkv / mix.dkv.norm", i);
     }
-    if (s.ff_kind == DSK_FF_DENSE && s.ff_act == DSK_ACT_GEGLU) {
+    if (s.ff_kind == DSK_FF_DENSE && s.ff_act != DSK_ACT_XIELU) {
       if (!L.gate_d.present || !L.up.present || !L.down.present) return fail(-5, "layer %d: missing feed-forward tensors (mlp.gate, up, down)", i);
     } else if (s.ff_kind == DSK_FF_DENSE && (!L.up.present || !L.down.present || !L.up_b || !L.down_b || !L.act))
       return fail(-5, "layer %d: missing feed-forward tensors (mlp.up, up.b, down, down.b, act)", i);
@@ -744,6 +887,12 @@ static double active_bytes(const dsk_model* m) {
     const dsk_layer_spec& s = L.sp;
     double mat = 0, f32 = W;
     if (R.pass >= 0) f32 += W;
+    if (c.block == DSK_BLOCK_PRE && s.ff_kind != DSK_FF_NONE) f32 += W;
+    if (has_gdn(s)) {
+      const double KD = (double)gdn_qk(s), RV = (double)gdn_v(s);
+      mat += (2 * KD + 2 * RV + 2 * s.gdn_heads) * W + W * RV;
+      f32 += (2 * KD + RV) * s.gdn_conv + 2 * s.gdn_heads + s.gdn_vdim;
+    }
     if (c.block == DSK_BLOCK_SANDWICH) f32 += W * (s.ff_kind != DSK_FF_NONE ? 3 : 1);
     if (c.block == DSK_BLOCK_POST) {   // per sublayer: convolution taps, gate matrix and bias (the closing weight is the W counted above)
       const double subs = s.ff_kind != DSK_FF_NONE ? 2 : 1;
@@ -752,15 +901,20 @@ static double active_bytes(const dsk_model* m) {
     }
     if (c.token_shift) f32 += W;
     if (c.norm_bias) f32 += W * (s.ff_kind != DSK_FF_NONE ? 2 : 1);
-    if (s.mixer == DSK_MIX_HGRN2) {
+    if (s.mixer == DSK_MIX_GDN) {
+    } else if (s.mixer == DSK_MIX_LIGHTNING) {
+      const double HN = (double)s.lin_heads * s.lin_dim, HP = (double)s.lin_heads * s.lin_vdim;
+      mat += (2 * HN + 2 * HP) * W + W * HP;
+      f32 += HP;
+    } else if (s.mixer == DSK_MIX_HGRN2) {
       const double HN = (double)s.lin_heads * s.lin_dim, HP = (double)s.lin_heads * s.lin_vdim;
       mat += (2 * HN + HP) * W + W * HP;
       f32 += 3 * HN + 2 * HP;
     } else if (s.mixer == DSK_MIX_GQA) {
       const bool reads = s.att_kv_from >= 0;
       const double HD = (double)s.att_heads * s.att_dim, GD = reads ? 0.0 : (double)s.att_kv_heads * s.att_dim, GV = s.att_value_proj && !reads ? (double)s.att_kv_heads * s.att_vdim : 0.0;
-      mat += (HD + GD + GV) * W + W * s.att_heads * s.att_vdim * (s.att_out_gate ? 2 : 1);
-      f32 += (s.att_qk_norm == DSK_QKNORM_WHOLE ? HD + GD : 0.0) + (s.att_talk ? (double)s.att_heads * s.att_heads : 0.0) + (s.att_bias ? HD + GD + GV : 0.0) + (s.att_sink ? s.att_heads : 0);
+      mat += (HD + GD + GV) * W + W * s.att_heads * s.att_vdim + W * (double)att_layout(s).gate_rows;
+      f32 += (s.att_qk_norm == DSK_QKNORM_WHOLE ? HD + GD : s.att_qk_norm == DSK_QKNORM_HEAD_WEIGHT ? 2.0 * s.att_dim : 0.0) + (s.att_talk ? (double)s.att_heads * s.att_heads : 0.0) + (s.att_bias ? HD + GD + GV : 0.0) + (s.att_sink ? s.att_heads : 0);
     } else if (s.mixer == DSK_MIX_MLA) {
       const double H = s.att_heads, DK = s.att_dim + s.att_rot_dim, Rr = s.att_kv_rank, Q = s.att_q_rank;
       mat += (Q + Rr + s.att_rot_dim) * W + H * DK * Q + H * (s.att_dim + s.att_vdim) * Rr + (s.att_out_gate ? H * s.att_vdim * W : 0.0) + W * H * s.att_vdim;
@@ -771,12 +925,18 @@ static double active_bytes(const dsk_model* m) {
       if (s.att_kv_from < 0) { mat += (double)s.att_kv_rank * W; f32 += s.att_kv_rank; }
     }
     if (s.ff_kind == DSK_FF_MOE) { mat += (s.ff_expert == DSK_EXPERT_RELU2 ? 2.0 : 3.0) * s.ff_top * s.ff_hidden * W; f32 += (double)s.ff_experts * (W + 1); }
-    if (s.ff_kind == DSK_FF_DENSE && s.ff_act == DSK_ACT_GEGLU) mat += 3.0 * s.ff_hidden * W;
+    if (s.ff_kind == DSK_FF_DENSE && s.ff_act != DSK_ACT_XIELU) mat += 3.0 * s.ff_hidden * W;
     else if (s.ff_kind == DSK_FF_DENSE) { mat += 2.0 * s.ff_hidden * W; f32 += s.ff_hidden + W; }
     if (c.side_dim > 0) { mat += 2.0 * c.side_dim * W + c.side_dim; f32 += W; }
     tot += mat * ws + f32 * 4;
   }
   return tot;
+}
+
+// value channels x key rows of a head that one CTA of the token-by-token kernel holds
+static bool lin_decode_fits(int N, int P) {
+  const int PL = (P + 3) / 4;
+  return PL <= kLinDecodeThreads && (N + std::min(kLinDecodeThreads / PL, N) - 1) / std::min(kLinDecodeThreads / PL, N) <= 16;
 }
 
 // kernels one decoded token launches (embedding + layers + final norm + LM head + arg-max)
@@ -794,10 +954,15 @@ static int launches_per_token(const dsk_model* m) {
     else if (post) n += (s.ff_kind != DSK_FF_NONE ? 2 : 1) * (1 + (M->c.res_gate ? 1 : 0)) + (&R == &M->runs[0] && M->c.canon_taps > 0 ? 1 : 0);   // gate, closing norm + next convolution in one
     else if (fused_norms(M->c)) n += 1 + (s.ff_kind != DSK_FF_NONE ? 1 : 0) + (&R == &M->runs[0] ? 1 + (R.pass >= 0 ? 1 : 0) : 0);
     else n += 1 + (R.pass >= 0 ? 1 : 0) + (sandwich ? 1 + (s.ff_kind != DSK_FF_NONE ? 2 : 0) : 0);
-    if (s.mixer == DSK_MIX_HGRN2) n += 4;   // stacked projection, recurrence, head norm, o
+    if (M->c.block == DSK_BLOCK_PRE && s.ff_kind != DSK_FF_NONE) n += 1;
+    if (M->c.block == DSK_BLOCK_PRE && R.pass >= 0) n -= 1;   // the pass vector is added by the opening norm
+    if (has_gdn(s)) n += lin_decode_fits(s.gdn_dim, s.gdn_vdim) ? 1 : 3 + (s.gdn_conv > 1 ? 1 : 0);
+    if (s.mixer == DSK_MIX_GDN) n += 2;     // stacked projection, o
+    else if (s.mixer == DSK_MIX_LIGHTNING) n += lin_decode_fits(s.lin_dim, s.lin_vdim) ? 4 : 5;   // stacked projection, (records,) recurrence, norm, o
+    else if (s.mixer == DSK_MIX_HGRN2) n += 4;   // stacked projection, recurrence, head norm, o
     else if (s.mixer == DSK_MIX_GQA) n += s.att_value_proj ? 5 : 6;   // q, k (or one stacked q / k / v (/ gate) product), norm + rotation, attention, merge, o
     else if (s.mixer == DSK_MIX_MLA) n += 10 + (s.att_out_gate ? 1 : 0);   // down-projections, query norm, query up, latent preparation, absorbed query, attention, merge, value up, (gate,) o
-    else if (s.mixer != DSK_MIX_MLA && s.mixer != DSK_MIX_HGRN2 && s.mixer != DSK_MIX_GQA) n += is_ssd(s) ? 5 + (s.ssm_conv > 1 ? 1 : 0) : 5 + (s.att_kv_from < 0 ? 2 : 0);
+    else n += is_ssd(s) ? 5 + (s.ssm_conv > 1 ? 1 : 0) : 5 + (s.att_kv_from < 0 ? 2 : 0);
     if (s.ff_kind == DSK_FF_MOE) n += post && M->c.norm_kind == DSK_NORM_LAYER && !M->c.res_gate && M->c.dim <= 256 * kLnRegs ? 4 : 5;
     if (s.ff_kind == DSK_FF_DENSE) n += 2;
     if (M->c.side_dim > 0) n += 3;
@@ -857,6 +1022,7 @@ static dsk_state* state_create(dsk_model* m) {
   size_t mx0 = c.dim, mx1 = c.dim, mx2 = c.dim, mx3 = c.dim, mxE = 1, mxTop = 1;
   S->L.resize(M->runs.size());   // one state per layer run
   bool any_talk = false;
+  size_t mxLQ = 0, mxLV = 0, mxLH = 0;
   size_t mxGV = 0;
   for (size_t r = 0; r < M->runs.size(); r++) {
     const int i = M->runs[r].layer;
@@ -871,7 +1037,23 @@ static dsk_state* state_create(dsk_model* m) {
       ls.shift_bytes = (size_t)c.dim * 4;
       if (salloc(S, (void**)&ls.shift, ls.shift_bytes)) return nullptr;
     }
-    if (sp.mixer == DSK_MIX_HGRN2) {
+    if (has_gdn(sp)) {
+      const size_t KD = gdn_qk(sp), RV = gdn_v(sp), NP = (size_t)sp.gdn_kv_heads * ((sp.gdn_dim + 3) & ~3);
+      ls.lin_bytes = (size_t)sp.gdn_heads * sp.gdn_dim * sp.gdn_vdim * 4;
+      ls.hist_bytes = (size_t)(sp.gdn_conv - 1 + kConvSpare) * (2 * KD + RV) * 4;
+      if (salloc(S, (void**)&ls.lin, ls.lin_bytes) || salloc(S, (void**)&ls.hist, ls.hist_bytes)) return nullptr;
+      mxLQ = std::max(mxLQ, NP); mxLV = std::max(mxLV, RV); mxLH = std::max<size_t>(mxLH, sp.gdn_heads);
+      mx0 = std::max<size_t>(mx0, att_layout(sp).total);
+      mx3 = std::max<size_t>(mx3, RV + (sp.mixer2 ? (size_t)sp.att_heads * sp.att_vdim : 0));
+    }
+    if (sp.mixer == DSK_MIX_GDN) {
+    } else if (sp.mixer == DSK_MIX_LIGHTNING) {
+      const size_t HN = (size_t)sp.lin_heads * sp.lin_dim, HP = (size_t)sp.lin_heads * sp.lin_vdim;
+      ls.lin_bytes = HN * sp.lin_vdim * 4;
+      if (salloc(S, (void**)&ls.lin, ls.lin_bytes)) return nullptr;
+      mx0 = std::max<size_t>(mx0, 2 * HN + 2 * HP); mx3 = std::max<size_t>(mx3, HP);
+      mxLV = std::max(mxLV, HP); mxLH = std::max<size_t>(mxLH, sp.lin_heads);
+    } else if (sp.mixer == DSK_MIX_HGRN2) {
       const size_t HN = (size_t)sp.lin_heads * sp.lin_dim, HP = (size_t)sp.lin_heads * sp.lin_vdim;
       ls.lin_bytes = HN * sp.lin_vdim * 4;
       if (salloc(S, (void**)&ls.lin, ls.lin_bytes)) return nullptr;
@@ -936,7 +1118,7 @@ static dsk_state* state_create(dsk_model* m) {
     size_t keys = 0, hd = 0, hv = 0, heads = 0, pack_es = 0;
     bool latent = false;
     for (const HLayer& L : M->L) {
-      if (L.sp.mixer == DSK_MIX_SSD || L.sp.mixer == DSK_MIX_HGRN2) continue;
+      if (L.sp.mixer == DSK_MIX_SSD || L.sp.mixer == DSK_MIX_HGRN2 || L.sp.mixer == DSK_MIX_GDN || L.sp.mixer == DSK_MIX_LIGHTNING) continue;
       const size_t kh = L.sp.mixer == DSK_MIX_GQA ? L.sp.att_kv_heads : L.sp.att_heads;
       latent |= L.sp.mixer == DSK_MIX_LATENT_SWA || L.sp.mixer == DSK_MIX_MLA;
       if (L.sp.mixer == DSK_MIX_LATENT_SWA) pack_es = std::max(pack_es, M->wsize);
@@ -956,7 +1138,10 @@ static dsk_state* state_create(dsk_model* m) {
     }
   }
   rc |= salloc(S, (void**)&S->x, Tc * c.dim * 4) | salloc(S, (void**)&S->h, Tc * c.dim * 4);
-  if (c.block != DSK_BLOCK_PARALLEL) rc |= salloc(S, (void**)&S->y, Tc * c.dim * 4);
+  if (c.loop_embed && c.loop_times > 1) rc |= salloc(S, (void**)&S->emb, Tc * c.dim * 4);
+  if (mxLH) rc |= salloc(S, (void**)&S->lrec, (Tc + kLinBlk - 1) / kLinBlk * mxLH * kRecFloats * 4) | salloc(S, (void**)&S->lout, Tc * mxLV * 4);
+  if (mxLQ) rc |= salloc(S, (void**)&S->lq, Tc * mxLQ * 4) | salloc(S, (void**)&S->lk, Tc * mxLQ * 4) | salloc(S, (void**)&S->lv, Tc * mxLV * 4);
+  if (c.block == DSK_BLOCK_SANDWICH || c.block == DSK_BLOCK_POST) rc |= salloc(S, (void**)&S->y, Tc * c.dim * 4);
   if (c.token_shift) rc |= salloc(S, (void**)&S->hs, Tc * c.dim * 4);
   if (mxGV) rc |= salloc(S, (void**)&S->vfirst, Tc * mxGV * 4);
   rc |= salloc(S, (void**)&S->d_prev, 16);
@@ -1028,6 +1213,8 @@ static void launch_gemm_mma(int epi, const GemmP& P, int Z, int tile_cap, cudaSt
     case HEPI_SIGMUL: gemm_mma<HEPI_SIGMUL><<<grid, 256, kMmaSmem, st>>>(P); break;
     case HEPI_RELU2: gemm_mma<HEPI_RELU2><<<grid, 256, kMmaSmem, st>>>(P); break;
     case HEPI_LINGATE: gemm_mma<HEPI_LINGATE><<<grid, 256, kMmaSmem, st>>>(P); break;
+    case HEPI_SILU_SIG: gemm_mma<HEPI_SILU_SIG><<<grid, 256, kMmaSmem, st>>>(P); break;
+    case HEPI_SOFTCAP: gemm_mma<HEPI_SOFTCAP><<<grid, 256, kMmaSmem, st>>>(P); break;
     default: gemm_mma<HEPI_GELU_MUL><<<grid, 256, kMmaSmem, st>>>(P); break;
   }
 }
@@ -1045,6 +1232,8 @@ static void launch_gemm_t(int epi, const GemmP& P, int Z, bool small, int tile_c
       case HEPI_SIGMUL: gemv_rows<WT, HEPI_SIGMUL><<<grid, 256, 0, st>>>(P); break;
       case HEPI_RELU2: gemv_rows<WT, HEPI_RELU2><<<grid, 256, 0, st>>>(P); break;
       case HEPI_LINGATE: gemv_rows<WT, HEPI_LINGATE><<<grid, 256, 0, st>>>(P); break;
+      case HEPI_SILU_SIG: gemv_rows<WT, HEPI_SILU_SIG><<<grid, 256, 0, st>>>(P); break;
+      case HEPI_SOFTCAP: gemv_rows<WT, HEPI_SOFTCAP><<<grid, 256, 0, st>>>(P); break;
       default: gemv_rows<WT, HEPI_GELU_MUL><<<grid, 256, 0, st>>>(P); break;
     }
   } else {
@@ -1058,6 +1247,8 @@ static void launch_gemm_t(int epi, const GemmP& P, int Z, bool small, int tile_c
       case HEPI_SIGMUL: gemm_tiled<WT, HEPI_SIGMUL><<<grid, 256, 0, st>>>(P); break;
       case HEPI_RELU2: gemm_tiled<WT, HEPI_RELU2><<<grid, 256, 0, st>>>(P); break;
       case HEPI_LINGATE: gemm_tiled<WT, HEPI_LINGATE><<<grid, 256, 0, st>>>(P); break;
+      case HEPI_SILU_SIG: gemm_tiled<WT, HEPI_SILU_SIG><<<grid, 256, 0, st>>>(P); break;
+      case HEPI_SOFTCAP: gemm_tiled<WT, HEPI_SOFTCAP><<<grid, 256, 0, st>>>(P); break;
       default: gemm_tiled<WT, HEPI_GELU_MUL><<<grid, 256, 0, st>>>(P); break;
     }
   }
@@ -1125,6 +1316,68 @@ static void launch_hgrn2(const dsk_layer_spec& sp, const float* proj, int ld, fl
 #undef DSK_LIN
 }
 
+// the walk over the blocks of a step (lin_scan): lanes per channel group by the key size, warps per CTA by how many CTAs there are
+static void launch_lin_scan(bool delta, const float* q, const float* k, int ldq, int hs, int rep, const float* v, int ldv, const float* rec, float* state,
+                            float* out, int ldo, int T, int H, int N, int P, cudaStream_t st) {
+  const int TPC = N <= 32 ? 8 : N <= 64 ? 16 : 32, RQ = N <= 128 ? 1 : 2, CW = 4 * (32 / TPC);
+  int warps = std::max(1, std::min(8, (P + CW - 1) / CW));
+  while (warps > 1 && H * ((P + warps * CW - 1) / (warps * CW)) < 148) warps = (warps + 1) / 2;
+  if (const char* e = getenv("DSK_LIN_WARPS")) warps = std::max(1, std::min(8, atoi(e)));   // A/B switch
+  const int PB = warps * CW;
+  const dim3 grid((unsigned)H, (unsigned)((P + PB - 1) / PB));
+  const size_t smem = lin_scan_smem(4 * TPC * RQ, PB, warps, CW);
+#define DSK_LSCAN(D, A, B) lin_scan<D, A, B><<<grid, 32 * warps, smem, st>>>(q, k, ldq, hs, rep, v, ldv, rec, state, out, ldo, T, H, N, P, PB)
+#define DSK_LSCANS(D) do { if (N <= 32) DSK_LSCAN(D, 8, 1); else if (N <= 64) DSK_LSCAN(D, 16, 1); else if (N <= 128) DSK_LSCAN(D, 32, 1); else DSK_LSCAN(D, 32, 2); } while (0)
+  if (delta) DSK_LSCANS(true); else DSK_LSCANS(false);
+#undef DSK_LSCANS
+#undef DSK_LSCAN
+}
+
+static void launch_lin_decode(bool delta, const GdnP& D, const float* decay, float* state, const float* norm_w, float eps, int gate_off, float alpha,
+                              float* out, int ldo, cudaStream_t st) {
+  const int NG = std::min(kLinDecodeThreads / ((D.P + 3) / 4), D.N), need = (D.N + NG - 1) / NG;
+  const size_t smem = lin_decode_smem(D.N, D.P);
+#define DSK_LDEC(X, R) lin_decode<X, R><<<D.H, kLinDecodeThreads, smem, st>>>(D, decay, state, norm_w, eps, gate_off, alpha, out, ldo)
+#define DSK_LDECS(X) do { if (need <= 1) DSK_LDEC(X, 1); else if (need <= 2) DSK_LDEC(X, 2); else if (need <= 4) DSK_LDEC(X, 4); else if (need <= 8) DSK_LDEC(X, 8); else DSK_LDEC(X, 16); } while (0)
+  if (delta) DSK_LDECS(true); else DSK_LDECS(false);
+#undef DSK_LDECS
+#undef DSK_LDEC
+}
+
+// gated delta rule of T tokens from the raw projections in S->b0 (columns of att_layout) -> out rows (pitch ldo), times alpha
+static void gdn_forward(State* S, const HLayer& L, LayerState& ls, int ldp, const AttLayout& a, float* out, int ldo, float alpha, float eps, int T, cudaStream_t st) {
+  const dsk_layer_spec& sp = L.sp;
+  const int H = sp.gdn_heads, G = sp.gdn_kv_heads, N = sp.gdn_dim, P = sp.gdn_vdim, RV = H * P, NP = (N + 3) & ~3, CH = 2 * G * N + RV;
+  const GdnP D{S->b0, ldp, (int)a.dq, (int)a.db, (int)a.da, L.gdn_conv_w, L.A_log, L.dt_bias, ls.hist, sp.gdn_conv - 1 + kConvSpare, sp.gdn_conv, T, H, G, N, P, S->d_ctl};
+  if (T <= kLinDecodeTokens && lin_decode_fits(N, P)) {
+    launch_lin_decode(true, D, nullptr, ls.lin, L.lin_norm, eps, (int)a.dg, alpha, out, ldo, st);
+    S->launches++;
+    return;
+  }
+  const int nb = (T + kLinBlk - 1) / kLinBlk;
+  const size_t smem = (size_t)(2 * kLinBlk * (NP + 4) + 2 * kLinBlk * kLinBlk + 8 * kLinBlk * kLinBlk) * 4;
+  gdn_prepare<<<dim3((unsigned)nb, (unsigned)(G + (RV + 255) / 256)), 256, smem, st>>>(D, S->lq, S->lk, S->lv, NP, S->lrec);
+  launch_lin_scan(true, S->lq, S->lk, G * NP, NP, H / G, S->lv, RV, S->lrec, ls.lin, S->lout, RV, T, H, N, P, st);
+  if (sp.gdn_conv > 1) { conv_ring_store<<<(CH + 127) / 128, 128, 0, st>>>(S->b0, ldp, (int)a.dq, ls.hist, D.ring, T, CH, sp.gdn_conv, S->d_ctl); S->launches++; }
+  head_rmsnorm<<<(unsigned)(((long long)T * H + 7) / 8), 256, 0, st>>>(S->lout, RV, L.lin_norm, out, ldo, T, H, P, eps, S->b0 + a.dg, ldp, alpha);
+  S->launches += 3;
+}
+
+// lightning attention of T tokens from [silu q | silu k | silu v | sigmoid g] rows in S->b0 -> S->lout (ahead of the norm)
+static void lightning_forward(State* S, const HLayer& L, LayerState& ls, int ldp, int T, cudaStream_t st) {
+  const dsk_layer_spec& sp = L.sp;
+  const int H = sp.lin_heads, N = sp.lin_dim, P = sp.lin_vdim, HN = H * N, HP = H * P;
+  if (T <= kLinDecodeTokens && lin_decode_fits(N, P)) {
+    const GdnP D{S->b0, ldp, 0, 0, 0, nullptr, nullptr, nullptr, nullptr, 1, 1, T, H, H, N, P, S->d_ctl};
+    launch_lin_decode(false, D, L.decay, ls.lin, nullptr, 0.f, 0, 1.f, S->lout, HP, st);
+    S->launches++;
+    return;
+  }
+  lin_gram<<<dim3((unsigned)((T + kLinBlk - 1) / kLinBlk), (unsigned)H), 256, (size_t)2 * kLinBlk * (((N + 3) & ~3) + 4) * 4, st>>>(S->b0, S->b0 + HN, ldp, L.log_decay, T, H, N, S->lrec);
+  launch_lin_scan(false, S->b0, S->b0 + HN, ldp, N, 1, S->b0 + 2 * HN, ldp, S->lrec, ls.lin, S->lout, HP, T, H, N, P, st);
+  S->launches += 2;
+}
+
 static int R0(const Model* M, size_t ri) { return M->runs[ri].owner_run; }
 
 static void launch_attn(const float* qa, const float* cache, float* out, int T, int H, int R, const int* ctl, int mask, int window, int ring,
@@ -1150,8 +1403,8 @@ static void enqueue_head(dsk_model* m, dsk_state* s, int first, int count, cudaS
   State* S = s->hy;
   const dsk_hybrid_config& c = M->c;
   GemmP P = gp(S->h, c.dim, c.tie_head ? M->embed.p : M->head.p, c.dim, S->logits, c.vocab_size, count, c.vocab_size, c.dim);
-  P.a_map = S->d_want + first; P.alpha = c.logit_scale;
-  linear(S, c.quant == DSK_BF16, HEPI_STORE, P, 1, st);
+  P.a_map = S->d_want + first; P.alpha = c.logit_scale; P.lim = c.logit_softcap;
+  linear(S, c.quant == DSK_BF16, c.logit_softcap > 0.f ? HEPI_SOFTCAP : HEPI_STORE, P, 1, st);
 }
 
 // the model's norm over the T rows of `in` (width values each): stored into `out`, or added into it times alpha (mode 1)
@@ -1178,15 +1431,15 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
   State* S = s->hy;
   const dsk_hybrid_config& c = M->c;
   const bool bf = c.quant == DSK_BF16;
-  const bool sandwich = c.block == DSK_BLOCK_SANDWICH, post = c.block == DSK_BLOCK_POST;
+  const bool sandwich = c.block == DSK_BLOCK_SANDWICH, post = c.block == DSK_BLOCK_POST, pre = c.block == DSK_BLOCK_PRE;
   const int W = c.dim;
   const float mult = c.residual_mult;
   const float es = c.embed_scale != 0.f ? c.embed_scale : 1.f;
   const int nb = c.bigram_buckets;
   if (bf) embed_rows<__nv_bfloat16><<<T, 256, 0, st>>>(S->d_tok, (const __nv_bfloat16*)M->embed.p, W, S->x, es, nb > 0 ? (const __nv_bfloat16*)M->bigram.p : nullptr,
-                                                       nb, c.bigram_mul_prev, c.bigram_mul_cur, S->d_ctl, S->d_prev);
+                                                       nb, c.bigram_mul_prev, c.bigram_mul_cur, S->d_ctl, S->d_prev, S->emb);
   else embed_rows<float><<<T, 256, 0, st>>>(S->d_tok, (const float*)M->embed.p, W, S->x, es, nb > 0 ? (const float*)M->bigram.p : nullptr, nb, c.bigram_mul_prev,
-                                            c.bigram_mul_cur, S->d_ctl, S->d_prev);
+                                            c.bigram_mul_cur, S->d_ctl, S->d_prev, S->emb);
   S->launches++;
   if (nb > 0) { carry_token<<<1, 1, 0, st>>>(S->d_tok, T, S->d_prev); S->launches++; }   // the next step's first token pairs with this step's last
   if (pos0 < 0) S->tl_used = 0;   // a captured step records no events
@@ -1239,7 +1492,11 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
     const bool has_next = ri + 1 < M->runs.size();
     const float* hin = S->h;   // what the mixer reads
     if (post) { if (!h_ready) hin = open_post(L.canon1, 0); }
-    else if (!h_ready) {
+    else if (pre) {   // a pass of the layer loop opens with its vector (and, but for the first, the embedding) added to the stream
+      const bool again = c.loop_embed && run.pass > 0;
+      rms_open<<<T, 256, 0, st>>>(S->x, again ? S->emb : nullptr, run.pass >= 0 ? M->loop_step + (size_t)run.pass * W : nullptr, L.norm1, S->h, W, c.norm_eps);
+      S->launches++;
+    } else if (!h_ready) {
       if (run.pass >= 0) {   // a pass of the layer loop opens with its own vector added to the residual stream
         add_row<<<T, 256, 0, st>>>(S->x, W, M->loop_step + (size_t)run.pass * W, W);
         S->launches++;
@@ -1276,9 +1533,13 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       float *kc = (float*)S->L[R0(M, ri)].cache, *vc = (float*)S->L[R0(M, ri)].vcache;
       const ScoreMods sm{sp.att_softcap, sp.att_rel_max > 0 ? L.rel : nullptr, L.rel_bucket, sp.att_rel_max, sp.att_sink ? L.sink : nullptr, keep};
       MK("norm");
-      const int HV = sp.att_out_gate ? H * V : 0;   // the output gate's raw values come out of the stacked product, behind q / k / v
-      const int ldp = reads ? HD + HV : HD + GD + GV + HV;
-      const float* gate = HV ? S->b0 + (ldp - HV) : nullptr;
+      const AttLayout lay = att_layout(sp);
+      const int HV = (int)lay.gate_rows;   // the output gate's raw values come out of the stacked product
+      const int ldp = reads ? HD + HV : (int)lay.total;
+      const float* gate = HV ? S->b0 + (reads ? HD : (int)lay.gate) : nullptr;
+      const int gate_head = sp.att_out_gate == DSK_GATE_HEAD;
+      const int ldo = H * V + (sp.mixer2 ? (int)gdn_v(sp) : 0);   // a second mixer's heads stand behind this one's
+      const float lscale = sp.mixer2 ? sp.mix_scale : 1.f;
       if (reads) {
         linear(S, bf, HEPI_STORE, gp(hin, W, L.qkv.p, W, S->b0, ldp, T, ldp, W), 1, st);
         MK("att.qk");
@@ -1325,12 +1586,12 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
           softmax_band<<<dim3((unsigned)Tq, (unsigned)H), 128, 0, st>>>(pr, Tq, Lk, first, qpos0, sp.att_mask, sp.att_window, nk, sm);
           S->launches++;
           MK("att.softmax");
-          GemmP Ov = gp(pr, Lk, S->vf, Lk, S->b3 + (size_t)t0 * H * V, H * V, Tq, V, Lk);
-          Ov.sA = (long long)Tq * Lk; Ov.sW = (long long)V * Lk; Ov.z_wdiv = rep; Ov.sC = V;
+          GemmP Ov = gp(pr, Lk, S->vf, Lk, S->b3 + (size_t)t0 * ldo, ldo, Tq, V, Lk);
+          Ov.sA = (long long)Tq * Lk; Ov.sW = (long long)V * Lk; Ov.z_wdiv = rep; Ov.sC = V; Ov.alpha = lscale;
           linear(S, false, HEPI_STORE, Ov, H, st);
           MK("att.pv");
         }
-        if (gate) { gate_rows<<<T, 256, 0, st>>>(S->b3, H * V, gate, ldp, H * V); S->launches++; }   // heads *= sigmoid(g h)
+        if (gate) { gate_rows<<<T, 256, 0, st>>>(S->b3, ldo, gate, ldp, H * V, gate_head ? V : 1); S->launches++; }   // heads *= sigmoid(g h)
       } else {
         int NS = 1;
         if (T <= kAttnSplitTokens) NS = std::max(1, std::min((std::min(sp.att_window, ring) + keep + 31) / 32, kAttnSplitMax));
@@ -1340,12 +1601,16 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
           for (int d = G; d >= 1; d--) if (G % d == 0 && d * rep >= 4) GL = d;
         gqa_attn<<<dim3((unsigned)T, (unsigned)NS, (unsigned)(G / GL)), 256, gqa_attn_smem_floats(H, G, D, V) * 4, st>>>(
             S->b2, kc, vc, S->b3, sp.att_talk ? L.talk : nullptr, T, H, G, D, V, S->d_ctl, sp.att_mask, sp.att_window, ring, sp.att_scale, NS, S->part, sm,
-            NS > 1 ? nullptr : gate, ldp);
-        if (NS > 1) latent_swa_merge<<<dim3((unsigned)(T * H), (unsigned)((V + 127) / 128)), 128, 0, st>>>(S->part, S->b3, V, NS, gate, ldp, H);
+            NS > 1 ? nullptr : gate, ldp, gate_head, ldo, lscale);
+        if (NS > 1) latent_swa_merge<<<dim3((unsigned)(T * H), (unsigned)((V + 127) / 128)), 128, 0, st>>>(S->part, S->b3, V, NS, gate, ldp, H, gate_head, ldo, lscale);
         S->launches += NS > 1 ? 2 : 1;
         MK("att.decode");
       }
-      GemmP P = gp(S->b3, H * V, L.o.p, H * V, sink.C, W, T, W, H * V);
+      if (sp.mixer2 == DSK_MIX_GDN) {
+        gdn_forward(S, L, ls, ldp, lay, S->b3 + H * V, ldo, sp.mix2_scale, c.norm_eps, T, st);
+        MK("gdn");
+      }
+      GemmP P = gp(S->b3, ldo, L.o.p, ldo, sink.C, W, T, W, ldo);   // both mixers' output matrices in one product
       P.alpha = sink.alpha;
       linear(S, bf, sink.epi, P, 1, st);
       MK("att.o");
@@ -1413,6 +1678,34 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       P.alpha = sink.alpha;
       linear(S, bf, sink.epi, P, 1, st);
       MK("att.o");
+    } else if (sp.mixer == DSK_MIX_GDN) {
+      const AttLayout lay = att_layout(sp);
+      const int ldp = (int)lay.total, RV = (int)gdn_v(sp);
+      MK("norm");
+      linear(S, bf, HEPI_STORE, gp(hin, W, L.qkv.p, W, S->b0, ldp, T, ldp, W), 1, st);
+      MK("gdn.in");
+      gdn_forward(S, L, ls, ldp, lay, S->b3, RV, 1.f, c.norm_eps, T, st);
+      MK("gdn");
+      GemmP P = gp(S->b3, RV, L.o.p, RV, sink.C, W, T, W, RV);
+      P.alpha = sink.alpha;
+      linear(S, bf, sink.epi, P, 1, st);
+      MK("gdn.o");
+    } else if (sp.mixer == DSK_MIX_LIGHTNING) {
+      const int HN = sp.lin_heads * sp.lin_dim, HP = sp.lin_heads * sp.lin_vdim, pw = 2 * HN + 2 * HP;
+      MK("norm");
+      GemmP In = gp(hin, W, L.lin_in.p, W, S->b0, pw, T, pw, W);   // [silu q | silu k | silu v | sigmoid g]: the activations run in the product's epilogue
+      In.aux_off = 2 * HN + HP;
+      linear(S, bf, HEPI_SILU_SIG, In, 1, st);
+      MK("lin.in");
+      lightning_forward(S, L, ls, pw, T, st);
+      MK("lin.scan");
+      group_rmsnorm<float><<<T, 256, 0, st>>>(S->lout, HP, L.mnorm, S->b3, HP, HP, 1, c.norm_eps, 0, 0.f, nullptr, 0, S->b0 + 2 * HN + HP, pw);
+      S->launches++;
+      MK("lin.norm");
+      GemmP P = gp(S->b3, HP, L.o.p, HP, sink.C, W, T, W, HP);
+      P.alpha = sink.alpha;
+      linear(S, bf, sink.epi, P, 1, st);
+      MK("lin.o");
     } else if (sp.mixer == DSK_MIX_HGRN2) {
       const int H = sp.lin_heads, HN = H * sp.lin_dim, HP = H * sp.lin_vdim, pw = 2 * HN + HP;
       MK("norm");
@@ -1529,11 +1822,17 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       }
       MK("norm");
     }
-    if (sp.ff_kind == DSK_FF_DENSE && sp.ff_act == DSK_ACT_GEGLU) {
+    if (pre && sp.ff_kind != DSK_FF_NONE) {
+      rms_open<<<T, 256, 0, st>>>(S->x, nullptr, nullptr, L.norm2, S->h, W, c.norm_eps);
+      S->launches++;
+      hin = S->h;
+      MK("norm");
+    }
+    if (sp.ff_kind == DSK_FF_DENSE && sp.ff_act != DSK_ACT_XIELU) {
       const int ff = sp.ff_hidden;
       GemmP U = gp(hin, W, L.gate_d.p, W, S->b2, ff, T, ff, W);
-      U.W2 = L.up.p;
-      linear(S, bf, HEPI_GEGLU, U, 1, st);
+      U.W2 = L.up.p; U.lim = sp.ff_limit;
+      linear(S, bf, sp.ff_act == DSK_ACT_GLU_CLAMPED ? HEPI_GLU : HEPI_GEGLU, U, 1, st);
       MK("ff.up");
       GemmP Dn = gp(S->b2, ff, L.down.p, ff, sink.C, W, T, W, ff);
       Dn.alpha = sink.alpha;

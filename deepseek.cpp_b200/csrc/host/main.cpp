@@ -8,6 +8,7 @@
 #include <cstdio>
 #include <cstdlib>
 #include <cstring>
+#include <deque>
 #include <fstream>
 #include <iostream>
 #include <memory>
@@ -327,10 +328,67 @@ static bool nalizen_config_from(const JValue& j, const std::string& quant, int c
   return true;
 }
 
+// The Zetivik design: pre-norm blocks whose norm weights are stored around zero, a layer loop that adds the embedding again, a tied
+// head with a logit cap; layers of grouped-query attention (biases, weighted per-head query / key norm, half-split rotation, chunk
+// mask, one output gate per head) beside the gated delta rule, or of lightning attention; clamped gated feed-forwards.
+static bool zetivik_config_from(const JValue& j, const std::string& quant, int context, dsk_hybrid_config* hc, std::vector<dsk_layer_spec>* specs) {
+  static std::deque<std::vector<float>> decays;   // the specs point at them until the model is created
+  const JValue& layers = j.at("layers");
+  if (layers.kind != JValue::Arr || layers.arr.empty()) { fprintf(stderr, "FATAL: config.json has no layers\n"); return false; }
+  *hc = dsk_hybrid_config{};
+  hc->dim = j.integer("width", 0); hc->vocab_size = j.integer("vocab", 0); hc->n_layers = (int)layers.arr.size();
+  hc->max_seq_len = context > 0 ? context : 1 << 30;
+  hc->quant = quant == "fp32" ? DSK_F32 : DSK_BF16;
+  hc->chunk = context > 0 ? std::min(256, context) : 256;
+  hc->norm_eps = (float)j.at("norm").number("eps", 1e-5); hc->norm_groups = 1;
+  hc->residual_mult = 1.f; hc->logit_scale = 1.f;
+  hc->block = DSK_BLOCK_PRE; hc->norm_kind = DSK_NORM_RMS; hc->norm_one_plus = 1; hc->tie_head = 1;
+  hc->logit_softcap = (float)j.number("logit_softcap", 0.0);
+  if (j.has("loop")) {
+    const JValue& loop = j.at("loop");
+    hc->loop_start = loop.integer("start", 0); hc->loop_stop = loop.integer("stop", 0); hc->loop_times = loop.integer("times", 0); hc->loop_embed = 1;
+  }
+  for (size_t i = 0; i < layers.arr.size(); i++) {
+    const JValue& lc = layers.arr[i];
+    const JValue& mx = lc.at("mixer");
+    const std::string type = lc.at("type").str;
+    dsk_layer_spec sp{};
+    sp.att_kv_from = -1;
+    if (type == "parallel") {
+      const JValue &a = mx.at("left"), &b = mx.at("right");
+      sp.mixer = DSK_MIX_GQA; sp.mixer2 = DSK_MIX_GDN;
+      sp.mix_scale = (float)mx.number("left_scale", 1.0); sp.mix2_scale = (float)mx.number("right_scale", 1.0);
+      sp.att_heads = a.integer("heads", 0); sp.att_kv_heads = a.integer("kv_heads", sp.att_heads);
+      sp.att_dim = a.integer("dim", 0); sp.att_vdim = a.integer("vdim", 0); sp.att_scale = (float)a.number("scale", 1.0);
+      sp.att_mask = DSK_MASK_CHUNK; sp.att_window = a.at("mask").integer("size", 1 << 30);
+      sp.att_value_proj = 1; sp.att_bias = 1; sp.att_out_gate = DSK_GATE_HEAD; sp.att_qk_norm = DSK_QKNORM_HEAD_WEIGHT;
+      sp.rot_dims = a.at("rot").integer("dims", 0); sp.rot_base = (float)a.at("rot").number("base", 10000.0); sp.rot_layout = DSK_ROT_HALF;
+      sp.gdn_heads = b.integer("heads", 0); sp.gdn_kv_heads = b.integer("kv_heads", sp.gdn_heads);
+      sp.gdn_dim = b.integer("dim", 0); sp.gdn_vdim = b.integer("vdim", 0); sp.gdn_conv = b.integer("conv", 0);
+    } else if (type == "lightning") {
+      sp.mixer = DSK_MIX_LIGHTNING;
+      sp.lin_heads = mx.integer("heads", 0); sp.lin_dim = mx.integer("dim", 0); sp.lin_vdim = mx.integer("vdim", 0);
+      const JValue& dec = mx.at("decay");
+      if (dec.kind != JValue::Arr || (int)dec.arr.size() != sp.lin_heads) { fprintf(stderr, "FATAL: layer %zu: one decay per head is needed\n", i); return false; }
+      decays.emplace_back();
+      for (const JValue& d : dec.arr) decays.back().push_back((float)d.num);
+      sp.lin_decay = decays.back().data();
+    } else { fprintf(stderr, "FATAL: layer %zu: unknown mixer type %s\n", i, type.c_str()); return false; }
+    if (lc.has("mlp")) {
+      const JValue& ff = lc.at("mlp");
+      if (ff.at("kind").str != "dense") { fprintf(stderr, "FATAL: layer %zu: unknown feed-forward kind %s\n", i, ff.at("kind").str.c_str()); return false; }
+      sp.ff_kind = DSK_FF_DENSE; sp.ff_hidden = ff.integer("ff", 0); sp.ff_act = DSK_ACT_GLU_CLAMPED; sp.ff_limit = (float)ff.number("limit", 0.0);
+    }
+    specs->push_back(sp);
+  }
+  return true;
+}
+
 // config.json "architecture" -> builder of the C-ABI model description
 typedef bool (*ArchBuilder)(const JValue&, const std::string&, int, dsk_hybrid_config*, std::vector<dsk_layer_spec>*);
 static const struct { const char* name; ArchBuilder build; } kArchitectures[] = {{"Desarax", hybrid_config_from}, {"Rutulix", rutulix_config_from},
-                                                                                {"Sakusun", sakusun_config_from}, {"Nalizen", nalizen_config_from}};
+                                                                                {"Sakusun", sakusun_config_from}, {"Nalizen", nalizen_config_from},
+                                                                                {"Zetivik", zetivik_config_from}};
 
 // completion over token ids: the prompt goes through dsk_forward_chunk (prefill in portions), then the usual
 // dsk_sample -> dsk_forward loop; the ids are printed (these checkpoints carry no tokenizer).
@@ -344,7 +402,7 @@ static int run_layer_list(const std::string& dir, const std::string& quant, cons
   const std::string arch = cfg.at("architecture").str;
   ArchBuilder builder = nullptr;
   for (const auto& a : kArchitectures) if (arch == a.name) builder = a.build;
-  if (!builder) { fprintf(stderr, "FATAL: unknown architecture '%s' (known: Desarax, Rutulix, Sakusun, Nalizen)\n", arch.c_str()); return 1; }
+  if (!builder) { fprintf(stderr, "FATAL: unknown architecture '%s' (known: Desarax, Rutulix, Sakusun, Nalizen, Zetivik)\n", arch.c_str()); return 1; }
   if (quant != "bf16" && quant != "fp32") { fprintf(stderr, "FATAL: -q must be bf16 or fp32\n"); return 1; }
   std::vector<int> enc;
   for (size_t i = 0; i < prompt_ids.size();) {

@@ -23,15 +23,16 @@ sys.path.insert(0, HERE)
 import dseek  # noqa: E402
 
 QUANT_IDS = {"fp32": 0, "fp16": 1, "f8e5m2": 2, "q2_k": 3, "q3_k": 4, "bf16": 5}
-MIX_SSD, MIX_LATENT_SWA, MIX_GQA, MIX_MLA, MIX_HGRN2 = 0, 1, 2, 3, 4
+MIX_SSD, MIX_LATENT_SWA, MIX_GQA, MIX_MLA, MIX_HGRN2, MIX_GDN, MIX_LIGHTNING = 0, 1, 2, 3, 4, 5, 6
 FF_NONE, FF_MOE, FF_DENSE = 0, 1, 2
 MASK_WINDOW, MASK_CHUNK = 0, 1
-ACT_XIELU, ACT_GEGLU = 0, 1
-BLOCK_PARALLEL, BLOCK_SANDWICH, BLOCK_POST = 0, 1, 2
+ACT_XIELU, ACT_GEGLU, ACT_GLU_CLAMPED = 0, 1, 2
+BLOCK_PARALLEL, BLOCK_SANDWICH, BLOCK_POST, BLOCK_PRE = 0, 1, 2, 3
 NORM_RMS, NORM_LAYER = 0, 1
 ROT_PAIRS, ROT_HALF = 0, 1
 ROTSCALE_YARN, ROTSCALE_BANDS = 0, 1
-QKNORM_WHOLE, QKNORM_HEAD = 0, 1
+QKNORM_WHOLE, QKNORM_HEAD, QKNORM_HEAD_WEIGHT = 0, 1, 2
+GATE_NONE, GATE_ENTRY, GATE_HEAD = 0, 1, 2
 ROUTER_SIGMOID, ROUTER_TOP_SOFTMAX = 0, 1
 EXPERT_GLU_CLAMPED, EXPERT_RELU2 = 0, 1
 HYDRATE_KV_CACHE, OUTPUT_LOGITS = 0, 1
@@ -103,7 +104,9 @@ class LayerSpec(C.Structure):
                [(n, C.c_int) for n in ("att_value_proj", "att_bias", "att_keep_first", "att_rel_max", "att_sink", "att_vmix")] + \
                [("att_softcap", C.c_float)] + \
                [(n, C.c_int) for n in ("att_q_rank", "att_rot_dim", "att_out_gate", "rot_layout", "rot_scale", "att_qk_norm",
-                                       "lin_heads", "lin_dim", "lin_vdim", "ff_router", "ff_expert")]
+                                       "lin_heads", "lin_dim", "lin_vdim", "ff_router", "ff_expert", "mixer2")] + \
+               [("mix_scale", C.c_float), ("mix2_scale", C.c_float)] + \
+               [(n, C.c_int) for n in ("gdn_heads", "gdn_kv_heads", "gdn_dim", "gdn_vdim", "gdn_conv")] + [("lin_decay", f32p)]
 
 
 class HybridConfig(C.Structure):
@@ -114,7 +117,7 @@ class HybridConfig(C.Structure):
                [(n, C.c_int) for n in ("block", "norm_kind", "tie_head", "loop_start", "loop_stop", "loop_times")] + \
                [("embed_scale", C.c_float)] + \
                [(n, C.c_int) for n in ("bigram_buckets", "bigram_mul_prev", "bigram_mul_cur", "norm_scalar", "canon_taps", "res_gate", "layer_scale",
-                                       "norm_bias", "token_shift")]
+                                       "norm_bias", "token_shift", "norm_one_plus", "loop_embed")] + [("logit_softcap", C.c_float)]
 
 
 # mixer "type" strings of a layer-list config.json -> mixer kernel family.  Two names may map to one mechanism.
@@ -332,11 +335,69 @@ def nalizen_from_config(cfg: dict, quant: str = "bf16", max_seq_len: int = 0, ch
     return hc, specs
 
 
+def zetivik_from_config(cfg: dict, quant: str = "bf16", max_seq_len: int = 0, chunk: int = 256):
+    """config.json of the Zetivik design -> (HybridConfig, LayerSpec array): pre-norm blocks whose norm weights are stored around
+    zero, a layer loop that adds the embedding again ahead of every pass but the first, a tied head with a logit cap, and per layer
+    either grouped-query attention (biases, weighted per-head query / key norm, half-split rotation, chunk mask, one output gate per
+    head) beside the gated delta rule on the same input, or lightning attention; clamped gated feed-forwards.  Absent keys switch a
+    part off."""
+    hc = HybridConfig()
+    layers = cfg["layers"]
+    hc.dim, hc.vocab_size, hc.n_layers = int(cfg["width"]), int(cfg["vocab"]), len(layers)
+    hc.quant, hc.chunk = QUANT_IDS[quant], int(chunk)
+    hc.max_seq_len = int(max_seq_len) if max_seq_len else 1 << 30
+    hc.norm_eps, hc.norm_groups = float(cfg["norm"]["eps"]), 1
+    hc.residual_mult, hc.logit_scale, hc.side_dim = 1.0, 1.0, 0
+    hc.block, hc.norm_kind, hc.norm_one_plus, hc.tie_head = BLOCK_PRE, NORM_RMS, 1, 1
+    hc.logit_softcap = float(cfg.get("logit_softcap") or 0.0)
+    loop = cfg.get("loop")
+    if loop:            # a loop of one pass is still a loop: its pass vector is added before the range
+        hc.loop_start, hc.loop_stop, hc.loop_times, hc.loop_embed = int(loop["start"]), int(loop["stop"]), int(loop["times"]), 1
+    specs = (LayerSpec * len(layers))()
+    keep = []           # the decay arrays the specs point at
+    for i, lc in enumerate(layers):
+        sp, mx = specs[i], lc["mixer"]
+        sp.att_kv_from = -1
+        if lc["type"] == "parallel":
+            a, b = mx["left"], mx["right"]
+            sp.mixer, sp.mixer2 = MIX_GQA, MIX_GDN
+            sp.mix_scale, sp.mix2_scale = float(mx["left_scale"]), float(mx["right_scale"])
+            sp.att_heads, sp.att_kv_heads = int(a["heads"]), int(a.get("kv_heads", a["heads"]))
+            sp.att_dim, sp.att_vdim, sp.att_scale = int(a["dim"]), int(a["vdim"]), float(a["scale"])
+            mask = a.get("mask") or {}
+            sp.att_mask = MASK_CHUNK
+            sp.att_window = int(mask["size"]) if "size" in mask else 1 << 30      # no mask size: one chunk, plain causal attention
+            sp.att_value_proj, sp.att_bias, sp.att_out_gate, sp.att_qk_norm = 1, 1, GATE_HEAD, QKNORM_HEAD_WEIGHT
+            rot = a.get("rot") or {}
+            sp.rot_dims, sp.rot_base, sp.rot_layout = int(rot.get("dims", 0)), float(rot.get("base", 10000.0)), ROT_HALF
+            sp.gdn_heads, sp.gdn_kv_heads = int(b["heads"]), int(b.get("kv_heads", b["heads"]))
+            sp.gdn_dim, sp.gdn_vdim, sp.gdn_conv = int(b["dim"]), int(b["vdim"]), int(b["conv"])
+        elif lc["type"] == "lightning":
+            sp.mixer = MIX_LIGHTNING
+            sp.lin_heads, sp.lin_dim, sp.lin_vdim = int(mx["heads"]), int(mx["dim"]), int(mx["vdim"])
+            if len(mx["decay"]) != sp.lin_heads:
+                raise DskError(f"layer {i}: {len(mx['decay'])} decays for {sp.lin_heads} heads")
+            keep.append((C.c_float * sp.lin_heads)(*[float(v) for v in mx["decay"]]))
+            sp.lin_decay = C.cast(keep[-1], f32p)
+        else:
+            raise DskError(f"layer {i}: unknown mixer type {lc['type']!r}")
+        ff = lc.get("mlp")
+        if ff:
+            if ff.get("kind") != "dense":
+                raise DskError(f"layer {i}: unknown feed-forward kind {ff.get('kind')!r}")
+            sp.ff_kind, sp.ff_hidden, sp.ff_act, sp.ff_limit = FF_DENSE, int(ff["ff"]), ACT_GLU_CLAMPED, float(ff["limit"])
+        else:
+            sp.ff_kind = FF_NONE
+    specs.keep = keep
+    return hc, specs
+
+
 # config.json "architecture" -> builder of the C-ABI model description (the DeepSeek families come as .dseek metadata instead)
-ARCHITECTURES = {"Desarax": hybrid_from_config, "Rutulix": rutulix_from_config, "Sakusun": sakusun_from_config, "Nalizen": nalizen_from_config}
+ARCHITECTURES = {"Desarax": hybrid_from_config, "Rutulix": rutulix_from_config, "Sakusun": sakusun_from_config, "Nalizen": nalizen_from_config,
+                 "Zetivik": zetivik_from_config}
 
 _lib = None
-ABI_VERSION = 7   # DSK_ABI_VERSION (include/dsk.h)
+ABI_VERSION = 8   # DSK_ABI_VERSION (include/dsk.h)
 
 
 def build(force: bool = False) -> str:

@@ -20,7 +20,7 @@
 extern "C" {
 #endif
 
-#define DSK_ABI_VERSION 7
+#define DSK_ABI_VERSION 8
 
 /* Quant: src/codec.h:79-85 (same numbering) */
 enum { DSK_F32 = 0, DSK_F16 = 1, DSK_F8E5M2 = 2, DSK_Q2_K = 3, DSK_Q3_K = 4,
@@ -71,15 +71,21 @@ typedef struct dsk_config {
  * DSK_FF_DENSE feed-forwards, a scaled embedding plus bigram table and an untied head; the Nalizen design is DSK_BLOCK_POST with
  * layer norms that carry a bias, a token shift in front of every mixer, DSK_MIX_GQA mixers (half-split rotation with wavelength-band
  * scaling, per-head query / key norm after the rotation, output gate, shared key / value caches) or DSK_MIX_HGRN2 mixers, gated dense
- * or DSK_ROUTER_TOP_SOFTMAX / DSK_EXPERT_RELU2 routed feed-forwards, a scaled and tied embedding and the per-layer token input.) */
-enum { DSK_MIX_SSD = 0, DSK_MIX_LATENT_SWA = 1, DSK_MIX_GQA = 2, DSK_MIX_MLA = 3, DSK_MIX_HGRN2 = 4 };
+ * or DSK_ROUTER_TOP_SOFTMAX / DSK_EXPERT_RELU2 routed feed-forwards, a scaled and tied embedding and the per-layer token input; the
+ * Zetivik design is DSK_BLOCK_PRE with RMS norms whose weight is stored around zero, layers of two mixers side by side (DSK_MIX_GQA
+ * with half-split rotation, weighted per-head query / key norm, one output gate per head and a chunk mask, beside DSK_MIX_GDN) or of
+ * DSK_MIX_LIGHTNING, clamped dense feed-forwards, a layer loop that adds the embedding again, a tied head and a logit cap.) */
+enum { DSK_MIX_SSD = 0, DSK_MIX_LATENT_SWA = 1, DSK_MIX_GQA = 2, DSK_MIX_MLA = 3, DSK_MIX_HGRN2 = 4,
+       DSK_MIX_GDN = 5, DSK_MIX_LIGHTNING = 6 };
 enum { DSK_FF_NONE = 0, DSK_FF_MOE = 1, DSK_FF_DENSE = 2 };
 enum { DSK_MASK_WINDOW = 0,   /* position i sees j with 0 <= i - j < att_window */
        DSK_MASK_CHUNK = 1 };  /* position i sees j <= i with floor(i / att_window) == floor(j / att_window): borders at multiples of att_window in sequence positions */
 enum { DSK_ACT_XIELU = 0,      /* z > 0: softplus(p) z^2 + z/2;  z <= 0: (1/2 + softplus(q)) (e^z - 1 - z) + z/2;  (p, q) = tensor mlp.act */
-       DSK_ACT_GEGLU = 1 };    /* gated: down(gelu_tanh(gate h) * (up h)), tensors mlp.gate / mlp.up / mlp.down, no biases */
+       DSK_ACT_GEGLU = 1,      /* gated: down(gelu_tanh(gate h) * (up h)), tensors mlp.gate / mlp.up / mlp.down, no biases */
+       DSK_ACT_GLU_CLAMPED = 2 };   /* gated: down(g sigmoid(1.702 g) (u + 1)), g = min(gate h, ff_limit), u = clamp(up h, +-ff_limit), the same tensors */
 enum { DSK_BLOCK_PARALLEL = 0,   /* h = norm1(x); x += residual_mult (mixer(h) + ff(h)) */
        DSK_BLOCK_SANDWICH = 1,   /* x += norm1b(mixer(norm1(x))); x += norm2b(ff(norm2(x))) */
+       DSK_BLOCK_PRE = 3,        /* x += residual_mult mixer(norm1(x)); x += residual_mult ff(norm2(x)) */
        DSK_BLOCK_POST = 2 };     /* the sublayers read the stream itself and only their result is normalised:
                                     u = x + conv(x) (canon_taps > 0; else u = x);  y = f(u) (* sigmoid(rg x + rg.b) with res_gate);
                                     x += norm(y) (* ls with layer_scale), for f = mixer (tensors norm1, canon1, rg1, ls1), then feed-forward (..2) */
@@ -91,7 +97,10 @@ enum { DSK_ROTSCALE_YARN = 0,    /* rot_factor > 0: YaRN ramp between rot_fast a
        DSK_ROTSCALE_BANDS = 1 }; /* rot_factor > 0: by wavelength l = 2 pi / f: f kept where l < rot_original / rot_fast, f / rot_factor where
                                     l > rot_original / rot_slow, between them (1 - s) f / rot_factor + s f with s = (rot_original / l - rot_slow) / (rot_fast - rot_slow) */
 enum { DSK_QKNORM_WHOLE = 0,     /* RMS norm with weights mix.q.norm / mix.k.norm over the whole projection, before the rotation */
-       DSK_QKNORM_HEAD = 1 };    /* every head of q and k divided by its own RMS after the rotation, no weight */
+       DSK_QKNORM_HEAD = 1,      /* every head of q and k divided by its own RMS after the rotation, no weight */
+       DSK_QKNORM_HEAD_WEIGHT = 2 };   /* every head divided by its own RMS and multiplied by mix.q.norm / mix.k.norm [att_dim], before the rotation */
+enum { DSK_GATE_NONE = 0, DSK_GATE_ENTRY = 1,   /* att_out_gate: heads multiplied by sigmoid(g h), one number per entry of the concatenated heads (mix.g [heads * vdim]) */
+       DSK_GATE_HEAD = 2 };      /* one number per head (mix.g [heads]); DSK_MIX_GQA */
 enum { DSK_ROUTER_SIGMOID = 0,   /* sigmoid scores, selection by score + mlp.correction, weights = chosen scores normalised x ff_router_scale */
        DSK_ROUTER_TOP_SOFTMAX = 1 };   /* logits = router h + mlp.router.b; the ff_top largest logits; weights = softmax over the chosen logits */
 enum { DSK_EXPERT_GLU_CLAMPED = 0,     /* down(g sigmoid(1.702 g) (u + 1)), g = min(gate h, limit), u = clamp(up h, +-limit) */
@@ -125,6 +134,17 @@ enum { DSK_EXPERT_GLU_CLAMPED = 0,     /* down(g sigmoid(1.702 g) (u + 1)), g = 
  *                       f = l + (1 - l) sigmoid(f h + f.b) with the lower bound l = tensor mix.lower; S <- diag(f) S + (1 - f) v^T,
  *                       o = S^T q; every head's o is RMS-normed with the weight mix.norm [lin_vdim] shared by the heads; output projection
  *                       mix.o.  Carries S [lin_heads][lin_dim][lin_vdim] in fp32 per sequence.
+ *   DSK_MIX_GDN         gated delta rule: q, k = mix.q h, mix.k h [gdn_kv_heads][gdn_dim], v = mix.v h [gdn_heads][gdn_vdim], each through a causal
+ *                       per-channel convolution of gdn_conv taps (mix.q.conv / k.conv / v.conv, last tap on the current token) and silu; q and k
+ *                       divided per head by sqrt(sum z^2 + 1e-6), q also by sqrt(gdn_dim); beta = sigmoid(mix.b h), g = exp(-exp(mix.A_log)
+ *                       softplus(mix.a h + mix.dt_bias)) per head; S <- g S, S <- S + k (beta (v - S^T k))^T, o = S^T q (head h uses q / k head
+ *                       h / (gdn_heads / gdn_kv_heads)); rms(o) mix.norm [gdn_vdim] silu(mix.g h); output projection mix.o.  Carries S
+ *                       [gdn_heads][gdn_dim][gdn_vdim] in fp32 and the convolutions' last inputs.
+ *   DSK_MIX_LIGHTNING   linear attention with a fixed decay per head: q, k = silu(.) [lin_heads][lin_dim], v = silu(.) [lin_heads][lin_vdim];
+ *                       S <- lin_decay[h] S + k v^T, o = S^T q; RMS norm with mix.norm over the concatenated heads, times sigmoid(mix.g h),
+ *                       output projection mix.o.  Carries S in fp32.
+ *   mixer2 = DSK_MIX_GDN runs beside a DSK_MIX_GQA mixer on the same input: x += residual_mult (mix_scale left + mix2_scale right), tensors
+ *                       mix.left.* and mix.right.*.
  *   DSK_FF_DENSE        down(act(up h + b_up)) + b_down with activation ff_act. */
 typedef struct dsk_layer_spec {
   int mixer;                                                            /* DSK_MIX_* */
@@ -145,6 +165,10 @@ typedef struct dsk_layer_spec {
   int rot_layout, rot_scale, att_qk_norm;                               /* DSK_MIX_GQA: DSK_ROT_*, DSK_ROTSCALE_*, DSK_QKNORM_* */
   int lin_heads, lin_dim, lin_vdim;                                     /* DSK_MIX_HGRN2 */
   int ff_router, ff_expert;                                             /* DSK_FF_MOE: DSK_ROUTER_*, DSK_EXPERT_* */
+  int mixer2;                                                           /* 0: one mixer; DSK_MIX_GDN: a second one beside it (above) */
+  float mix_scale, mix2_scale;
+  int gdn_heads, gdn_kv_heads, gdn_dim, gdn_vdim, gdn_conv;             /* DSK_MIX_GDN */
+  const float* lin_decay;                                               /* DSK_MIX_LIGHTNING (with lin_heads, lin_dim, lin_vdim): lin_heads decays, read by dsk_model_create_hybrid */
 } dsk_layer_spec;
 typedef struct dsk_hybrid_config {
   int dim, vocab_size, n_layers;
@@ -170,6 +194,9 @@ typedef struct dsk_hybrid_config {
   int norm_bias;             /* DSK_NORM_LAYER: every norm outside the mixers adds a bias, tensor "<norm>.b" */
   int token_shift;           /* 1: a mixer reads h + (h' - h) * shift (tensor l<i>.shift [dim]) instead of its input h, h' being the previous token's h
                                 (zeros for the first token of a sequence); the last h of every layer run is part of the sequence's state */
+  int norm_one_plus;         /* 1: the norms outside the mixers multiply by 1 + their stored weight */
+  int loop_embed;            /* 1: ahead of every loop pass but the first, the embedding output is added to the residual stream */
+  float logit_softcap;       /* > 0: logits <- cap tanh(logits / cap) */
 } dsk_hybrid_config;
 
 typedef struct dsk_model dsk_model;
