@@ -54,13 +54,14 @@ def softplus(z):
 
 
 def rotate_half(v, rot, pos):
-    """Entries (i, i + dims/2) of the first rot["dims"] entries of v turn together; the rest pass."""
+    """Entries (i, i + dims/2) of the first rot["dims"] entries of v turn together; the rest pass.  Positions and angles are
+    32-bit numbers in this design, so the angle is a 32-bit product here too."""
     out = np.array(v, dtype=np.float64)
     if not rot or not rot.get("dims"):
         return out
     half = rot["dims"] // 2
     for i in range(half):
-        a = pos * rot["base"] ** (-2.0 * i / rot["dims"])
+        a = float(np.float32(pos) * np.float32(rot["base"] ** (-2.0 * i / rot["dims"])))
         c, s = math.cos(a), math.sin(a)
         u, w = out[i], out[i + half]
         out[i], out[i + half] = u * c - w * s, w * c + u * s
@@ -206,6 +207,27 @@ def run(cfg, W, tokens):
     return np.array(logits), np.array(traces).transpose(1, 0, 2)
 
 
+class RoundedProduct:
+    """A matrix whose products round the vector to bfloat16 first."""
+
+    def __init__(self, w):
+        self.w = w
+
+    def __matmul__(self, x):
+        return self.w @ bf16_to_f64(to_bf16(np.asarray(x, dtype=np.float64))).reshape(np.shape(x))
+
+    def __getitem__(self, i):
+        return self.w[i]
+
+
+def rounding_noise(cfg, W, tokens):
+    """Per-token error of the logits (largest entry, in units of the largest logit) that rounding the activations of every matrix
+    product to bfloat16 causes on its own."""
+    R = {k: RoundedProduct(v) if v.ndim == 2 and not k.endswith(".conv") and k != "loop.step" else v for k, v in W.items()}
+    exact = run(cfg, W, tokens)[0]
+    return np.abs(run(cfg, R, tokens)[0] - exact).max(-1) / np.abs(exact).max()
+
+
 # ---- synthetic checkpoints ------------------------------------------------------------------------------------------------
 def tensor_shapes(cfg):
     Wd, V = cfg["width"], cfg["vocab"]
@@ -292,7 +314,7 @@ def par(left=None, right=None, cl=0.7, cr=1.1, ff=None, limit=1.5):
 
 def light(heads=3, dim=8, vdim=8, decay=None, ff=None, limit=1.5):
     """One lightning layer; decay: one number per head."""
-    return {"type": "lightning", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay or np.linspace(0.5, 0.99, heads))},
+    return {"type": "lightning", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": [float(d) for d in (np.linspace(0.5, 0.99, heads) if decay is None else decay)]},
             "mlp": ff_config(ff, limit)}
 
 

@@ -260,3 +260,74 @@ def test_nalizen_oracle_invariants(no):
     assert np.allclose(no.token_shift(np.array([1.0, 2.0]), np.array([3.0, 6.0]), np.array([0.0, 0.25])), [1.0, 3.0])
     y = no.layer_norm(np.array([1.0, 3.0]), np.array([2.0, 2.0]), np.array([0.5, 0.5]), 0.0)
     assert np.allclose(y, [-1.5, 2.5])
+
+
+# ---- the Zetivik design ----------------------------------------------------------------------------------------------------------
+@pytest.fixture(scope="module")
+def zo():
+    import zetivik_oracle
+    return zetivik_oracle
+
+
+def test_zetivik_config_to_layer_specs(zo):
+    import dsk
+    cfg = zo.small_config()
+    hc, specs = dsk.ARCHITECTURES[cfg["architecture"]](cfg, quant="fp32", max_seq_len=77, chunk=16)
+    assert (hc.dim, hc.vocab_size, hc.n_layers, hc.max_seq_len, hc.chunk, hc.quant) == (44, 61, 5, 77, 16, dsk.QUANT_IDS["fp32"])
+    assert (hc.block, hc.norm_kind, hc.norm_one_plus, hc.tie_head, hc.loop_start, hc.loop_stop, hc.loop_times, hc.loop_embed) == \
+        (dsk.BLOCK_PRE, dsk.NORM_RMS, 1, 1, 1, 3, 3, 1)
+    assert hc.logit_softcap == 8.0 and abs(hc.norm_eps - 1e-5) < 1e-12 and (hc.norm_bias, hc.token_shift, hc.norm_scalar, hc.side_dim) == (0, 0, 0, 0)
+    a, b, c = specs[0], specs[1], specs[2]
+    assert (a.mixer, a.mixer2) == (dsk.MIX_GQA, dsk.MIX_GDN) and abs(a.mix_scale - 0.7) < 1e-7 and abs(a.mix2_scale - 1.1) < 1e-7
+    assert (a.att_heads, a.att_kv_heads, a.att_dim, a.att_vdim, a.att_mask, a.att_window, a.att_kv_from) == (6, 2, 10, 6, dsk.MASK_CHUNK, 7, -1)
+    assert (a.att_value_proj, a.att_bias, a.att_out_gate, a.att_qk_norm, a.att_talk, a.att_sink, a.rot_layout, a.rot_dims) == \
+        (1, 1, dsk.GATE_HEAD, dsk.QKNORM_HEAD_WEIGHT, 0, 0, dsk.ROT_HALF, 6)
+    assert (a.gdn_heads, a.gdn_kv_heads, a.gdn_dim, a.gdn_vdim, a.gdn_conv) == (4, 2, 5, 7, 3)
+    assert (a.ff_kind, a.ff_hidden, a.ff_act) == (dsk.FF_DENSE, 28, dsk.ACT_GLU_CLAMPED) and abs(a.ff_limit - 0.8) < 1e-7
+    assert (b.mixer, b.mixer2, b.lin_heads, b.lin_dim, b.lin_vdim, b.ff_kind) == (dsk.MIX_LIGHTNING, 0, 3, 5, 9, dsk.FF_NONE)
+    assert np.allclose([b.lin_decay[h] for h in range(3)], [0.4, 0.9, 0.995], rtol=1e-6)
+    assert (c.gdn_kv_heads, c.gdn_conv, c.ff_kind) == (1, 5, dsk.FF_NONE)
+    left = cfg["layers"][0]["mixer"]["left"]
+    del left["rot"], left["mask"], left["kv_heads"], cfg["layers"][0]["mixer"]["right"]["kv_heads"]
+    del cfg["loop"], cfg["logit_softcap"]
+    hc, specs = dsk.zetivik_from_config(cfg)
+    assert (specs[0].rot_dims, specs[0].att_window, specs[0].att_kv_heads, specs[0].gdn_kv_heads, hc.loop_times, hc.logit_softcap) == (0, 1 << 30, 6, 4, 0, 0.0)
+    cfg["layers"][1]["mixer"]["decay"].append(0.5)
+    with pytest.raises(dsk.DskError):
+        dsk.zetivik_from_config(cfg)
+    cfg["layers"][1]["type"] = "hgrn2"
+    with pytest.raises(dsk.DskError):
+        dsk.zetivik_from_config(cfg)
+
+
+def test_zetivik_oracle_invariants(zo):
+    """(1) a sequence fed token by token equals the whole; (2) the order of layer runs; (3) chunk starts; (4) the delta rule
+    overwrites: with step size 1 and no decay, writing a second value under the same key replaces the first; (5) the convolution
+    pairs its last tap with the current input; (6) unit vectors; (7) the clamps of the feed-forward; (8) the cap."""
+    cfg = zo.small_config()
+    W = zo.random_weights(cfg, 5)
+    toks = np.arange(20) % 61
+    whole = zo.run(cfg, W, toks)[0]
+    seq = zo.Sequence(cfg, W)
+    assert np.allclose(np.array([seq.feed(int(t)) for t in toks]), whole, rtol=0, atol=1e-12)
+    assert zo.layer_runs(cfg) == [(0, None), (1, 0), (2, None), (1, 1), (2, None), (1, 2), (2, None), (3, None), (4, None)]
+    assert [zo.chunk_first(4, p) for p in (0, 3, 4, 7, 8)] == [0, 0, 4, 4, 8] and zo.chunk_first(None, 9) == 0
+    mx = {"heads": 1, "dim": 2, "vdim": 2}
+    big = 60.0
+    Wd = {"q": np.eye(2, 4), "k": np.eye(2, 4), "v": np.eye(4)[2:], "b": np.full((1, 4), big), "a": np.zeros((1, 4)), "A_log": np.array([-60.0]), "dt_bias": np.zeros(1),
+          "norm": np.ones(2), "g": np.ones((2, 4)), "o": np.eye(2)}
+    for n in "qkv":
+        Wd[n + ".conv"] = np.ones((2, 1))
+    Wd = {"m." + k: v for k, v in Wd.items()}
+    S, past = np.zeros((1, 2, 2)), {n: [] for n in "qkv"}
+    zo.delta_step(Wd, "m.", mx, np.array([30.0, 0.0, 1.0, 2.0]), S, past, 1e-6)
+    zo.delta_step(Wd, "m.", mx, np.array([30.0, 0.0, 5.0, 7.0]), S, past, 1e-6)
+    assert np.allclose(S[0, 0], zo.silu(np.array([5.0, 7.0])), rtol=1e-6) and np.allclose(S[0, 1], 0.0)
+    w = np.array([[1.0, 10.0, 100.0]])
+    assert zo.short_conv(w, [np.array([2.0]), np.array([3.0])], np.array([4.0]))[0] == 2.0 + 30.0 + 400.0
+    assert zo.short_conv(w, [], np.array([4.0]))[0] == 400.0
+    assert abs(np.linalg.norm(zo.unit(np.array([3.0, 4.0]))) - 1.0) < 1e-7
+    Wf = {"gate": np.array([[5.0]]), "up": np.array([[-9.0]]), "down": np.array([[1.0]])}
+    y = zo.clamped_glu({"f." + k: v for k, v in Wf.items()}, "f.", np.array([1.0]), 2.0)[0]
+    assert abs(y - 2.0 / (1.0 + np.exp(-3.404)) * (-1.0)) < 1e-12
+    assert abs(zo.soft_cap(np.array([1e9]), 4.0)[0] - 4.0) < 1e-9 and zo.soft_cap(np.array([3.0]), 0)[0] == 3.0
