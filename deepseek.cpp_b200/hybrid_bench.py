@@ -4,7 +4,9 @@ experts; the Rutulix sizes run beside the closest layer-list model, a Desarax mo
 layer runs, heads, mask size and feed-forward matrix elements; the Sakusun sizes run beside a Rutulix model (the framework's other
 attention-only design with dense feed-forwards) at equal width, depth, heads, window and feed-forward matrix elements; the
 Nalizen sizes run beside a Desarax model (the framework's other design with a recurrence, shared attention caches, routed
-feed-forwards and the per-layer token input) at equal width, depth, layer pattern, heads, window and active matrix elements.
+feed-forwards and the per-layer token input) at equal width, depth, layer pattern, heads, window and active matrix elements; the
+Zetivik sizes run beside a Nalizen model (the framework's other design of attention with an output gate, a gated linear recurrence
+and gated dense feed-forwards), one Nalizen layer per mixer of every layer run, at equal width, heads, sizes and feed-forwards.
 
 Used by `bench.py --hybrid`.  Random weights generated on the GPU (bf16), uploaded through dsk_upload_tensor(src_on_device).
 Decode is the device-side greedy loop (CUDA events around the captured step graph); prefill is dsk_forward_chunk over a prompt
@@ -40,7 +42,139 @@ SIZES = {
                           att_dim=64, rot=32, window=512, experts=16, top=2, ff=768, side=32),
     "nalizen_large": dict(design="Nalizen", width=2048, vocab=102400, pattern="rrarrArrarrA", lin_heads=16, lin_dim=128, lin_vdim=128, att_heads=16,
                           kv_heads=4, att_dim=128, rot=64, window=1024, experts=64, top=6, ff=2112, side=64),
+    # Zetivik: layers of attention beside the delta rule (p) and of lightning attention (l); layers loop[0] .. loop[1]-1 run loop[2] times
+    "zetivik_small": dict(design="Zetivik", width=1024, vocab=32000, pattern="plpplp", loop=(2, 4, 2), att_heads=16, kv_heads=4, att_dim=64, window=512,
+                          lin_heads=16, lin_kv_heads=8, lin_dim=64, lin_vdim=64, conv=4, ff=2816),
+    "zetivik_large": dict(design="Zetivik", width=2048, vocab=102400, pattern="plpplppl", loop=(3, 5, 2), att_heads=16, kv_heads=4, att_dim=128, window=1024,
+                          lin_heads=16, lin_kv_heads=8, lin_dim=128, lin_vdim=128, conv=4, ff=5632),
 }
+
+
+def zetivik_config(z):
+    layers = []
+    for ch in z["pattern"]:
+        if ch == "l":
+            H = z["lin_heads"]
+            layers.append({"type": "lightning", "mlp": None, "mixer": {"heads": H, "dim": z["lin_dim"], "vdim": z["lin_vdim"],
+                                                                       "decay": [1.0 - 2.0 ** (-1.0 - 8.0 * h / H) for h in range(H)]}})
+            continue
+        left = {"heads": z["att_heads"], "kv_heads": z["kv_heads"], "dim": z["att_dim"], "vdim": z["att_dim"], "scale": z["att_dim"] ** -0.5,
+                "mask": {"size": z["window"]}, "rot": {"dims": z["att_dim"], "base": 500000.0}}
+        right = {"heads": z["lin_heads"], "kv_heads": z["lin_kv_heads"], "dim": z["lin_dim"], "vdim": z["lin_vdim"], "conv": z["conv"]}
+        layers.append({"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.5, "right_scale": 0.5},
+                       "mlp": {"kind": "dense", "ff": z["ff"], "limit": 7.0}})
+    a, b, t = z["loop"]
+    return {"architecture": "Zetivik", "vocab": z["vocab"], "width": z["width"], "layers": layers, "norm": {"eps": 1e-5}, "logit_softcap": 50.0,
+            "loop": {"start": a, "stop": b, "times": t}}
+
+
+def zetivik_runs(z):
+    a, b, t = z["loop"]
+    return z["pattern"][:a] + z["pattern"][a:b] * t + z["pattern"][b:]
+
+
+def closest_nalizen(z):
+    """Nalizen layers at a Zetivik size: for every layer run of two mixers an attention layer and a recurrence layer with the
+    feed-forward, for every lightning run a recurrence layer; same width, heads, key and value sizes, mask size as the window."""
+    layers = []
+    rec = {"heads": z["lin_heads"], "dim": z["lin_dim"], "vdim": z["lin_vdim"]}
+    for ch in zetivik_runs(z):
+        if ch == "p":
+            layers.append({"type": "attention", "mlp": None, "mixer": {"heads": z["att_heads"], "kv_heads": z["kv_heads"], "dim": z["att_dim"], "vdim": z["att_dim"],
+                                                                       "scale": z["att_dim"] ** -0.5, "mask": {"size": z["window"]},
+                                                                       "rot": {"dims": z["att_dim"], "base": 500000.0}}})
+        layers.append({"type": "hgrn2", "mixer": rec, "mlp": {"kind": "dense", "ff": z["ff"]} if ch == "p" else None})
+    return {"architecture": "Nalizen", "vocab": z["vocab"], "width": z["width"], "layers": layers, "norm": {"eps": 1e-5}}
+
+
+def mint_zetivik(dsk, torch, cfg, quant, chunk, context, device=0):
+    import hashlib
+    hc, specs = dsk.zetivik_from_config(cfg, quant=quant, max_seq_len=context, chunk=chunk)
+    m = dsk.Model(hc, 0, 1, device, layers=specs)
+    dev = torch.device("cuda", device)
+    W, V = cfg["width"], cfg["vocab"]
+
+    def up(name, shape, kind="mat"):
+        torch.manual_seed(int(hashlib.md5(name.encode()).hexdigest()[:8], 16))
+        if kind == "mat":
+            t = torch.randn(*shape, device=dev) * (shape[-1] ** -0.5)
+        elif kind == "embed":
+            t = torch.randn(*shape, device=dev)
+        elif kind == "norm":
+            t = 1.0 + 0.1 * torch.randn(*shape, device=dev)
+        elif kind == "alog":
+            t = torch.log(torch.empty(*shape, device=dev).uniform_(0.5, 4.0))
+        elif kind == "dtb":
+            t = torch.empty(*shape, device=dev).uniform_(-5.0, -1.0)
+        else:
+            t = 0.1 * torch.randn(*shape, device=dev)
+        t = t.to(torch.bfloat16).contiguous()
+        m.upload_device(name, "BF16", shape, t.data_ptr(), t.numel() * 2)
+        torch.cuda.synchronize()
+
+    up("embed", (V, W), "embed"); up("final.norm", (W,), "small"); up("loop.step", (cfg["loop"]["times"], W), "small")
+    for i, lc in enumerate(cfg["layers"]):
+        p, mx = f"l{i}.", lc["mixer"]
+        up(p + "norm1", (W,), "small")
+        if lc["type"] == "parallel":
+            a, b = mx["left"], mx["right"]
+            l, r = p + "mix.left.", p + "mix.right."
+            H, G, D, P = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+            for t, n in (("q", H * D), ("k", G * D), ("v", G * P)):
+                up(l + t, (n, W)); up(l + t + ".b", (n,), "small")
+            up(l + "q.norm", (D,), "norm"); up(l + "k.norm", (D,), "norm"); up(l + "g", (H, W)); up(l + "o", (W, H * P))
+            H, G, D, P = b["heads"], b["kv_heads"], b["dim"], b["vdim"]
+            for t, n in (("q", G * D), ("k", G * D), ("v", H * P)):
+                up(r + t, (n, W)); up(r + t + ".conv", (n, b["conv"]))
+            up(r + "b", (H, W)); up(r + "a", (H, W)); up(r + "A_log", (H,), "alog"); up(r + "dt_bias", (H,), "dtb"); up(r + "norm", (P,), "norm")
+            up(r + "g", (H * P, W)); up(r + "o", (W, H * P))
+        else:
+            H, D, P = mx["heads"], mx["dim"], mx["vdim"]
+            for t, n in (("q", H * D), ("k", H * D), ("v", H * P), ("g", H * P)):
+                up(p + "mix." + t, (n, W))
+            up(p + "mix.norm", (H * P,), "norm"); up(p + "mix.o", (W, H * P))
+        if lc["mlp"]:
+            ff = lc["mlp"]["ff"]
+            up(p + "norm2", (W,), "small"); up(p + "mlp.gate", (ff, W)); up(p + "mlp.up", (ff, W)); up(p + "mlp.down", (W, ff))
+    m.finalize()
+    return m
+
+
+def zetivik_matrix_elements(cfg, z):
+    """Matrix elements one token multiplies with over all layer runs (projections, gates, feed-forward, head), and the attention's
+    own multiply-adds per token at the mean number of visible keys (half the mask size)."""
+    W, n, att = cfg["width"], cfg["width"] * cfg["vocab"], 0.0
+    for ch in zetivik_runs(z):
+        LH, LG, LD, LP = z["lin_heads"], z["lin_kv_heads"], z["lin_dim"], z["lin_vdim"]
+        if ch == "l":
+            n += (2 * LH * LD + 3 * LH * LP) * W
+            continue
+        H, G, D = z["att_heads"], z["kv_heads"], z["att_dim"]
+        n += (2 * H * D + 2 * G * D + H) * W + (2 * LG * LD + 3 * LH * LP + 2 * LH) * W + 3 * z["ff"] * W
+        att += 2 * H * D * (z["window"] / 2.0)
+    return n, att
+
+
+def run_zetivik(dsk, torch, name, hbm, tfl, prompt_len, gen, chunk, log):
+    """A Zetivik size and the closest layer-list model (Nalizen) at equal size."""
+    z = SIZES[name]
+    cfg = zetivik_config(z)
+    t0 = time.time()
+    m = mint_zetivik(dsk, torch, cfg, "bf16", chunk, prompt_len + gen + 8)
+    log(f"hybrid/{name}/bf16: minted {m.resident_bytes() / 1e9:.2f} GB in {time.time() - t0:.1f} s")
+    mat, att = zetivik_matrix_elements(cfg, z)
+    res = [measure_layer_list(m, f"Zetivik {name}", z["vocab"], 2.0 * mat, hbm, tfl, prompt_len, gen, chunk, log,
+                              {"layer_runs": len(zetivik_runs(z)), "width": z["width"], "attention_flops_per_token_fp32": 2.0 * att})]
+    m.close()
+    cfgn = closest_nalizen(z)
+    t0 = time.time()
+    m = mint_nalizen(dsk, torch, cfgn, "bf16", chunk, prompt_len + gen + 8)
+    log(f"hybrid/{name}/closest Nalizen/bf16: minted {m.resident_bytes() / 1e9:.2f} GB in {time.time() - t0:.1f} s")
+    matn, attn = nalizen_matrix_elements(cfgn, z)
+    res.append(measure_layer_list(m, f"Nalizen layers at {name}", z["vocab"], 2.0 * matn, hbm, tfl, prompt_len, gen, chunk, log,
+                                  {"layers": len(cfgn["layers"]), "width": z["width"], "attention_flops_per_token_fp32": 2.0 * attn}))
+    m.close()
+    return res
 
 
 def nalizen_config(z):
@@ -80,7 +214,7 @@ def mint_nalizen(dsk, torch, cfg, quant, chunk, context, device=0):
     m = dsk.Model(hc, 0, 1, device, layers=specs)
     dev = torch.device("cuda", device)
     W, V, L = cfg["width"], cfg["vocab"], len(cfg["layers"])
-    sd = cfg["token_side"]["dim"]
+    sd = (cfg.get("token_side") or {}).get("dim", 0)
 
     def up(name, shape, kind="mat"):
         torch.manual_seed(int(hashlib.md5(name.encode()).hexdigest()[:8], 16))
@@ -98,10 +232,12 @@ def mint_nalizen(dsk, torch, cfg, quant, chunk, context, device=0):
         m.upload_device(name, "BF16", shape, t.data_ptr(), t.numel() * 2)
         torch.cuda.synchronize()
 
-    up("embed", (V, W), "embed"); up("final.norm", (W,), "norm"); up("final.norm.b", (W,), "small"); up("side.embed", (V, sd * L), "embed")
+    up("embed", (V, W), "embed"); up("final.norm", (W,), "norm"); up("final.norm.b", (W,), "small")
+    if sd:
+        up("side.embed", (V, sd * L), "embed")
     for i, lc in enumerate(cfg["layers"]):
         p, mx, ff = f"l{i}.", lc["mixer"], lc["mlp"]
-        for nm in ("norm1", "norm2"):
+        for nm in ("norm1", "norm2") if ff else ("norm1",):
             up(p + nm, (W,), "norm"); up(p + nm + ".b", (W,), "small")
         up(p + "shift", (W,), "unit")
         H, D, Vd = mx["heads"], mx["dim"], mx["vdim"]
@@ -113,14 +249,17 @@ def mint_nalizen(dsk, torch, cfg, quant, chunk, context, device=0):
         else:
             up(p + "mix.q", (H * D, W)); up(p + "mix.f", (H * D, W)); up(p + "mix.f.b", (H * D,), "small"); up(p + "mix.lower", (H * D,), "unit")
             up(p + "mix.v", (H * Vd, W)); up(p + "mix.norm", (Vd,), "norm"); up(p + "mix.o", (W, H * Vd))
-        if ff["kind"] == "dense":
+        if not ff:
+            pass
+        elif ff["kind"] == "dense":
             up(p + "mlp.gate", (ff["ff"], W)); up(p + "mlp.up", (ff["ff"], W)); up(p + "mlp.down", (W, ff["ff"]))
         else:
             E, fe = ff["router"]["experts"], ff["expert"]["ff"]
             up(p + "mlp.router", (E, W)); up(p + "mlp.router.b", (E,), "small")
             for e in range(E):
                 up(f"{p}mlp.e{e}.up", (fe, W)); up(f"{p}mlp.e{e}.down", (W, fe))
-        up(p + "side.gate", (sd, W)); up(p + "side.proj", (W, sd)); up(p + "side.norm", (W,), "norm")
+        if sd:
+            up(p + "side.gate", (sd, W)); up(p + "side.proj", (W, sd)); up(p + "side.norm", (W,), "norm")
     m.finalize()
     return m
 
@@ -137,8 +276,9 @@ def nalizen_matrix_elements(cfg, z):
             att += H * (D + Vd) * (z["window"] / 2.0)
         else:
             n += (2 * H * D + H * Vd) * W + W * H * Vd
-        n += 3 * ff["ff"] * W if ff["kind"] == "dense" else 2 * ff["router"]["top"] * ff["expert"]["ff"] * W + ff["router"]["experts"] * W
-        n += 2 * cfg["token_side"]["dim"] * W
+        if ff:
+            n += 3 * ff["ff"] * W if ff["kind"] == "dense" else 2 * ff["router"]["top"] * ff["expert"]["ff"] * W + ff["router"]["experts"] * W
+        n += 2 * (cfg.get("token_side") or {}).get("dim", 0) * W
     return n, att
 
 
@@ -496,6 +636,9 @@ def run(dsk, torch, repo, bench_module, sizes=("small", "v2lite_like"), prompt_l
             continue
         if z.get("design") == "Nalizen":
             out["results"] += run_nalizen(dsk, torch, name, hbm, tfl, prompt_len, gen, chunk, log)
+            continue
+        if z.get("design") == "Zetivik":
+            out["results"] += run_zetivik(dsk, torch, name, hbm, tfl, prompt_len, gen, chunk, log)
             continue
         cfg = desarax_config(z)
         for quant in ("bf16",):
