@@ -207,6 +207,23 @@ __global__ void __launch_bounds__(256) group_rmsnorm(const float* __restrict__ i
   if (ring > 0) orow %= ring;
   OT* o = out + (size_t)orow * ld_out;
   const int gs = n / groups;
+  if (groups == 1 && gate && n <= 256 * 16) {   // one gated group: the row and its gate stay in registers, all loads in flight at once
+    float v[16], gt[16], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < 16; k++) {
+      const int i = threadIdx.x + 256 * k;
+      v[k] = i < n ? x[i] : 0.f;
+      gt[k] = i < n ? gate[(size_t)t * ld_gate + i] * w[i] : 0.f;
+      ss = fmaf(v[k], v[k], ss);
+    }
+    const float sc = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+#pragma unroll
+    for (int k = 0; k < 16; k++) {
+      const int i = threadIdx.x + 256 * k;
+      if (i < n) o[i] = from_f<OT>(mode == 0 ? v[k] * sc * gt[k] : to_f<OT>(o[i]) + alpha * (v[k] * sc * gt[k]));
+    }
+    return;
+  }
   for (int g = 0; g < groups; g++) {
     float ss = 0.f;
     for (int i = threadIdx.x; i < gs; i += blockDim.x) { const float v = x[g * gs + i]; ss += v * v; }
@@ -1418,6 +1435,7 @@ __global__ void add_row(float* __restrict__ x, int ld, const float* __restrict__
 // otherwise v_src rows are cached, blended with the rows of v_first [T][GV] when that is given: (1 - lam) v + lam v_first.
 // v_keep [T][GV], nullable, receives a copy of what is cached (the rows a later layer blends in).
 // k == nullptr: a layer that reads another layer's caches prepares its queries only and caches nothing.
+// With a norm per head, the heads of a token may be dealt over gridDim.y CTAs.
 // ---------------------------------------------------------------------------------------------------------------------
 __device__ __forceinline__ float rot_entry(const float* __restrict__ src, int c, int d, int rot_dims, int layout, float nrm, const float* __restrict__ w,
                                            float fpos, const float* __restrict__ freq, float mag) {
@@ -1451,7 +1469,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q,
   if (!k) GD = 0;
   if (head_norm) {   // a warp per head: rotated entries are stored, summed, and scaled by the lane that stored them
     const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nh = (HD + GD) / D;
-    for (int hh = w; hh < nh; hh += 8) {
+    for (int hh = w + 8 * (int)blockIdx.y; hh < nh; hh += 8 * (int)gridDim.y) {
       const bool isq = hh * D < HD;
       const int c0 = isq ? hh * D : hh * D - HD;
       const float* src = isq ? qr : kr;
@@ -1485,7 +1503,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q,
       else kcache[row * GD + c] = v;
     }
   }
-  if (!k) return;
+  if (!k || blockIdx.y > 0) return;
   const float* vr = v_src ? v_src + (size_t)t * ld_v : kr;
   for (int e = threadIdx.x; e < GV; e += blockDim.x) {
     float v = vr[e];
@@ -1832,10 +1850,25 @@ __global__ void __launch_bounds__(1024) argmax_row(const float* __restrict__ log
                                                    int* log, int step) {
   __shared__ unsigned long long best[32];
   unsigned long long b = 0ull;
-  for (int i = threadIdx.x; i < vocab; i += blockDim.x) {
-    const unsigned long long key = ((unsigned long long)orderable(logits[i]) << 32) | (unsigned long long)(0xFFFFFFFFu - (unsigned)i);
+  auto see = [&](float v, int i) {
+    const unsigned long long key = ((unsigned long long)orderable(v) << 32) | (unsigned long long)(0xFFFFFFFFu - (unsigned)i);
     if (key > b) b = key;
+  };
+  int done = 0;
+  if ((reinterpret_cast<uintptr_t>(logits) & 15) == 0) {   // whole rounds of four 16-byte loads per thread, all in flight together
+    const int round = 16 * (int)blockDim.x;
+    for (; done + round <= vocab; done += round) {
+      float4 v[4];
+#pragma unroll
+      for (int u = 0; u < 4; u++) v[u] = *reinterpret_cast<const float4*>(logits + done + 4 * (u * (int)blockDim.x + (int)threadIdx.x));
+#pragma unroll
+      for (int u = 0; u < 4; u++) {
+        const int i = done + 4 * (u * (int)blockDim.x + (int)threadIdx.x);
+        see(v[u].x, i); see(v[u].y, i + 1); see(v[u].z, i + 2); see(v[u].w, i + 3);
+      }
+    }
   }
+  for (int i = done + threadIdx.x; i < vocab; i += blockDim.x) see(logits[i], i);
   for (int o = 16; o; o >>= 1) { const unsigned long long v = __shfl_xor_sync(0xffffffffu, b, o); if (v > b) b = v; }
   if ((threadIdx.x & 31) == 0) best[threadIdx.x >> 5] = b;
   __syncthreads();

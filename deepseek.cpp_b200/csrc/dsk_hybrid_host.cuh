@@ -148,6 +148,9 @@ struct State {
   float *x = nullptr, *h = nullptr, *b0 = nullptr, *b1 = nullptr, *b2 = nullptr, *b3 = nullptr, *wgt = nullptr, *logits = nullptr;
   int *h_tok = nullptr, *h_want = nullptr;   // pinned staging of a chunk's token ids / wanted rows
   std::vector<void*> allocs;
+  // side-by-side mixers run on two streams, forked and joined by events
+  cudaStream_t side = nullptr;
+  cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
   cudaGraphExec_t step_graph = nullptr;      // captured greedy decode step (arg-max -> token -> one-token chunk)
   // DSK_HY_TIMELINE=1: CUDA events between the groups of launches of every step, summed per label and printed to stderr
   bool timeline = false;
@@ -321,11 +324,11 @@ static void set_kernel_attrs() {
   cudaFuncSetAttribute(hgrn2_scan<1, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(hgrn2_scan<2, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   cudaFuncSetAttribute(gemm_mma<HEPI_SILU_SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMmaSmem);
   cudaFuncSetAttribute(gemm_mma<HEPI_SOFTCAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMmaSmem);
-  cudaFuncSetAttribute(lin_scan<true, 8, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 8, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
-  cudaFuncSetAttribute(lin_scan<true, 16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
-  cudaFuncSetAttribute(lin_scan<true, 32, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 32, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
-  cudaFuncSetAttribute(lin_scan<true, 16, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 16, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
-  cudaFuncSetAttribute(lin_scan<true, 32, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); cudaFuncSetAttribute(lin_scan<false, 32, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
+#define DSK_LSCAN_ATTR(A, B, C) \
+  cudaFuncSetAttribute(lin_scan<true, A, B, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, big); \
+  cudaFuncSetAttribute(lin_scan<false, A, B, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)
+  DSK_LSCAN_ATTR(8, 1, 2); DSK_LSCAN_ATTR(16, 1, 2); DSK_LSCAN_ATTR(32, 1, 2); DSK_LSCAN_ATTR(8, 1, 4); DSK_LSCAN_ATTR(16, 1, 4); DSK_LSCAN_ATTR(32, 1, 4); DSK_LSCAN_ATTR(32, 2, 4);
+#undef DSK_LSCAN_ATTR
   cudaFuncSetAttribute(gqa_attn, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   cudaFuncSetAttribute(mix_heads, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   done = true;
@@ -1140,6 +1143,9 @@ static dsk_state* state_create(dsk_model* m) {
   rc |= salloc(S, (void**)&S->x, Tc * c.dim * 4) | salloc(S, (void**)&S->h, Tc * c.dim * 4);
   if (c.loop_embed && c.loop_times > 1) rc |= salloc(S, (void**)&S->emb, Tc * c.dim * 4);
   if (mxLH) rc |= salloc(S, (void**)&S->lrec, (Tc + kLinBlk - 1) / kLinBlk * mxLH * kRecFloats * 4) | salloc(S, (void**)&S->lout, Tc * mxLV * 4);
+  for (const HLayer& L : M->L)
+    if (L.sp.mixer2 && !S->side && (cudaStreamCreateWithFlags(&S->side, cudaStreamNonBlocking) != cudaSuccess || cudaEventCreateWithFlags(&S->ev_fork, cudaEventDisableTiming) != cudaSuccess ||
+                                    cudaEventCreateWithFlags(&S->ev_join, cudaEventDisableTiming) != cudaSuccess)) { fail(-2, "stream creation failed"); return nullptr; }
   if (mxLQ) rc |= salloc(S, (void**)&S->lq, Tc * mxLQ * 4) | salloc(S, (void**)&S->lk, Tc * mxLQ * 4) | salloc(S, (void**)&S->lv, Tc * mxLV * 4);
   if (c.block == DSK_BLOCK_SANDWICH || c.block == DSK_BLOCK_POST) rc |= salloc(S, (void**)&S->y, Tc * c.dim * 4);
   if (c.token_shift) rc |= salloc(S, (void**)&S->hs, Tc * c.dim * 4);
@@ -1161,6 +1167,7 @@ static void state_free(dsk_state* s) {
   State* S = s->hy;
   if (!S) return;
   if (S->step_graph) cudaGraphExecDestroy(S->step_graph);
+  if (S->side) { cudaStreamSynchronize(S->side); cudaStreamDestroy(S->side); cudaEventDestroy(S->ev_fork); cudaEventDestroy(S->ev_join); }
   for (cudaEvent_t e : S->tl_events) cudaEventDestroy(e);
   for (void* p : S->allocs) cudaFree(p);
   cudaFreeHost(S->h_tok); cudaFreeHost(S->h_want);
@@ -1319,15 +1326,19 @@ static void launch_hgrn2(const dsk_layer_spec& sp, const float* proj, int ld, fl
 // the walk over the blocks of a step (lin_scan): lanes per channel group by the key size, warps per CTA by how many CTAs there are
 static void launch_lin_scan(bool delta, const float* q, const float* k, int ldq, int hs, int rep, const float* v, int ldv, const float* rec, float* state,
                             float* out, int ldo, int T, int H, int N, int P, cudaStream_t st) {
-  const int TPC = N <= 32 ? 8 : N <= 64 ? 16 : 32, RQ = N <= 128 ? 1 : 2, CW = 4 * (32 / TPC);
+  const int TPC = N <= 32 ? 8 : N <= 64 ? 16 : 32, RQ = N <= 128 ? 1 : 2;
+  int CPT = N > 128 ? 4 : 2;          // value channels per lane
+  if (const char* e = getenv("DSK_LIN_CPT")) CPT = atoi(e) == 4 || N > 128 ? 4 : 2;   // A/B switch
+  const int CW = CPT * (32 / TPC);
   int warps = std::max(1, std::min(8, (P + CW - 1) / CW));
-  while (warps > 1 && H * ((P + warps * CW - 1) / (warps * CW)) < 148) warps = (warps + 1) / 2;
+  while (warps > 2 && H * ((P + warps * CW - 1) / (warps * CW)) < 148) warps = (warps + 1) / 2;
   if (const char* e = getenv("DSK_LIN_WARPS")) warps = std::max(1, std::min(8, atoi(e)));   // A/B switch
   const int PB = warps * CW;
   const dim3 grid((unsigned)H, (unsigned)((P + PB - 1) / PB));
   const size_t smem = lin_scan_smem(4 * TPC * RQ, PB, warps, CW);
-#define DSK_LSCAN(D, A, B) lin_scan<D, A, B><<<grid, 32 * warps, smem, st>>>(q, k, ldq, hs, rep, v, ldv, rec, state, out, ldo, T, H, N, P, PB)
-#define DSK_LSCANS(D) do { if (N <= 32) DSK_LSCAN(D, 8, 1); else if (N <= 64) DSK_LSCAN(D, 16, 1); else if (N <= 128) DSK_LSCAN(D, 32, 1); else DSK_LSCAN(D, 32, 2); } while (0)
+#define DSK_LSCAN(D, A, B, C) lin_scan<D, A, B, C><<<grid, 32 * (warps + kLinStage), smem, st>>>(q, k, ldq, hs, rep, v, ldv, rec, state, out, ldo, T, H, N, P, PB)
+#define DSK_LSCANS(D) do { if (N > 128) DSK_LSCAN(D, 32, 2, 4); else if (CPT == 2) { if (N <= 32) DSK_LSCAN(D, 8, 1, 2); else if (N <= 64) DSK_LSCAN(D, 16, 1, 2); else DSK_LSCAN(D, 32, 1, 2); } \
+  else { if (N <= 32) DSK_LSCAN(D, 8, 1, 4); else if (N <= 64) DSK_LSCAN(D, 16, 1, 4); else DSK_LSCAN(D, 32, 1, 4); } } while (0)
   if (delta) DSK_LSCANS(true); else DSK_LSCANS(false);
 #undef DSK_LSCANS
 #undef DSK_LSCAN
@@ -1540,10 +1551,12 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       const int gate_head = sp.att_out_gate == DSK_GATE_HEAD;
       const int ldo = H * V + (sp.mixer2 ? (int)gdn_v(sp) : 0);   // a second mixer's heads stand behind this one's
       const float lscale = sp.mixer2 ? sp.mix_scale : 1.f;
+      // a decoded token's heads over several CTAs, where each head has a norm of its own
+      const dim3 qk_grid((unsigned)T, (unsigned)(sp.att_qk_norm != DSK_QKNORM_WHOLE && T <= kAttnSplitTokens ? (H + (reads ? 0 : G) + 7) / 8 : 1));
       if (reads) {
         linear(S, bf, HEPI_STORE, gp(hin, W, L.qkv.p, W, S->b0, ldp, T, ldp, W), 1, st);
         MK("att.qk");
-        qk_norm_rope<<<T, 256, 0, st>>>(S->b0, S->b2, HD, nullptr, nullptr, GD, GV, ldp, 0, 0, L.q_norm, nullptr, c.norm_eps, D, sp.rot_dims, L.rot_freq,
+        qk_norm_rope<<<qk_grid, 256, 0, st>>>(S->b0, S->b2, HD, nullptr, nullptr, GD, GV, ldp, 0, 0, L.q_norm, nullptr, c.norm_eps, D, sp.rot_dims, L.rot_freq,
                                         L.rot_mag, S->d_ctl, nullptr, nullptr, ring, keep, nullptr, 0.f, nullptr, sp.rot_layout, sp.att_qk_norm);
       } else if (sp.att_value_proj) {   // one product for the stacked q / k / v rows; the first value-mixing layer keeps its values for the later ones
         const int ld = ldp;
@@ -1551,15 +1564,21 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
         P.bias = sp.att_bias ? L.qkv_b : nullptr;
         linear(S, bf, HEPI_STORE, P, 1, st);
         MK("att.qk");
+        if (sp.mixer2 == DSK_MIX_GDN && !tl) {   // the second mixer on its own stream: it shares nothing with the first but the projections
+          CKL(cudaEventRecord(S->ev_fork, st));
+          CKL(cudaStreamWaitEvent(S->side, S->ev_fork, 0));
+          gdn_forward(S, L, ls, ldp, lay, S->b3 + H * V, ldo, sp.mix2_scale, c.norm_eps, T, S->side);
+          CKL(cudaEventRecord(S->ev_join, S->side));
+        }
         const bool blend = sp.att_vmix && li != M->vmix_first;
-        qk_norm_rope<<<T, 256, 0, st>>>(S->b0, S->b2, HD, S->b0 + HD, S->b0 + HD + GD, GD, GV, ld, ld, ld, L.q_norm, L.k_norm, c.norm_eps, D, sp.rot_dims,
+        qk_norm_rope<<<qk_grid, 256, 0, st>>>(S->b0, S->b2, HD, S->b0 + HD, S->b0 + HD + GD, GD, GV, ld, ld, ld, L.q_norm, L.k_norm, c.norm_eps, D, sp.rot_dims,
                                         L.rot_freq, L.rot_mag, S->d_ctl, kc, vc, ring, keep, blend ? S->vfirst : nullptr, L.vmix,
                                         sp.att_vmix && li == M->vmix_first ? S->vfirst : nullptr, sp.rot_layout, sp.att_qk_norm);
       } else {
         linear(S, bf, HEPI_STORE, gp(hin, W, L.q.p, W, S->b0, HD, T, HD, W), 1, st);
         linear(S, bf, HEPI_STORE, gp(hin, W, L.kproj.p, W, S->b1, GD, T, GD, W), 1, st);
         MK("att.qk");
-        qk_norm_rope<<<T, 256, 0, st>>>(S->b0, S->b2, HD, S->b1, nullptr, GD, GV, HD, GD, GD, L.q_norm, L.k_norm, c.norm_eps, D, sp.rot_dims, L.rot_freq,
+        qk_norm_rope<<<qk_grid, 256, 0, st>>>(S->b0, S->b2, HD, S->b1, nullptr, GD, GV, HD, GD, GD, L.q_norm, L.k_norm, c.norm_eps, D, sp.rot_dims, L.rot_freq,
                                         L.rot_mag, S->d_ctl, kc, vc, ring, keep, nullptr, 0.f, nullptr, sp.rot_layout, sp.att_qk_norm);
       }
       S->launches++;
@@ -1606,7 +1625,8 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
         S->launches += NS > 1 ? 2 : 1;
         MK("att.decode");
       }
-      if (sp.mixer2 == DSK_MIX_GDN) {
+      if (sp.mixer2 == DSK_MIX_GDN && !tl) CKL(cudaStreamWaitEvent(st, S->ev_join, 0));
+      else if (sp.mixer2 == DSK_MIX_GDN) {   // timeline: one after the other
         gdn_forward(S, L, ls, ldp, lay, S->b3 + H * V, ldo, sp.mix2_scale, c.norm_eps, T, st);
         MK("gdn");
       }
@@ -1917,7 +1937,8 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
     if (trace) CKL(cudaMemcpyAsync(trace + ri * (size_t)T * W, S->x, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, st));
   }
   if (n_want > 0) {   // final norm of every row, LM head on the first group of wanted rows (enqueue_head does the others)
-    if (!h_ready) norm_rows(c, S, S->x, M->final_norm, M->final_norm_b, S->h, T, 0, 0.f, st);
+    if (pre) { rms_open<<<T, 256, 0, st>>>(S->x, nullptr, nullptr, M->final_norm, S->h, W, c.norm_eps); S->launches++; }
+    else if (!h_ready) norm_rows(c, S, S->x, M->final_norm, M->final_norm_b, S->h, T, 0, 0.f, st);
     enqueue_head(m, s, 0, std::min(n_want, S->head_rows), st);
     MK("head");
   }

@@ -206,41 +206,45 @@ __device__ __forceinline__ int reduce_index(int s) {
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
-// The walk over the blocks of a step.  CTA = (head, slice of value channels).  A warp owns (32 / TPC) x 4 value channels with the
-// whole key dimension: lane (grp, s) holds the rows n = 4 (s + TPC r) + i, r < RQ, of the four channels grp * 4 .. + 3 in
+// The walk over the blocks of a step.  CTA = (head, slice of value channels).  A warp owns (32 / TPC) x CPT value channels with the
+// whole key dimension: lane (grp, s) holds the rows n = 4 (s + TPC r) + i, r < RQ, of the CPT channels from grp * CPT on in
 // registers.  S0^T k and S0^T q of a block are 32 dot products per channel, reduced across the TPC lanes by reduce-scatter;
-// everything behind them stays inside the warp (its own shared-memory strip).  The blocks' q, k, v and records arrive through
-// two buffers: 16-byte asynchronous copies where the rows allow it, plain loads otherwise.
+// everything behind them stays inside the warp (its own shared-memory strip).  The CTA's last kLinStage warps do not compute:
+// they bring the blocks' q, k, v and records through three buffers, two blocks ahead (16-byte asynchronous copies where the rows
+// allow it, plain loads otherwise), so a block costs the computing warps one barrier.
 // q, k: head stride hs (rows of N entries), v: head stride P; head h reads q / k head h / rep.
 // ---------------------------------------------------------------------------------------------------------------------
-template <bool DELTA, int TPC, int RQ>
-__global__ void __launch_bounds__(256) lin_scan(const float* __restrict__ q, const float* __restrict__ k, int ldq, int hs, int rep,
+constexpr int kLinStage = 2;           // staging warps of a CTA
+template <bool DELTA, int TPC, int RQ, int CPT>
+__global__ void __launch_bounds__(320) lin_scan(const float* __restrict__ q, const float* __restrict__ k, int ldq, int hs, int rep,
                                                 const float* __restrict__ v, int ldv, const float* __restrict__ rec, float* __restrict__ state,
                                                 float* __restrict__ out, int ldo, int T, int H, int N, int P, int PB) {
   extern __shared__ __align__(16) float sm[];
-  constexpr int C = kLinBlk, PITCH = 4 * TPC * RQ, CW = 4 * (32 / TPC);
+  constexpr int C = kLinBlk, PITCH = 4 * TPC * RQ, CW = CPT * (32 / TPC), VB = 32 / CPT;
   const int per = 2 * C * PITCH + C * PB + kRecFloats;     // one buffer: k [C][PITCH], q [C][PITCH], v [C][PB], record
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5, s = lane & (TPC - 1), grp = lane / TPC;
   const int h = blockIdx.x, p0 = blockIdx.y * PB, hk = h / rep, cw = w * CW;   // cw: the warp's first channel inside the slice
-  float* Rw = sm + 2 * per + w * (4 * C * CW);   // [S0^T k | S0^T q][C][CW]
+  float* Rw = sm + 3 * per + w * (4 * C * CW);   // [S0^T k | S0^T q][C][CW]
   float* Uw = Rw + 2 * C * CW;                   // [C][CW]  w, then R(end, .) u
   float* Xw = Uw + C * CW;                       // [C][CW]  u
-  float S[RQ][4][4];                             // [row group][row][channel]
-  const int pc = p0 + cw + grp * 4;              // the lane's first channel of the head
+  float S[RQ][4][CPT];                           // [row group][row][channel]
+  const int pc = p0 + cw + grp * CPT;              // the lane's first channel of the head
 #pragma unroll
   for (int r = 0; r < RQ; r++)
 #pragma unroll
     for (int i = 0; i < 4; i++) {
       const int n = 4 * (s + TPC * r) + i;
 #pragma unroll
-      for (int c = 0; c < 4; c++) S[r][i][c] = (n < N && pc + c < P && cw + grp * 4 + c < PB) ? state[((size_t)h * N + n) * P + pc + c] : 0.f;
+      for (int c = 0; c < CPT; c++) S[r][i][c] = (n < N && pc + c < P && cw + grp * CPT + c < PB) ? state[((size_t)h * N + n) * P + pc + c] : 0.f;
     }
   const bool vec = (N & 3) == 0 && (ldq & 3) == 0 && (hs & 3) == 0 && ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k)) & 15) == 0;
   const bool vecv = (P & 3) == 0 && (PB & 3) == 0 && (ldv & 3) == 0 && (reinterpret_cast<uintptr_t>(v) & 15) == 0 && p0 + PB <= P;
-  const int np = (N + 3) & ~3;
-  for (int e = tid; e < 2 * per; e += blockDim.x) sm[e] = 0.f;   // padding columns stay zero
+  const int nc = (blockDim.x >> 5) - kLinStage;   // computing warps
+  for (int e = tid; e < 3 * per; e += blockDim.x) sm[e] = 0.f;   // padding columns stay zero
   __syncthreads();
-  auto stage = [&](int buf, int t0) {
+  const int sw = w - nc, stid = tid - 32 * nc;
+  constexpr int ST = 32 * kLinStage;
+  auto stage = [&](int buf, int t0) {   // by the staging warps
     float* bk = sm + buf * per;
     float* bq = bk + C * PITCH;
     float* bv = bq + C * PITCH;
@@ -248,75 +252,84 @@ __global__ void __launch_bounds__(256) lin_scan(const float* __restrict__ q, con
     const int nt = min(C, T - t0);
     const size_t base = (size_t)t0 * ldq + (size_t)hk * hs;
     if (vec) {
-      const int n4 = np >> 2;
-      for (int e = tid; e < C * n4; e += blockDim.x) {
-        const int t = e / n4, c = (e - t * n4) * 4;
-        const size_t src = base + (size_t)(t < nt ? t : 0) * ldq + c;
-        const int bytes = t < nt ? 16 : 0;                        // rows past the end are zero-filled
-        cp_async_16(bk + t * PITCH + c, k + src, bytes);
-        cp_async_16(bq + t * PITCH + c, q + src, bytes);
+      for (int t = sw; t < C; t += kLinStage) {                   // a warp per row; rows past the end are zero-filled
+        const size_t src = base + (size_t)(t < nt ? t : 0) * ldq;
+        const int bytes = t < nt ? 16 : 0;
+        for (int c = 4 * lane; c < N; c += 128) {
+          cp_async_16(bk + t * PITCH + c, k + src + c, bytes);
+          cp_async_16(bq + t * PITCH + c, q + src + c, bytes);
+        }
       }
     } else {
-      for (int e = tid; e < C * N; e += blockDim.x) {
-        const int t = e / N, c = e - t * N;
-        bk[t * PITCH + c] = t < nt ? k[base + (size_t)t * ldq + c] : 0.f;
-        bq[t * PITCH + c] = t < nt ? q[base + (size_t)t * ldq + c] : 0.f;
-      }
+      for (int t = sw; t < C; t += kLinStage)
+        for (int c = lane; c < N; c += 32) {
+          bk[t * PITCH + c] = t < nt ? k[base + (size_t)t * ldq + c] : 0.f;
+          bq[t * PITCH + c] = t < nt ? q[base + (size_t)t * ldq + c] : 0.f;
+        }
     }
     const float* vs = v + (size_t)t0 * ldv + (size_t)h * P + p0;
     if (vecv) {
       const int b4 = PB >> 2;
-      for (int e = tid; e < C * b4; e += blockDim.x) {
+      for (int e = stid; e < C * b4; e += ST) {
         const int t = e / b4, c = (e - t * b4) * 4;
         cp_async_16(bv + t * PB + c, vs + (size_t)(t < nt ? t : 0) * ldv + c, t < nt ? 16 : 0);
       }
     } else {
-      for (int e = tid; e < C * PB; e += blockDim.x) {
+      for (int e = stid; e < C * PB; e += ST) {
         const int t = e / PB, c = e - t * PB;
         bv[e] = t < nt && p0 + c < P ? vs[(size_t)t * ldv + c] : 0.f;
       }
     }
     const float* rs = rec + ((size_t)(t0 / C) * H + h) * kRecFloats;
-    for (int e = (DELTA ? 0 : kRecM / 4) + tid; e < kRecFloats / 4; e += blockDim.x) cp_async_16(br + 4 * e, rs + 4 * e, 16);
+    for (int e = (DELTA ? 0 : kRecM / 4) + stid; e < kRecFloats / 4; e += ST) cp_async_16(br + 4 * e, rs + 4 * e, 16);
     cp_async_commit();
   };
   const int nb = (T + C - 1) / C;
-  stage(0, 0);
+  if (sw >= 0) {
+    stage(0, 0);
+    if (nb > 1) { stage(1, C); cp_async_wait<1>(); } else cp_async_wait<0>();
+    __syncthreads();                   // block 0 has landed
+    for (int b = 0; b < nb; b++) {     // while the others work on block b: start block b + 2, see block b + 1 land
+      if (b + 2 < nb) { stage((b + 2) % 3, (b + 2) * C); cp_async_wait<1>(); }
+      else cp_async_wait<0>();
+      __syncthreads();
+    }
+    return;
+  }
+  __syncthreads();
   for (int b = 0; b < nb; b++) {
-    if (b + 1 < nb) { stage((b + 1) & 1, (b + 1) * C); cp_async_wait<1>(); }
-    else cp_async_wait<0>();
-    __syncthreads();
-    const float* bk = sm + (b & 1) * per;
+    const float* bk = sm + (b % 3) * per;
     const float* bq = bk + C * PITCH;
     const float* bv = bq + C * PITCH;
     const float* br = bv + C * PB;
     const int t0 = b * C, nt = min(C, T - t0);
-    // S0^T k_j (delta rule) and S0^T q_j: eight tokens x four channels per reduction
+    // S0^T k_j (delta rule) and S0^T q_j: VB tokens x CPT channels per reduction
 #pragma unroll
     for (int which = DELTA ? 0 : 1; which < 2; which++) {
       const float* src = which ? bq : bk;
 #pragma unroll
-      for (int half = 0; half < C; half += 8) {
+      for (int half = 0; half < C; half += VB) {
         float a[32];
 #pragma unroll
         for (int e = 0; e < 32; e++) a[e] = 0.f;
 #pragma unroll
-        for (int t = 0; t < 8; t++)
+        for (int t = 0; t < VB; t++)
 #pragma unroll
           for (int r = 0; r < RQ; r++) {
             const float4 x = *reinterpret_cast<const float4*>(src + (half + t) * PITCH + 4 * (s + TPC * r));
 #pragma unroll
-            for (int c = 0; c < 4; c++) {
-              a[t * 4 + c] = fmaf(x.x, S[r][0][c], a[t * 4 + c]); a[t * 4 + c] = fmaf(x.y, S[r][1][c], a[t * 4 + c]);
-              a[t * 4 + c] = fmaf(x.z, S[r][2][c], a[t * 4 + c]); a[t * 4 + c] = fmaf(x.w, S[r][3][c], a[t * 4 + c]);
+            for (int c = 0; c < CPT; c++) {
+              float& acc = a[t * CPT + c];
+              acc = fmaf(x.x, S[r][0][c], acc); acc = fmaf(x.y, S[r][1][c], acc);
+              acc = fmaf(x.z, S[r][2][c], acc); acc = fmaf(x.w, S[r][3][c], acc);
             }
           }
         reduce_scatter<TPC>(a, s);
         const int idx = reduce_index<TPC>(s);
 #pragma unroll
         for (int e = 0; e < 32 / TPC; e++) {
-          const int t = (idx + e) >> 2, c = (idx + e) & 3;
-          Rw[which * C * CW + (half + t) * CW + grp * 4 + c] = a[e];
+          const int t = (idx + e) / CPT, c = (idx + e) % CPT;
+          Rw[which * C * CW + (half + t) * CW + grp * CPT + c] = a[e];
         }
       }
     }
@@ -367,22 +380,23 @@ __global__ void __launch_bounds__(256) lin_scan(const float* __restrict__ q, con
 #pragma unroll
       for (int i = 0; i < 4; i++)
 #pragma unroll
-        for (int c = 0; c < 4; c++) S[r][i][c] *= ge;
+        for (int c = 0; c < CPT; c++) S[r][i][c] *= ge;
 #pragma unroll
     for (int j = 0; j < C; j++) {
-      const float4 uu = *reinterpret_cast<const float4*>(Uw + j * CW + grp * 4);
+      float uu[CPT];
+#pragma unroll
+      for (int c = 0; c < CPT; c++) uu[c] = Uw[j * CW + grp * CPT + c];
 #pragma unroll
       for (int r = 0; r < RQ; r++) {
         const float4 x = *reinterpret_cast<const float4*>(bk + j * PITCH + 4 * (s + TPC * r));
         const float xs[4] = {x.x, x.y, x.z, x.w};
 #pragma unroll
-        for (int i = 0; i < 4; i++) {
-          S[r][i][0] = fmaf(xs[i], uu.x, S[r][i][0]); S[r][i][1] = fmaf(xs[i], uu.y, S[r][i][1]);
-          S[r][i][2] = fmaf(xs[i], uu.z, S[r][i][2]); S[r][i][3] = fmaf(xs[i], uu.w, S[r][i][3]);
-        }
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+          for (int c = 0; c < CPT; c++) S[r][i][c] = fmaf(xs[i], uu[c], S[r][i][c]);
       }
     }
-    __syncthreads();   // the buffer is free for the block after next
+    __syncthreads();   // block b's buffer is free, block b + 1 is there
   }
 #pragma unroll
   for (int r = 0; r < RQ; r++)
@@ -390,10 +404,10 @@ __global__ void __launch_bounds__(256) lin_scan(const float* __restrict__ q, con
     for (int i = 0; i < 4; i++) {
       const int n = 4 * (s + TPC * r) + i;
 #pragma unroll
-      for (int c = 0; c < 4; c++) if (n < N && pc + c < P && cw + grp * 4 + c < PB) state[((size_t)h * N + n) * P + pc + c] = S[r][i][c];
+      for (int c = 0; c < CPT; c++) if (n < N && pc + c < P && cw + grp * CPT + c < PB) state[((size_t)h * N + n) * P + pc + c] = S[r][i][c];
     }
 }
-inline size_t lin_scan_smem(int pitch, int PB, int warps, int cw) { return ((size_t)2 * (2 * kLinBlk * pitch + kLinBlk * PB + kRecFloats) + (size_t)warps * 4 * kLinBlk * cw) * 4; }
+inline size_t lin_scan_smem(int pitch, int PB, int warps, int cw) { return ((size_t)3 * (2 * kLinBlk * pitch + kLinBlk * PB + kRecFloats) + (size_t)warps * 4 * kLinBlk * cw) * 4; }
 
 // ---------------------------------------------------------------------------------------------------------------------
 // Steps of up to kLinDecodeTokens tokens, one CTA per value head, the head's state in registers: thread (pl, ng) owns the value
