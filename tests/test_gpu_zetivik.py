@@ -528,6 +528,24 @@ def test_greedy_generation(full, zo):
         assert host == want
 
 
+@pytest.mark.parametrize("vocab", [16384, 40001])
+def test_arg_max_over_a_large_vocabulary(mk, zo, vocab):
+    """The device's arg-max against numpy's on the same logits; of two equal largest logits the lower index wins."""
+    cfg = zo.model_config([zo.light(heads=1, dim=4, vdim=4)], width=12, vocab=vocab, cap=0)
+    m, W = mk(cfg, seed=2)
+    for t in (3, 77, vocab - 1):
+        lg = m.forward_chunk([5, t], 0, [1])[0]
+        assert m.sample(temperature=0.0) == int(np.argmax(lg))
+    best = int(np.argmax(m.forward_chunk([5, 77], 0, [1])[0]))
+    twin = vocab - 2 if best < vocab // 2 else 9
+
+    def edit(W):
+        W["embed"][twin] = W["embed"][best]
+    m2, _ = mk(cfg, seed=2, edit=edit)
+    lg = m2.forward_chunk([5, 77], 0, [1])[0]
+    assert lg[best] == lg[twin] and m2.sample(temperature=0.0) == min(best, twin)
+
+
 def test_device_loop_continues_and_hands_over(full, zo):
     """The captured step carries positions, rings and states on the device: a second run of the loop and a host step continue it."""
     cfg, m, W, toks, exp, _ = full
