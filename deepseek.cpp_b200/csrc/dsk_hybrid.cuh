@@ -23,13 +23,15 @@
 //   token_shift       h_t + (h_(t-1) - h_t) * mu in front of a mixer, the last row carried from step to step
 //   rms_add_shift_small   decode-sized steps: an RMS-normed addition into the stream and the next layer's token shift in one launch
 //   rms_open          opening of a pre-norm sublayer: additions of a loop pass and the RMS norm in one launch
+//   rms_add_norm      sandwich blocks of RMS norms: the weighted sum of the experts' outputs, the closing norm, the addition into the
+//                     stream and the next norm in one launch
 //   head_rmsnorm      RMS norm per head with one weight vector for all heads, optionally gated
-//   (the gated delta rule and lightning attention are in dsk_linattn.cuh)
+//   (the gated delta rule, lightning attention and the mLSTM matrix memory are in dsk_linattn.cuh)
 //   hgrn2_scan        the gated linear recurrence S <- diag(f) S + (1 - f) v^T, o = S^T silu(q), f = l + (1 - l) sigmoid(.)
 //   moe_route         sigmoid scores, selection by score + correction, weights = normalised scores x scale; or the largest
-//                     logits with a softmax over the chosen ones
+//                     logits with a softmax over the chosen ones; or a softmax over all experts, limited to the best groups
 //   moe_plan          groups the (token, slot) pairs of a chunk by expert into row tiles for gemm_tiled
-//   moe_combine       residual += alpha * sum_k w_k y_k (or stored, when a norm follows)
+//   moe_combine       residual += alpha * sum_k w_k y_k (or stored, when a norm follows), a shared expert's row included
 //
 // Numerics: the residual stream, norms, router, softmax, recurrent state, decays, step sizes and gates are fp32 in every mode;
 // DSK_BF16 models keep their matrices in bfloat16 and accumulate in fp32: decode-sized products multiply them with the fp32
@@ -101,18 +103,18 @@ __global__ void advance_ctl(int* ctl, int by) { ctl[0] += by; }
 // x[t] = scale * table[tok[t]] (+ bigram[row]).  The second table is indexed by the pair (previous token, token): row
 // (prev * mul_prev + tok * mul_cur) mod buckets, and row `buckets` for the first token of a sequence (position ctl[0] + t == 0).
 // The token before the step's first one is carried[0]; carry_token stores the step's last token there afterwards.  x_keep
-// (nullable) receives a copy (a layer loop may add the embedding again).
+// (nullable, row pitch ld_keep) receives a copy (a layer loop may read the embedding again).
 template <typename WT>
 __global__ void embed_rows(const int* __restrict__ tok, const WT* __restrict__ table, int width, float* __restrict__ x, float scale,
                            const WT* __restrict__ bigram, int buckets, int mul_prev, int mul_cur, const int* __restrict__ ctl,
-                           const int* __restrict__ carried, float* __restrict__ x_keep = nullptr) {
+                           const int* __restrict__ carried, float* __restrict__ x_keep = nullptr, int ld_keep = 0) {
   const int t = blockIdx.x;
   const WT* row = table + (size_t)tok[t] * width;
   if (!bigram) {
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
       const float v = scale * to_f<WT>(row[c]);
       x[(size_t)t * width + c] = v;
-      if (x_keep) x_keep[(size_t)t * width + c] = v;
+      if (x_keep) x_keep[(size_t)t * ld_keep + c] = v;
     }
     return;
   }
@@ -125,7 +127,7 @@ __global__ void embed_rows(const int* __restrict__ tok, const WT* __restrict__ t
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     const float v = fmaf(scale, to_f<WT>(row[c]), to_f<WT>(brow[c]));
     x[(size_t)t * width + c] = v;
-    if (x_keep) x_keep[(size_t)t * width + c] = v;
+    if (x_keep) x_keep[(size_t)t * ld_keep + c] = v;
   }
 }
 // the ring rows of the last taps - 1 positions of a step of T >= taps - 1 tokens (see canon_conv)
@@ -245,8 +247,8 @@ __global__ void __launch_bounds__(256) group_rmsnorm(const float* __restrict__ i
 // matrix products
 // ---------------------------------------------------------------------------------------------------------------------
 enum { HEPI_STORE = 0, HEPI_ADD = 1, HEPI_GLU = 2, HEPI_GELU_MUL = 3, HEPI_XIELU = 4, HEPI_GEGLU = 5, HEPI_SIGMUL = 6, HEPI_RELU2 = 7, HEPI_LINGATE = 8,
-       HEPI_SILU_SIG = 9, HEPI_SOFTCAP = 10 };
-__host__ __device__ constexpr bool epi_dual(int epi) { return epi == HEPI_GLU || epi == HEPI_GEGLU; }   // two weight matrices per output
+       HEPI_SILU_SIG = 9, HEPI_SOFTCAP = 10, HEPI_SWIGLU = 11 };
+__host__ __device__ constexpr bool epi_dual(int epi) { return epi == HEPI_GLU || epi == HEPI_GEGLU || epi == HEPI_SWIGLU; }   // two weight matrices per output
 
 struct GemmP {
   const float* A;          // activations, row pitch lda
@@ -266,7 +268,7 @@ struct GemmP {
   const int* n_tiles;
   float alpha;             // STORE: C = alpha acc; ADD: C += alpha acc
   float lim;               // GLU: g = min(gate, lim), u = clamp(up, -lim, lim), C = g sigmoid(1.702 g) (u + 1)
-                           // GEGLU: C = gelu_tanh(gate) * up;  SIGMUL: C *= sigmoid(acc) (a gate on what C already holds);
+                           // GEGLU: C = gelu_tanh(gate) * up;  SWIGLU: C = silu(gate) * up;  SIGMUL: C *= sigmoid(acc) (a gate on what C already holds);
                            // RELU2: C = max(acc, 0)^2;  LINGATE (the stacked [q | f | v] projection of a gated linear recurrence, aux_off
                            // columns of q and of f): q columns silu(acc), f columns l + (1 - l) sigmoid(acc) with l = aux[n - aux_off] (fp32), v columns acc;
                            // SILU_SIG: columns below aux_off silu(acc), the others sigmoid(acc);  SOFTCAP: C = lim tanh(alpha acc / lim)
@@ -275,6 +277,12 @@ struct GemmP {
   int aux_ld, aux_off;
   const float* bias;       // [N], nullable: added to the accumulator before the epilogue
   float act_a, act_b;      // XIELU: z > 0 ? act_a z^2 + z/2 : act_b (e^z - 1 - z) + z/2
+  // gemv_rows with z_expert only, n_shared > 0: batches z_shared .. z_shared + n_shared - 1 are rows of a second product of sizes of its own
+  // (the shared expert of a routed feed-forward), row r = z - z_shared:  A row r of As, C row r of Cs
+  int z_shared, n_shared, sN, sK, s_lda, s_ldc;
+  const void *sW1, *sW2;   // [sN][sK], packed
+  const float* As;
+  float* Cs;
 };
 
 template <typename WT, int EPI>
@@ -284,6 +292,7 @@ __device__ __forceinline__ void gemm_epilogue(const GemmP& P, float* __restrict_
   else if (EPI == HEPI_ADD) crow[n] += P.alpha * v;
   else if (EPI == HEPI_XIELU) crow[n] = v > 0.f ? fmaf(P.act_a * v, v, 0.5f * v) : fmaf(P.act_b, expm1f(v) - v, 0.5f * v);
   else if (EPI == HEPI_GEGLU) crow[n] = gelu_tanh_f(v) * v2;
+  else if (EPI == HEPI_SWIGLU) crow[n] = silu_f(v) * v2;
   else if (EPI == HEPI_SIGMUL) crow[n] *= sigmoid_f(v);
   else if (EPI == HEPI_RELU2) { const float r = fmaxf(v, 0.f); crow[n] = r * r; }
   else if (EPI == HEPI_SILU_SIG) crow[n] = n < P.aux_off ? silu_f(v) : sigmoid_f(v);
@@ -699,11 +708,21 @@ __global__ void __launch_bounds__(256) gemv_rows(const GemmP P) {
   constexpr int MR = 4, V = WVec<WT>::N;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, z = blockIdx.y;
   long long aoff, woff, coff;
-  int M = P.M;
-  if (P.z_expert) {
+  int M = P.M, N = P.N, K = P.K, lda = P.lda, ldw = P.ldw, ldc = P.ldc;
+  const void *Wp = P.W, *W2p = P.W2;
+  const float* Ap = P.A;
+  float* Cp = P.C;
+  if (P.z_expert && P.n_shared > 0 && z >= P.z_shared) {
+    N = P.sN; K = P.sK; lda = P.s_lda; ldw = P.sK; ldc = P.s_ldc;
+    Wp = P.sW1; W2p = P.sW2; Ap = P.As; Cp = P.Cs;
+    woff = 0;
+    aoff = (long long)(z - P.z_shared) * lda;
+    coff = (long long)(z - P.z_shared) * ldc;
+    M = 1;
+  } else if (P.z_expert) {
     woff = (long long)P.z_expert[z] * P.sW;
-    aoff = (long long)(z / P.z_adiv) * P.lda;
-    coff = (long long)z * P.ldc;
+    aoff = (long long)(z / P.z_adiv) * lda;
+    coff = (long long)z * ldc;
     M = 1;
   } else if (P.z_rows > 0) {
     aoff = woff = coff = 0;
@@ -712,27 +731,27 @@ __global__ void __launch_bounds__(256) gemv_rows(const GemmP P) {
     aoff = (long long)z * P.sA; woff = (long long)(z / P.z_wdiv) * P.sW; coff = (long long)z * P.sC;
   }
   const int mbase = P.z_rows > 0 ? z * MR : 0;
-  const WT* __restrict__ W = reinterpret_cast<const WT*>(P.W) + woff;
-  const WT* __restrict__ W2 = DUAL ? reinterpret_cast<const WT*>(P.W2) + woff : nullptr;
+  const WT* __restrict__ W = reinterpret_cast<const WT*>(Wp) + woff;
+  const WT* __restrict__ W2 = DUAL ? reinterpret_cast<const WT*>(W2p) + woff : nullptr;
   const float* arow[MR];
   int crow_i[MR];
 #pragma unroll
   for (int m = 0; m < MR; m++) {
     const int mm = mbase + (m < M ? m : 0);
     const int ar = (!P.z_expert && P.a_map) ? P.a_map[mm] / P.a_div : mm;
-    arow[m] = P.A + aoff + (size_t)ar * P.lda;
+    arow[m] = Ap + aoff + (size_t)ar * lda;
     crow_i[m] = (!P.z_expert && P.c_map) ? P.c_map[mm] : mm;
   }
-  const bool vec = (P.K % V == 0) && (P.ldw % V == 0) && (P.lda % 4 == 0) && ((woff * (long long)sizeof(WT)) % 16 == 0) &&
-                   ((reinterpret_cast<uintptr_t>(P.W) | (DUAL ? reinterpret_cast<uintptr_t>(P.W2) : 0)) % 16 == 0) &&
-                   (reinterpret_cast<uintptr_t>(P.A + aoff) % 16 == 0);
-  for (int n = blockIdx.x * 8 + warp; n < P.N; n += gridDim.x * 8) {
+  const bool vec = (K % V == 0) && (ldw % V == 0) && (lda % 4 == 0) && ((woff * (long long)sizeof(WT)) % 16 == 0) &&
+                   ((reinterpret_cast<uintptr_t>(Wp) | (DUAL ? reinterpret_cast<uintptr_t>(W2p) : 0)) % 16 == 0) &&
+                   (reinterpret_cast<uintptr_t>(Ap + aoff) % 16 == 0);
+  for (int n = blockIdx.x * 8 + warp; n < N; n += gridDim.x * 8) {
     float acc[MR] = {0.f, 0.f, 0.f, 0.f}, acc2[MR] = {0.f, 0.f, 0.f, 0.f};
-    const WT* w = W + (size_t)n * P.ldw;
-    const WT* w2 = DUAL ? W2 + (size_t)n * P.ldw : nullptr;
+    const WT* w = W + (size_t)n * ldw;
+    const WT* w2 = DUAL ? W2 + (size_t)n * ldw : nullptr;
     if (vec) {
 #pragma unroll 4
-      for (int k = lane * V; k < P.K; k += 32 * V) {   // unrolled: several 16-byte weight loads in flight per lane
+      for (int k = lane * V; k < K; k += 32 * V) {   // unrolled: several 16-byte weight loads in flight per lane
         float wv[V], wv2[V];
         WVec<WT>::load(w + k, wv);
         if (DUAL) WVec<WT>::load(w2 + k, wv2);
@@ -753,7 +772,7 @@ __global__ void __launch_bounds__(256) gemv_rows(const GemmP P) {
         }
       }
     } else {
-      for (int k = lane; k < P.K; k += 32) {
+      for (int k = lane; k < K; k += 32) {
         const float wv = to_f<WT>(w[k]);
         const float wv2 = DUAL ? to_f<WT>(w2[k]) : 0.f;
 #pragma unroll
@@ -771,7 +790,7 @@ __global__ void __launch_bounds__(256) gemv_rows(const GemmP P) {
       if (m < M) {
         const float v = warp_sum(acc[m]);
         const float v2 = DUAL ? warp_sum(acc2[m]) : 0.f;
-        if (lane == 0) gemm_epilogue<WT, EPI>(P, P.C + coff + (size_t)crow_i[m] * P.ldc, crow_i[m], n, v, v2);
+        if (lane == 0) gemm_epilogue<WT, EPI>(P, Cp + coff + (size_t)crow_i[m] * ldc, crow_i[m], n, v, v2);
       }
     }
   }
@@ -1055,7 +1074,8 @@ __global__ void __launch_bounds__(512, 1) hgrn2_scan(const float* __restrict__ p
 // position j is row j % ring of `cache`.  A CTA of 8 warps takes TQ consecutive tokens x 8 / TQ heads (one warp each) and walks
 // the union of their windows in tiles of 32 keys staged in shared memory, so a tile is read once per CTA; lane = key for the
 // scores, lane = latent channel (mod 32) for the weighted sum.  Online softmax in fp32.  With NS > 1 (few tokens: decoding) the
-// key range is cut into NS shares over blockIdx.z and latent_swa_merge combines the partial results.
+// key range is cut into NS shares over blockIdx.z and latent_swa_merge combines the partial results.  sink (nullable, one number
+// per head): e^sink joins the softmax denominator.
 // ---------------------------------------------------------------------------------------------------------------------
 // first position that position i sees: mask 0 is a sliding window of `size` positions (i included), mask 1 cuts the sequence
 // into chunks of `size` positions (borders at multiples of `size`), and i sees its own chunk up to itself
@@ -1088,7 +1108,7 @@ __device__ __forceinline__ float mod_score(const ScoreMods& sm, float s, int dis
 template <typename CT, int RV>
 __global__ void __launch_bounds__(256) latent_swa_attn(const float* __restrict__ qa, const CT* __restrict__ cache, float* __restrict__ out,
                                                        int T, int H, int R, const int* __restrict__ ctl, int mask, int window, int ring,
-                                                       float scale, int TQ, int NS, float* __restrict__ part) {
+                                                       float scale, int TQ, int NS, float* __restrict__ part, const float* __restrict__ sink) {
   extern __shared__ float sm[];
   const int NW = 8, HB = NW / TQ;
   float* qs = sm;                 // [NW][R]
@@ -1165,6 +1185,13 @@ __global__ void __launch_bounds__(256) latent_swa_attn(const float* __restrict__
     m = m_new;
   }
   if (!active) return;
+  if (sink && blockIdx.z == 0) {   // the sink joins the first share like a key with a zero value vector
+    const float sk = sink[h], m_new = fmaxf(m, sk), corr = expf(m - m_new);
+    l = l * corr + expf(sk - m_new);
+#pragma unroll
+    for (int k = 0; k < RV; k++) acc[k] *= corr;
+    m = m_new;
+  }
   if (NS > 1) {   // partial result of this key range: [t][h][split] -> {m, l, acc[R]} (not normalised); latent_swa_merge finishes
     float* pp = part + (((size_t)t * H + h) * NS + blockIdx.z) * (R + 2);
     if (lane == 0) { pp[0] = m; pp[1] = l; }
@@ -1398,23 +1425,78 @@ __global__ void __launch_bounds__(256) rms_open(float* __restrict__ x, const flo
   for (int i = threadIdx.x + 256 * kLnRegs; i < n; i += 256) hr[i] = xr[i] * sc * w[i];
 }
 
+// Sandwich blocks of RMS norms (rows of up to 256 * kLnRegs values): the end of one sublayer and the start of the next in one pass,
+//   x' = x + alpha rms(y) wy  -> xo (row pitch ldxo; the stream itself, or the input rows of the product that opens a loop pass);
+//   h = rms(x') wh            (wh nullable: no norm follows here).
+// wgt non-null: y_t = sum_k wgt[t][k] y[t * top + k] (+ wsh[t] ysh[t], nullable): routed experts' outputs and the shared one's.
+__global__ void __launch_bounds__(256) rms_add_norm(const float* __restrict__ y, const float* __restrict__ wgt, int top, const float* __restrict__ ysh,
+                                                    const float* __restrict__ wsh, const float* __restrict__ wy, const float* x, float* xo, int ldxo,
+                                                    const float* __restrict__ wh, float* __restrict__ h, int n,
+                                                    float eps, float alpha) {
+  __shared__ float red[33];
+  const size_t t = blockIdx.x;
+  float v[kLnRegs], u[kLnRegs], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < kLnRegs; k++) {
+    const int i = threadIdx.x + 256 * k;
+    v[k] = i < n && !wgt ? y[t * n + i] : 0.f;
+    u[k] = i < n ? x[t * n + i] : 0.f;
+  }
+  if (wgt) {
+    for (int e = 0; e < top; e++) {
+      const float we = wgt[t * top + e];
+      const float* yr = y + (t * top + e) * n;
+#pragma unroll
+      for (int k = 0; k < kLnRegs; k++) { const int i = threadIdx.x + 256 * k; if (i < n) v[k] = fmaf(we, yr[i], v[k]); }
+    }
+    if (ysh) {
+      const float we = wsh[t];
+#pragma unroll
+      for (int k = 0; k < kLnRegs; k++) { const int i = threadIdx.x + 256 * k; if (i < n) v[k] = fmaf(we, ysh[t * n + i], v[k]); }
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < kLnRegs; k++) ss = fmaf(v[k], v[k], ss);
+  float sc = alpha / sqrtf(block_sum(ss, red) / (float)n + eps);
+  ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < kLnRegs; k++) {
+    const int i = threadIdx.x + 256 * k;
+    if (i < n) { u[k] = fmaf(v[k] * sc, wy[i], u[k]); xo[t * ldxo + i] = u[k]; ss = fmaf(u[k], u[k], ss); }
+  }
+  if (!wh) return;
+  sc = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+#pragma unroll
+  for (int k = 0; k < kLnRegs; k++) { const int i = threadIdx.x + 256 * k; if (i < n) h[t * n + i] = u[k] * sc * wh[i]; }
+}
+
+// the T rows of a step (pitch ls) copied to rows of pitch ld
+__global__ void copy_rows(const float* __restrict__ src, int ls, float* __restrict__ dst, int ld, int n) {
+  for (int i = threadIdx.x; i < n; i += blockDim.x) dst[(size_t)blockIdx.x * ld + i] = src[(size_t)blockIdx.x * ls + i];
+}
+
 // RMS norm of every head of a row with one weight vector shared by the heads: out[t][h][:] = in[t][h][:] / rms(in[t][h][:]) * w[:].
-// One warp per (token, head) of P values.  gate (nullable, row pitch ld_gate): the result is multiplied by alpha silu(gate[t][h * P + i]).
+// One warp per (token, head) of P values.  gate (nullable, row pitch ld_gate): the result is multiplied by alpha silu(gate[t][h * P + i]),
+// or alpha sigmoid(.) with gate_sig.  w_stride: distance between the heads' weight vectors (0: one for all).  den (nullable, [T][H]): the head is
+// first divided by max(|den[t][h]|, e^-m) + 1e-6 with m = mrow[h * (T + 1) + t + 1] (the normaliser of a matrix memory).
 __global__ void __launch_bounds__(256) head_rmsnorm(const float* __restrict__ in, int ld_in, const float* __restrict__ w, float* __restrict__ out,
                                                     int ld_out, int T, int H, int P, float eps, const float* __restrict__ gate = nullptr,
-                                                    int ld_gate = 0, float alpha = 1.f) {
+                                                    int ld_gate = 0, float alpha = 1.f, int w_stride = 0, int gate_sig = 0,
+                                                    const float* __restrict__ den = nullptr, const float* __restrict__ mrow = nullptr) {
   const int lane = threadIdx.x & 31;
   const long long id = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   if (id >= (long long)T * H) return;
   const int t = (int)(id / H), h = (int)(id - (long long)t * H);
   const float* x = in + (size_t)t * ld_in + (size_t)h * P;
   float* o = out + (size_t)t * ld_out + (size_t)h * P;
+  w += (size_t)h * w_stride;
+  const float pre = den ? 1.f / (fmaxf(fabsf(den[(size_t)t * H + h]), expf(-mrow[(size_t)h * (T + 1) + t + 1])) + 1e-6f) : 1.f;
   float ss = 0.f;
-  for (int i = lane; i < P; i += 32) ss = fmaf(x[i], x[i], ss);
-  const float sc = 1.f / sqrtf(warp_sum(ss) / (float)P + eps);
+  for (int i = lane; i < P; i += 32) { const float v = x[i] * pre; ss = fmaf(v, v, ss); }
+  const float sc = pre / sqrtf(warp_sum(ss) / (float)P + eps);
   if (gate) {
     const float* g = gate + (size_t)t * ld_gate + (size_t)h * P;
-    for (int i = lane; i < P; i += 32) o[i] = x[i] * sc * w[i] * (alpha * silu_f(g[i]));
+    for (int i = lane; i < P; i += 32) o[i] = x[i] * sc * w[i] * (alpha * (gate_sig ? sigmoid_f(g[i]) : silu_f(g[i])));
   } else
     for (int i = lane; i < P; i += 32) o[i] = x[i] * sc * w[i];
 }
@@ -1438,6 +1520,8 @@ __global__ void add_row(float* __restrict__ x, int ld, const float* __restrict__
 // v_keep [T][GV], nullable, receives a copy of what is cached (the rows a later layer blends in).
 // k == nullptr: a layer that reads another layer's caches prepares its queries only and caches nothing.
 // With a norm per head, the heads of a token may be dealt over gridDim.y CTAs.
+// cv.w non-null (head_norm 2, separate values; q, k and v adjacent columns of the rows of q): every channel first goes through a causal
+// convolution over the tokens, continuing from the inputs in the ring cv.hist; 8 D floats of dynamic shared memory.
 // ---------------------------------------------------------------------------------------------------------------------
 __device__ __forceinline__ float rot_entry(const float* __restrict__ src, int c, int d, int rot_dims, int layout, float nrm, const float* __restrict__ w,
                                            float fpos, const float* __restrict__ freq, float mag) {
@@ -1455,13 +1539,33 @@ __device__ __forceinline__ float rot_entry(const float* __restrict__ src, int c,
   }
   return v;
 }
+// A causal convolution of the [q | k | v] channels: w [channels][taps], last tap on the current token; hist: ring over positions of `ring`
+// rows of inputs.  A step of at most ring - (taps - 1) tokens stores its inputs in rows that it does not read.
+struct ConvP {
+  const float* w;
+  float* hist;
+  int taps, ring, store;
+};
+__device__ __forceinline__ float conv_at(const ConvP& cv, const float* __restrict__ rows, int ld, int c, int ch, int pos0, int t) {
+  float acc = 0.f;
+  for (int j = 0; j < cv.taps; j++) {
+    const int tau = t - (cv.taps - 1) + j;
+    float v = 0.f;
+    if (tau >= 0) v = rows[(size_t)tau * ld + c];
+    else if (pos0 + tau >= 0) v = cv.hist[(size_t)((pos0 + tau) % cv.ring) * ch + c];
+    acc = fmaf(cv.w[(size_t)c * cv.taps + j], v, acc);
+  }
+  if (cv.store) cv.hist[(size_t)((pos0 + t) % cv.ring) * ch + c] = rows[(size_t)t * ld + c];
+  return acc;
+}
 __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q, float* __restrict__ q_out, int HD,
                                                     const float* __restrict__ k, const float* __restrict__ v_src, int GD, int GV, int ld_q, int ld_k, int ld_v,
                                                     const float* __restrict__ qw, const float* __restrict__ kw, float eps, int D,
                                                     int rot_dims, const float* __restrict__ freq, float mag,
                                                     const int* __restrict__ ctl, float* __restrict__ kcache,
                                                     float* __restrict__ vcache, int ring, int keep, const float* __restrict__ v_first,
-                                                    float lam, float* __restrict__ v_keep, int layout, int head_norm) {
+                                                    float lam, float* __restrict__ v_keep, int layout, int head_norm, const ConvP cv) {
+  extern __shared__ float cs[];   // [8][D] convolved head rows (cv.w)
   __shared__ float red[33];
   const int t = blockIdx.x, pos = ctl[0] + t;
   const size_t row = (size_t)cache_row(pos, keep, ring);
@@ -1475,12 +1579,19 @@ __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q,
       const bool isq = hh * D < HD;
       const int c0 = isq ? hh * D : hh * D - HD;
       const float* src = isq ? qr : kr;
+      if (cv.w) {
+        float* row_s = cs + w * D;
+        for (int d = lane; d < D; d += 32) row_s[d] = conv_at(cv, q, ld_q, hh * D + d, HD + GD + GV, ctl[0], t);
+        __syncwarp();
+        src = row_s - c0;
+      }
       float* dst = isq ? q_out + (size_t)t * HD + c0 : kcache + row * GD + c0;
       float ss = 0.f;
       if (head_norm == 2) {
         for (int d = lane; d < D; d += 32) ss = fmaf(src[c0 + d], src[c0 + d], ss);
         const float sc = 1.f / sqrtf(warp_sum(ss) / (float)D + eps);
         for (int d = lane; d < D; d += 32) dst[d] = rot_entry(src + c0, d, d, rot_dims, layout, sc, isq ? qw : kw, fpos, freq, mag);
+        __syncwarp();
         continue;
       }
       for (int d = lane; d < D; d += 32) {
@@ -1505,7 +1616,12 @@ __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q,
       else kcache[row * GD + c] = v;
     }
   }
-  if (!k || blockIdx.y > 0) return;
+  if (!k) return;
+  if (cv.w) {   // the value channels are dealt over the CTAs of the token too
+    for (int e = threadIdx.x + 256 * (int)blockIdx.y; e < GV; e += 256 * (int)gridDim.y) vcache[row * GV + e] = conv_at(cv, q, ld_q, HD + GD + e, HD + GD + GV, ctl[0], t);
+    return;
+  }
+  if (blockIdx.y > 0) return;
   const float* vr = v_src ? v_src + (size_t)t * ld_v : kr;
   for (int e = threadIdx.x; e < GV; e += blockDim.x) {
     float v = vr[e];
@@ -1528,8 +1644,9 @@ __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q,
 // the output is multiplied by sigmoid(gate[t][h * Dv + r]), with gate_head by sigmoid(gate[t][h]) (an output gate on the concatenated
 // heads; with NS > 1 the merge does it), and by alpha; ld_out: pitch of a token's output row.
 // ---------------------------------------------------------------------------------------------------------------------
-__host__ __device__ inline size_t gqa_attn_smem_floats(int H, int G, int D, int Dv) {
-  return (size_t)H * D + (size_t)H * 32 + (size_t)32 * (G * D + 1) + 2 * (size_t)H + (size_t)H * Dv + (size_t)H * H + 8 * 32 + 32 + 32;
+// HL query heads and GL key heads in a CTA (all of them with score mixing)
+__host__ __device__ inline size_t gqa_attn_smem_floats(int HL, int GL, int D, int Dv, bool talk) {
+  return (size_t)HL * D + (size_t)HL * 32 + (size_t)32 * (GL * D + 1) + 2 * (size_t)HL + (size_t)HL * Dv + (talk ? (size_t)HL * HL : 0) + 8 * 32 + 32 + 32;
 }
 __global__ void __launch_bounds__(256) gqa_attn(const float* __restrict__ q, const float* __restrict__ kc, const float* __restrict__ vc,
                                                 float* __restrict__ out, const float* __restrict__ talk, int T, int H, int G, int D,
@@ -1539,14 +1656,14 @@ __global__ void __launch_bounds__(256) gqa_attn(const float* __restrict__ q, con
   extern __shared__ float sm[];
   const int GD = G * D, GV = G * Dv, rep = H / G;
   const int GL = G / (int)gridDim.z, g0 = (int)blockIdx.z * GL, h0 = g0 * rep, HL = GL * rep, GDl = GL * D;   // this CTA's key heads and query heads
-  float* qs = sm;                              // [HL][D]   (the arrays are sized for all heads; a CTA uses the rows of its own)
-  float* sc = qs + (size_t)H * D;              // [HL][32] raw scores of the tile
-  float* ks = sc + (size_t)H * 32;             // [32][GDl + 1]
-  float* ms = ks + (size_t)32 * (GD + 1);      // [HL] running maximum
-  float* ls = ms + H;                          // [H] running sum
-  float* accs = ls + H;                        // [H][Dv]
-  float* tk = accs + (size_t)H * Dv;           // [H][H]
-  float* ps = tk + (size_t)H * H;              // [8][32] weights of the warp's current head
+  float* qs = sm;                              // [HL][D]
+  float* sc = qs + (size_t)HL * D;             // [HL][32] raw scores of the tile
+  float* ks = sc + (size_t)HL * 32;            // [32][GDl + 1]
+  float* ms = ks + (size_t)32 * (GDl + 1);     // [HL] running maximum
+  float* ls = ms + HL;                         // [HL] running sum
+  float* accs = ls + HL;                       // [HL][Dv]
+  float* tk = accs + (size_t)HL * Dv;          // [H][H] (score mixing: HL = H)
+  float* ps = tk + (talk ? (size_t)H * H : 0); // [8][32] weights of the warp's current head
   int* rowoff = reinterpret_cast<int*>(ps + 8 * 32);   // [32] cache rows of the tile's keys
   int* kdist = rowoff + 32;                            // [32] their distances from the query
   const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
@@ -1696,11 +1813,12 @@ __global__ void pack_ring_kv(const float* __restrict__ kc, const float* __restri
 //   q [T][H][D + Rd]: the last Rd entries of every head are rotated in place;  qa_rot (nullable) [T][H][R + Rd]: the rotated
 //   part is also copied behind the R entries that the absorbed key up-projection fills (decode-sized steps score
 //   [W_uk^T q_plain | q_rot] against the cache rows directly).
-// rot turns the pairs (2i, 2i + 1), i < rot_dims / 2, by pos * freq[i]; positions and angles are fp32.
+// rot turns the pairs (2i, 2i + 1) (layout 0) or (i, i + rot_dims / 2) (layout 1), i < rot_dims / 2, by pos * freq[i], cos and sin times
+// mag; positions and angles are fp32.
 // ---------------------------------------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256) mla_prepare(const float* __restrict__ dkv, int ld_dkv, const float* __restrict__ w, float eps,
                                                    float* __restrict__ q, float* __restrict__ qa_rot, int H, int D, int Rd, int R,
-                                                   int rot_dims, const float* __restrict__ freq, const int* __restrict__ ctl,
+                                                   int rot_dims, const float* __restrict__ freq, float mag, int layout, const int* __restrict__ ctl,
                                                    float* __restrict__ cache, int ring) {
   __shared__ float red[33];
   const int t = blockIdx.x, pos = ctl[0] + t, RW = R + Rd;
@@ -1714,19 +1832,20 @@ __global__ void __launch_bounds__(256) mla_prepare(const float* __restrict__ dkv
   const int half = rot_dims >> 1;
   // pairs of the shared key part (head index H) and of every query head
   for (int e = threadIdx.x; e < (H + 1) * half; e += blockDim.x) {
-    const int h = e / half, i = e - h * half;
+    const int h = e / half, i = e - h * half, ia = layout == 1 ? i : 2 * i, ib = layout == 1 ? i + half : 2 * i + 1;
     float sn, cs;
     sincosf(fpos * freq[i], &sn, &cs);
+    cs *= mag; sn *= mag;
     if (h == H) {
-      const float a = src[R + 2 * i], b = src[R + 2 * i + 1];
-      crow[R + 2 * i] = a * cs - b * sn;
-      crow[R + 2 * i + 1] = b * cs + a * sn;
+      const float a = src[R + ia], b = src[R + ib];
+      crow[R + ia] = a * cs - b * sn;
+      crow[R + ib] = b * cs + a * sn;
     } else {
       float* qr = q + ((size_t)t * H + h) * (D + Rd) + D;
-      const float a = qr[2 * i], b = qr[2 * i + 1];
+      const float a = qr[ia], b = qr[ib];
       const float ra = a * cs - b * sn, rb = b * cs + a * sn;
-      qr[2 * i] = ra; qr[2 * i + 1] = rb;
-      if (qa_rot) { float* o = qa_rot + ((size_t)t * H + h) * RW + R; o[2 * i] = ra; o[2 * i + 1] = rb; }
+      qr[ia] = ra; qr[ib] = rb;
+      if (qa_rot) { float* o = qa_rot + ((size_t)t * H + h) * RW + R; o[ia] = ra; o[ib] = rb; }
     }
   }
   for (int e = threadIdx.x; e < (H + 1) * (Rd - rot_dims); e += blockDim.x) {   // entries that pass unchanged
@@ -1775,21 +1894,48 @@ __global__ void __launch_bounds__(128) mix_heads(const float* __restrict__ in, f
 // Router of a routed feed-forward, one CTA per token.  mode 0: s = sigmoid(logits); the `top` experts with the largest
 // s + correction are taken (ties: lower index first), slot = rank; weights = s / (sum of the chosen s + 1e-20) * scale.
 // mode 1: the `top` experts with the largest logits are taken (ties: lower index first); weights = softmax over the chosen logits.
+// mode 2: s = softmax over all logits; the experts fall into `groups` equal runs of neighbours, and only those of the `keep` runs with the
+// largest best score may be taken (ties: lower index first); the `top` largest of them, weights = s * scale.
+// ldz: pitch of the logits' rows.  wsh (nullable): wsh[t] = sigmoid(logits[t][E]), the weight of a shared expert.
 // ---------------------------------------------------------------------------------------------------------------------
-__global__ void moe_route(const float* __restrict__ logits, const float* __restrict__ correction, int E, int top, float scale,
-                          int* __restrict__ idx, float* __restrict__ wgt, int mode) {
+__global__ void moe_route(const float* __restrict__ logits, int ldz, const float* __restrict__ correction, int E, int top, float scale,
+                          int* __restrict__ idx, float* __restrict__ wgt, int mode, int groups, int keep, float* __restrict__ wsh) {
   extern __shared__ float sm[];
+  __shared__ float red[33];
   float* sc = sm;            // [E]
   float* ch = sm + E;        // [E]
   float* sel = ch + E;       // [top]
+  float* gb = sel + top;     // [groups]
   const int t = blockIdx.x;
+  const float* z = logits + (size_t)t * ldz;
+  if (wsh && threadIdx.x == 0) wsh[t] = sigmoid_f(z[E]);
   for (int e = threadIdx.x; e < E; e += blockDim.x) {
-    const float z = logits[(size_t)t * E + e];
-    const float s = mode == 1 ? z : sigmoid_f(z);
+    const float s = mode == 0 ? sigmoid_f(z[e]) : z[e];
     sc[e] = s;
     ch[e] = s + (correction ? correction[e] : 0.f);
   }
   __syncthreads();
+  float zmax = 0.f, zsum = 1.f;
+  if (mode == 2) {           // selection by the logits (the softmax keeps their order)
+    const int per = E / groups;
+    for (int g = threadIdx.x; g < groups; g += blockDim.x) {
+      float b = sc[g * per];
+      for (int e = g * per + 1; e < (g + 1) * per; e++) b = fmaxf(b, sc[e]);
+      gb[g] = b;
+    }
+    __syncthreads();
+    zmax = gb[0];
+    for (int g = 1; g < groups; g++) zmax = fmaxf(zmax, gb[g]);
+    float s = 0.f;
+    for (int e = threadIdx.x; e < E; e += blockDim.x) {
+      s += expf(sc[e] - zmax);
+      const int g = e / per;
+      int rank = 0;
+      for (int i = 0; i < groups; i++) rank += (gb[i] > gb[g] || (gb[i] == gb[g] && i < g)) ? 1 : 0;
+      if (rank >= keep) ch[e] = -INFINITY;
+    }
+    zsum = block_sum(s, red);   // its barriers also order the writes of ch
+  }
   for (int e = threadIdx.x; e < E; e += blockDim.x) {
     const float c = ch[e];
     int rank = 0;
@@ -1797,7 +1943,9 @@ __global__ void moe_route(const float* __restrict__ logits, const float* __restr
     if (rank < top) { idx[(size_t)t * top + rank] = e; sel[rank] = sc[e]; }
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
+  if (mode == 2) {
+    for (int k = threadIdx.x; k < top; k += blockDim.x) wgt[(size_t)t * top + k] = expf(sel[k] - zmax) / zsum * scale;
+  } else if (threadIdx.x == 0) {
     if (mode == 1) {   // slot 0 holds the largest logit
       float sum = 0.f;
       for (int k = 0; k < top; k++) sum += expf(sel[k] - sel[0]);
@@ -1836,12 +1984,14 @@ __global__ void __launch_bounds__(1024) moe_plan(const int* __restrict__ idx, in
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) perm[atomicAdd(&off[idx[i]], 1)] = i;
 }
 
+// ysh (nullable, [T][width]): a shared expert's output, added with the weight wsh[t]
 __global__ void moe_combine(float* __restrict__ x, int ldx, const float* __restrict__ y, const float* __restrict__ wgt, int top,
-                            int width, float alpha, int add) {
+                            int width, float alpha, int add, const float* __restrict__ ysh = nullptr, const float* __restrict__ wsh = nullptr) {
   const int t = blockIdx.x;
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
     float s = 0.f;
     for (int k = 0; k < top; k++) s = fmaf(wgt[(size_t)t * top + k], y[((size_t)t * top + k) * width + c], s);
+    if (ysh) s = fmaf(wsh[t], ysh[(size_t)t * width + c], s);
     x[(size_t)t * ldx + c] = add ? x[(size_t)t * ldx + c] + alpha * s : alpha * s;
   }
 }

@@ -17,12 +17,14 @@
 //   mlp.router, mlp.router.b, mlp.e<j>.up|down                                                        (routed feed-forward, top-softmax router)
 //   mix.q|k|v (+ .conv), mix.b, mix.a, mix.A_log, mix.dt_bias, mix.norm, mix.g, mix.o                 (gated delta rule)
 //   mix.q|k|v|g, mix.norm, mix.o                                                                      (lightning attention)
+//   mix.q|k|v|g, mix.i, mix.i.b, mix.f, mix.f.b, mix.norm, mix.o                                      (mLSTM matrix memory)
+//   mlp.shared.gate|up|down|sg (shared expert), loop.in (product that opens a loop pass), mix.q|k|v.conv (attention behind convolutions)
 // Two mixers side by side name theirs mix.left.* and mix.right.*.
 // Grouped-query attention with its switches on adds mix.v, mix.q.b / k.b / v.b, mix.rel, mix.sink, mix.vmix; latent attention with a
-// rotated key part (DSK_MIX_MLA) has mix.dq, dq.norm, uq, dkv, dkv.norm, uk, uv, g, o; a gated dense feed-forward mlp.gate / up / down;
+// rotated key part (DSK_MIX_MLA) has mix.dq, dq.norm, uq, dkv, dkv.norm, uk, uv, sink, g, o; a gated dense feed-forward mlp.gate / up / down;
 // DSK_BLOCK_POST layers norm1 / norm2, ls1 / ls2, canon1 / canon2, rg1 / rg2 (+ .b); the model "bigram" beside "embed".
 // A parallel block computes, with h = norm1(x):  x += m (mixer(h) + ff(h));  a sandwich block  x += norm1b(mixer(norm1(x))),
-// x += norm2b(ff(norm2(x)));  a pre-norm block  x += m mixer(norm1(x)), x += m ff(norm2(x)).  Then, when the model has a per-layer token table,
+// x += norm2b(ff(norm2(x))) (with layer scales: ls1 / ls2 times the norms' results);  a pre-norm block  x += m mixer(norm1(x)), x += m ff(norm2(x)).  Then, when the model has a per-layer token table,
 // g = gelu_tanh(side.gate x) * side.embed[token][i*sd : (i+1)*sd],  y = side.proj g,  x += m * rmsnorm(y) * side.norm.
 // A layer loop repeats a range of layers with the same weights; each repetition ("layer run") keeps a separate cache / state.
 #pragma once
@@ -65,7 +67,7 @@ struct HLayer {
   HTensor in2, uq, gmat;
   float* dq_norm = nullptr;
   char have_in2[2] = {0, 0};
-  // DSK_BLOCK_POST: input convolutions, residual gates, closing norm weights (norm weight x layer scale, folded when the model is finalised)
+  // DSK_BLOCK_POST: input convolutions, residual gates; closing norm weights (norm weight x layer scale, folded when the model is finalised)
   HTensor rg1, rg2;
   float *rg1_b = nullptr, *rg2_b = nullptr, *canon1 = nullptr, *canon2 = nullptr, *ls1 = nullptr, *ls2 = nullptr, *close1 = nullptr, *close2 = nullptr;
   float norm1_s = 1.f, norm2_s = 1.f;   // single-number norm weights
@@ -77,7 +79,9 @@ struct HLayer {
   // routed feed-forward
   HTensor gate_s, up_s, down_s;     // expert stacks [E][ff][width], [E][ff][width], [E][width][ff]
   std::vector<char> have;           // 3 E flags
-  float *router = nullptr, *correction = nullptr;
+  float *router = nullptr, *correction = nullptr;   // with a shared expert the row of its weight (mlp.shared.sg) stands behind the router's
+  HTensor gate_sh, up_sh, down_sh;  // shared expert
+  char have_router[2] = {0, 0};
   // per-layer token input
   HTensor sgate, sproj;
   float* snorm = nullptr;
@@ -92,6 +96,9 @@ struct HLayer {
   // gated delta rule: its projections ride in qkv (att_layout), convolution taps of the [q | k | v] channels in one array; A_log, dt_bias
   // and lin_norm as above.  Side by side with attention, o holds both output matrices column by column: [left | right]
   float* gdn_conv_w = nullptr;
+  // attention behind short convolutions: taps of the [q | k | v] channels in conv_w, have_conv as below.  mLSTM: lin_in [q | k | v | g | i | f],
+  // padded to a multiple of 8 rows, lin_bias with the gates' biases, mnorm
+  char have_gate[2] = {0, 0}, have_gateb[2] = {0, 0};
   char have_gdn[6] = {0, 0, 0, 0, 0, 0}, have_conv[3] = {0, 0, 0}, have_o[2] = {0, 0};
 };
 
@@ -106,7 +113,7 @@ struct Model {
   dsk_hybrid_config c;
   std::vector<HLayer> L;
   std::vector<Run> runs;
-  HTensor embed, side_embed, head, bigram;
+  HTensor embed, side_embed, head, bigram, loop_in;
   float *final_norm = nullptr, *final_norm_b = nullptr, *loop_step = nullptr;
   int vmix_first = -1;              // the first layer whose values later value-mixing layers blend in
   size_t wsize = 4;                 // bytes per matrix element
@@ -119,8 +126,8 @@ struct LayerState {
   void* vcache = nullptr;           // grouped-query attention: values [ring][kv_heads * vdim]
   float* canon = nullptr;           // DSK_BLOCK_POST: [2][taps - 1][width] rings of the two input convolutions
   float* shift = nullptr;           // token shift: the mixer input of the sequence's last token [width]
-  float* lin = nullptr;             // gated linear recurrence: [heads][dim][vdim]
-  // gated delta rule: state in lin, the convolutions' inputs in hist, a ring over positions of taps - 1 + kConvSpare rows
+  float* lin = nullptr;             // gated linear recurrence: [heads][dim][vdim]; mLSTM: then n [heads][dim] and m [heads]
+  // gated delta rule (and attention behind convolutions): state in lin, the convolutions' inputs in hist, a ring over positions of taps - 1 + kConvSpare rows
   size_t ssm_bytes = 0, hist_bytes = 0, cache_bytes = 0, vcache_bytes = 0, canon_bytes = 0, shift_bytes = 0, lin_bytes = 0;
 };
 
@@ -140,6 +147,9 @@ struct State {
   int prefill_keys = 0;                      // keys a block of queries can see at most; 0: the matrix path is off
   float* y = nullptr;                        // a sublayer's output before its closing norm (sandwich and post blocks)
   float* emb = nullptr;                      // the step's embedding output (a layer loop that adds it again)
+  float* xin = nullptr;                      // [chunk][2 width]: [stream | embedding output], what the product that opens a loop pass reads
+  float *lgate = nullptr, *lden = nullptr;   // mLSTM: log gates and running maxima of the step, normalisers
+  float* wsh = nullptr;                      // [chunk] weights of the shared expert
   // linear attention: prepared q, k and v rows, per-block records, outputs ahead of their norm
   float *lq = nullptr, *lk = nullptr, *lv = nullptr, *lrec = nullptr, *lout = nullptr;
   float* hs = nullptr;                       // the token-shifted mixer input of the step
@@ -191,6 +201,24 @@ static AttLayout att_layout(const dsk_layer_spec& s) {
   return a;
 }
 
+// rows of an mLSTM mixer's stacked projection: [q | k | v | g | i | f], padded with zero rows to a multiple of 8
+struct MlstmLayout { long long k, v, g, i, f, total; };
+static MlstmLayout mlstm_layout(const dsk_layer_spec& s) {
+  const long long HN = (long long)s.lin_heads * s.lin_dim, HP = (long long)s.lin_heads * s.lin_vdim;
+  MlstmLayout a{HN, 2 * HN, 2 * HN + HP, 2 * HN + 2 * HP, 2 * HN + 2 * HP + s.lin_heads, 0};
+  a.total = (a.f + s.lin_heads + 7) / 8 * 8;
+  return a;
+}
+static bool has_attn(const dsk_layer_spec& s) { return s.mixer == DSK_MIX_GQA || s.mixer == DSK_MIX_MLA || s.mixer == DSK_MIX_LATENT_SWA; }
+
+// key heads per CTA of the decode-sized attention kernel: without score mixing as few as keep four query heads (half the warps) busy
+static int gqa_key_heads(int H, int G, bool talk) {
+  int GL = G;
+  if (!talk)
+    for (int d = G; d >= 1; d--) if (G % d == 0 && d * (H / G) >= 4) GL = d;
+  return GL;
+}
+
 static int validate(const dsk_hybrid_config& c, const dsk_layer_spec* L) {
   if (c.dim <= 0 || c.vocab_size <= 0 || c.n_layers <= 0 || c.max_seq_len <= 0) return fail(-1, "hybrid model: bad dimensions");
   if (c.quant != DSK_F32 && c.quant != DSK_BF16) return fail(-1, "hybrid models run with quant fp32 or bf16");
@@ -208,8 +236,10 @@ static int validate(const dsk_hybrid_config& c, const dsk_layer_spec* L) {
   if (c.block == DSK_BLOCK_POST && c.norm_kind == DSK_NORM_LAYER && c.norm_scalar) return fail(-1, "single-number norm weights belong to RMS norms");
   if (c.norm_bias && c.norm_kind != DSK_NORM_LAYER) return fail(-1, "norm biases belong to layer norms");
   if (c.norm_bias && c.block == DSK_BLOCK_SANDWICH) return fail(-1, "sandwich blocks run their layer norms without a bias");
-  if (c.block != DSK_BLOCK_POST && (c.canon_taps || c.res_gate || c.layer_scale || c.norm_scalar))
-    return fail(-1, "input convolutions, gated residuals, layer scales and single-number norm weights belong to post-norm blocks");
+  if (c.block != DSK_BLOCK_POST && (c.canon_taps || c.res_gate || c.norm_scalar))
+    return fail(-1, "input convolutions, gated residuals and single-number norm weights belong to post-norm blocks");
+  if (c.layer_scale && c.block != DSK_BLOCK_POST && c.block != DSK_BLOCK_SANDWICH) return fail(-1, "layer scales belong to post-norm and sandwich blocks");
+  if (c.loop_in && (c.block != DSK_BLOCK_SANDWICH || c.loop_embed)) return fail(-1, "loop passes that open with a product belong to sandwich blocks");
   if (c.canon_taps < 0 || c.canon_taps > kCanonMaxTaps) return fail(-1, "input convolution of %d taps unsupported (at most %d)", c.canon_taps, kCanonMaxTaps);
   if (c.bigram_buckets < 0) return fail(-1, "negative bigram table size");
   if (c.norm_kind != DSK_NORM_RMS && c.norm_kind != DSK_NORM_LAYER) return fail(-1, "unknown norm kind %d", c.norm_kind);
@@ -266,7 +296,12 @@ static int validate(const dsk_hybrid_config& c, const dsk_layer_spec* L) {
             !s.att_value_proj || s.att_vmix || s.att_bias)
           return fail(-1, "layer %d: a layer that reads layer %d's keys and values needs its key heads, sizes and kept positions, a value matrix there, and no biases or value mixing of its own", i, j);
       }
-      if (gqa_attn_smem_floats(s.att_heads, s.att_kv_heads, s.att_dim, s.att_vdim) * 4 > 200 * 1024)
+      if (s.att_sink < DSK_SINK_NONE || s.att_sink > DSK_SINK_ONE) return fail(-1, "layer %d: unknown softmax sink %d", i, s.att_sink);
+      if (s.att_conv < 0 || (s.att_conv > 0 && (!s.att_value_proj || s.att_qk_norm != DSK_QKNORM_HEAD_WEIGHT || s.att_kv_from >= 0 || s.att_vmix || s.mixer2)))
+        return fail(-1, "layer %d: convolutions behind the projections need a value matrix, weighted per-head norms, and no shared caches, value mixing or second mixer", i);
+      if (s.att_conv > 0 && s.att_dim > 1024) return fail(-1, "layer %d: head size %d > 1024 unsupported behind convolutions", i, s.att_dim);
+      const int GL = gqa_key_heads(s.att_heads, s.att_kv_heads, s.att_talk != 0);
+      if (gqa_attn_smem_floats(GL * (s.att_heads / s.att_kv_heads), GL, s.att_dim, s.att_vdim, s.att_talk != 0) * 4 > 200 * 1024)
         return fail(-1, "layer %d: %d heads x %d with %d key heads do not fit the attention kernel's shared memory", i, s.att_heads, s.att_dim, s.att_kv_heads);
     } else if (s.mixer == DSK_MIX_MLA) {
       if (s.att_heads <= 0 || s.att_dim <= 0 || s.att_rot_dim < 0 || s.att_vdim <= 0 || s.att_kv_rank <= 0 || s.att_q_rank <= 0 || s.att_window <= 0)
@@ -274,6 +309,13 @@ static int validate(const dsk_hybrid_config& c, const dsk_layer_spec* L) {
       if (s.att_kv_rank + s.att_rot_dim > 1024) return fail(-1, "layer %d: kv_rank + rot_dim %d > 1024 unsupported", i, s.att_kv_rank + s.att_rot_dim);
       if (s.rot_dims < 0 || s.rot_dims > s.att_rot_dim || s.rot_dims % 2 != 0) return fail(-1, "layer %d: rot dims %d must be even and at most rot_dim %d", i, s.rot_dims, s.att_rot_dim);
       if (s.rot_dims > 0 && !(s.rot_base > 0.f)) return fail(-1, "layer %d: bad rotation base", i);
+      if (s.rot_layout != DSK_ROT_PAIRS && s.rot_layout != DSK_ROT_HALF) return fail(-1, "layer %d: unknown rotation layout", i);
+      if (s.rot_factor > 0.f && (s.rot_scale != DSK_ROTSCALE_YARN || !(s.rot_base > 1.f) || s.rot_original <= 0 || !(s.rot_fast > 0.f) || !(s.rot_slow > 0.f)))
+        return fail(-1, "layer %d: bad rotation scaling", i);
+      if (s.att_sink < DSK_SINK_NONE || s.att_sink > DSK_SINK_ONE) return fail(-1, "layer %d: unknown softmax sink %d", i, s.att_sink);
+    } else if (s.mixer == DSK_MIX_MLSTM) {
+      if (s.lin_heads <= 0 || s.lin_dim <= 0 || s.lin_vdim <= 0 || !(s.lin_gate_cap > 0.f)) return fail(-1, "layer %d: bad matrix-memory sizes or gate cap", i);
+      if (s.lin_dim > 256) return fail(-1, "layer %d: key size %d > 256 unsupported (the recurrence keeps the state in registers)", i, s.lin_dim);
     } else if (s.mixer == DSK_MIX_HGRN2) {
       if (s.lin_heads <= 0 || s.lin_dim <= 0 || s.lin_vdim <= 0) return fail(-1, "layer %d: bad linear-recurrence sizes", i);
       if (s.lin_dim > 256) return fail(-1, "layer %d: key size %d > 256 unsupported (the recurrence keeps the state in registers)", i, s.lin_dim);
@@ -282,15 +324,20 @@ static int validate(const dsk_hybrid_config& c, const dsk_layer_spec* L) {
       if (s.lin_dim > 256) return fail(-1, "layer %d: key size %d > 256 unsupported (the recurrence keeps the state in registers)", i, s.lin_dim);
       for (int h = 0; h < s.lin_heads; h++) if (!(s.lin_decay[h] >= 0.f && s.lin_decay[h] <= 1.f)) return fail(-1, "layer %d: decay %g of head %d outside 0..1", i, (double)s.lin_decay[h], h);
     } else if (s.mixer != DSK_MIX_GDN) return fail(-1, "layer %d: unknown mixer %d", i, s.mixer);
-    if (s.mixer != DSK_MIX_SSD && s.mixer != DSK_MIX_HGRN2 && s.mixer != DSK_MIX_GDN && s.mixer != DSK_MIX_LIGHTNING && s.att_mask != DSK_MASK_WINDOW && s.att_mask != DSK_MASK_CHUNK) return fail(-1, "layer %d: unknown mask %d", i, s.att_mask);
+    if (has_attn(s) && s.att_mask != DSK_MASK_WINDOW && s.att_mask != DSK_MASK_CHUNK) return fail(-1, "layer %d: unknown mask %d", i, s.att_mask);
     if (s.ff_kind == DSK_FF_DENSE) {
       if (s.ff_hidden <= 0) return fail(-1, "layer %d: bad feed-forward size", i);
-      if (s.ff_act != DSK_ACT_XIELU && s.ff_act != DSK_ACT_GEGLU && s.ff_act != DSK_ACT_GLU_CLAMPED) return fail(-1, "layer %d: unknown activation %d", i, s.ff_act);
+      if (s.ff_act != DSK_ACT_XIELU && s.ff_act != DSK_ACT_GEGLU && s.ff_act != DSK_ACT_GLU_CLAMPED && s.ff_act != DSK_ACT_SWIGLU) return fail(-1, "layer %d: unknown activation %d", i, s.ff_act);
     } else if (s.ff_kind == DSK_FF_MOE) {
       if (s.ff_experts <= 0 || s.ff_top <= 0 || s.ff_top > s.ff_experts || s.ff_hidden <= 0) return fail(-1, "layer %d: bad routed feed-forward sizes", i);
       if (s.ff_experts > 4096) return fail(-1, "layer %d: more than 4096 experts unsupported", i);
-      if ((s.ff_router != DSK_ROUTER_SIGMOID && s.ff_router != DSK_ROUTER_TOP_SOFTMAX) || (s.ff_expert != DSK_EXPERT_GLU_CLAMPED && s.ff_expert != DSK_EXPERT_RELU2))
+      if (s.ff_router < DSK_ROUTER_SIGMOID || s.ff_router > DSK_ROUTER_SOFTMAX_GROUPS || s.ff_expert < DSK_EXPERT_GLU_CLAMPED || s.ff_expert > DSK_EXPERT_SWIGLU)
         return fail(-1, "layer %d: unknown router or expert kind", i);
+      const int groups = std::max(1, s.ff_groups), keep = s.ff_groups > 0 ? s.ff_groups_keep : 1;
+      if (s.ff_groups < 0 || s.ff_experts % groups != 0 || keep < 1 || keep > groups || s.ff_top > s.ff_experts / groups * keep)
+        return fail(-1, "layer %d: %d expert groups, %d kept, do not fit %d experts of which %d are taken", i, s.ff_groups, s.ff_groups_keep, s.ff_experts, s.ff_top);
+      if (groups > 1 && s.ff_router != DSK_ROUTER_SOFTMAX_GROUPS) return fail(-1, "layer %d: expert groups belong to the softmax router", i);
+      if (s.ff_shared < 0 || (s.ff_shared > 0 && s.ff_expert == DSK_EXPERT_RELU2)) return fail(-1, "layer %d: a shared expert needs gated experts", i);
     } else if (s.ff_kind != DSK_FF_NONE) return fail(-1, "layer %d: unknown feed-forward kind %d", i, s.ff_kind);
   }
   return 0;
@@ -329,6 +376,7 @@ static void set_kernel_attrs() {
   cudaFuncSetAttribute(lin_scan<false, A, B, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, big)
   DSK_LSCAN_ATTR(8, 1, 2); DSK_LSCAN_ATTR(16, 1, 2); DSK_LSCAN_ATTR(32, 1, 2); DSK_LSCAN_ATTR(8, 1, 4); DSK_LSCAN_ATTR(16, 1, 4); DSK_LSCAN_ATTR(32, 1, 4); DSK_LSCAN_ATTR(32, 2, 4);
 #undef DSK_LSCAN_ATTR
+  cudaFuncSetAttribute(gemm_mma<HEPI_SWIGLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMmaSmem);
   cudaFuncSetAttribute(gqa_attn, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   cudaFuncSetAttribute(mix_heads, cudaFuncAttributeMaxDynamicSharedMemorySize, big);
   done = true;
@@ -362,6 +410,11 @@ static dsk_model* model_create(const dsk_hybrid_config* cfg, const dsk_layer_spe
       }
     }
     L.sp.lin_decay = nullptr;   // the caller's array
+    if ((L.sp.mixer == DSK_MIX_GQA || L.sp.mixer == DSK_MIX_MLA) && L.sp.att_sink == DSK_SINK_ONE) {   // e^0 joins the softmax denominators
+      if (dmalloc(m, (void**)&L.sink, (size_t)L.sp.att_heads * 4) || cudaMemset(L.sink, 0, (size_t)L.sp.att_heads * 4) != cudaSuccess) {
+        fail(-2, "sink allocation failed"); dsk_model_destroy(m); return nullptr;
+      }
+    }
     if (L.sp.ff_kind == DSK_FF_MOE) L.have.assign(3 * (size_t)L.sp.ff_experts, 0);
     if (L.sp.mixer == DSK_MIX_LATENT_SWA) L.owner = L.sp.att_kv_from >= 0 ? L.sp.att_kv_from : i;
     if (L.sp.mixer == DSK_MIX_GQA) L.owner = L.sp.att_kv_from >= 0 ? L.sp.att_kv_from : i;
@@ -558,6 +611,10 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
     if (c.loop_times < 1) return fail(-4, "tensor %s: the model has no layer loop", name);
     return F32(&M->loop_step, c.loop_times, c.dim);
   }
+  if (nm == "loop.in") {
+    if (c.loop_times < 1 || !c.loop_in) return fail(-4, "tensor %s: the model has no such layer loop", name);
+    return MAT(M->loop_in, c.dim, 2LL * c.dim);
+  }
   if (nm == "side.embed") {
     if (c.side_dim <= 0) return fail(-4, "tensor %s: the model has no per-layer token input", name);
     return MAT(M->side_embed, c.vocab_size, (long long)c.side_dim * c.n_layers);
@@ -598,6 +655,8 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
     if (rest == "norm1b") return F32(&L.norm1b, c.dim, 0);
     if (rest == "norm2" && s.ff_kind != DSK_FF_NONE) return F32(&L.norm2, c.dim, 0);
     if (rest == "norm2b" && s.ff_kind != DSK_FF_NONE) return F32(&L.norm2b, c.dim, 0);
+    if (rest == "ls1" && c.layer_scale) return F32(&L.ls1, c.dim, 0);
+    if (rest == "ls2" && c.layer_scale && s.ff_kind != DSK_FF_NONE) return F32(&L.ls2, c.dim, 0);
   }
   if (rest.rfind("mix.", 0) == 0) {
     std::string k = rest.substr(4);
@@ -636,6 +695,24 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
       if (k == "g") return STACK(L.lin_in, tot, c.dim, 2 * HN + HP, HP, &L.have_lin[3]);
       if (k == "norm") return F32(&L.mnorm, HP, 0);
       if (k == "o") return MAT(L.o, c.dim, HP);
+    } else if (s.mixer == DSK_MIX_MLSTM) {
+      const long long H = s.lin_heads, HN = H * s.lin_dim, HP = H * s.lin_vdim;
+      const MlstmLayout a = mlstm_layout(s);
+      if (!L.lin_in.p) {
+        if (dmalloc(m, &L.lin_in.p, (size_t)a.total * c.dim * M->wsize + 16) || dmalloc(m, (void**)&L.lin_bias, (size_t)a.total * 4)) return -2;
+        CK(cudaMemset(L.lin_in.p, 0, (size_t)a.total * c.dim * M->wsize)); CK(cudaMemset(L.lin_bias, 0, (size_t)a.total * 4));
+        L.lin_in.rows = a.total; L.lin_in.cols = c.dim;
+      }
+      if (k == "q") return STACK(L.lin_in, a.total, c.dim, 0, HN, &L.have_lin[0]);
+      if (k == "k") return STACK(L.lin_in, a.total, c.dim, a.k, HN, &L.have_lin[1]);
+      if (k == "v") return STACK(L.lin_in, a.total, c.dim, a.v, HP, &L.have_lin[2]);
+      if (k == "g") return STACK(L.lin_in, a.total, c.dim, a.g, HP, &L.have_lin[3]);
+      if (k == "i") return STACK(L.lin_in, a.total, c.dim, a.i, H, &L.have_gate[0]);
+      if (k == "f") return STACK(L.lin_in, a.total, c.dim, a.f, H, &L.have_gate[1]);
+      if (k == "i.b") return STACKV(&L.lin_bias, a.total, a.i, H, &L.have_gateb[0]);
+      if (k == "f.b") return STACKV(&L.lin_bias, a.total, a.f, H, &L.have_gateb[1]);
+      if (k == "norm") return F32(&L.mnorm, HP, 0);
+      if (k == "o") return MAT(L.o, c.dim, HP);
     } else if (is_ssd(s)) {
       const long long inner = ssd_inner(s), ch = ssd_channels(s);
       if (k == "in") return MAT(L.in, ssd_proj(s), c.dim);
@@ -667,6 +744,7 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
       if (k == "uq") return MAT(L.uq, H * DK, Q);
       if (k == "uk") { if (int rc = MAT(L.ukT, H * s.att_dim, R, s.att_dim)) return rc; return MAT(L.uk, H * s.att_dim, R); }
       if (k == "uv") return MAT(L.uv, H * s.att_vdim, R);
+      if (k == "sink" && s.att_sink == DSK_SINK_HEAD) return F32(&L.sink, H, 0);
       if (k == "g" && s.att_out_gate) return MAT(L.gmat, H * s.att_vdim, c.dim);
       if (k == "o") return MAT(L.o, c.dim, H * s.att_vdim);
     } else if (s.mixer == DSK_MIX_GQA) {
@@ -690,12 +768,20 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
           if (k == "v.b") return STACKV(&L.qkv_b, tot, HD + GD, GV, &L.have_qkvb[2]);
         }
       }
+      if (s.att_conv > 0)
+        for (int n = 0; n < 3; n++)
+          if (k == std::string(1, "qkv"[n]) + ".conv") {   // taps of the stacked [q | k | v] channels
+            if (L.have_conv[n]) return fail(-4, "tensor %s uploaded twice", name);
+            if (!L.conv_w && dmalloc(m, (void**)&L.conv_w, (size_t)(HD + GD + GV) * s.att_conv * 4)) return -2;
+            L.have_conv[n] = 1;
+            return put(name, dtype, shape, data, nbytes, on_dev, n == 0 ? HD : n == 1 ? GD : GV, s.att_conv, L.conv_w + (size_t)(n == 0 ? 0 : n == 1 ? HD : HD + GD) * s.att_conv, false, 0);
+          }
       if (k == "rel" && s.att_rel_max > 0) {   // the number of distance buckets is the tensor's first size
         if (shape[0] < 2 || shape[0] > (1 << 20)) return fail(-4, "tensor %s: %lld distance buckets", name, (long long)shape[0]);
         L.rel_rows = (int)shape[0];
         return F32(&L.rel, shape[0], s.att_heads);
       }
-      if (k == "sink" && s.att_sink) return F32(&L.sink, s.att_heads, 0);
+      if (k == "sink" && s.att_sink == DSK_SINK_HEAD) return F32(&L.sink, s.att_heads, 0);
       if (k == "vmix" && s.att_vmix) return SCALAR(&L.vmix, &L.have_vmix);
       if (k == "vmix" || (k == "rel" && s.att_rel_max <= 0)) return 0;   // a checkpoint may carry them for layers that do not use them
       if (k == "q" && !s.att_value_proj) return MAT(L.q, HD, c.dim);
@@ -747,6 +833,19 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
   if (rest.rfind("mlp.", 0) == 0 && s.ff_kind == DSK_FF_MOE) {
     const std::string k = rest.substr(4);
     const long long E = s.ff_experts, ff = s.ff_hidden;
+    if (s.ff_shared > 0) {   // the shared expert's weight row stands behind the router's rows: one product for both
+      auto ROWS = [&](long long row0, long long rows, char* have) -> int {
+        if (*have) return fail(-4, "tensor %s uploaded twice", name);
+        if (!L.router && dmalloc(m, (void**)&L.router, (size_t)(E + 1) * c.dim * 4)) return -2;
+        *have = 1;
+        return put(name, dtype, shape, data, nbytes, on_dev, rows, c.dim, L.router + row0 * c.dim, false, 0);
+      };
+      if (k == "router") return ROWS(0, E, &L.have_router[0]);
+      if (k == "shared.sg") return ROWS(E, 1, &L.have_router[1]);
+      if (k == "shared.gate") return MAT(L.gate_sh, s.ff_shared, c.dim);
+      if (k == "shared.up") return MAT(L.up_sh, s.ff_shared, c.dim);
+      if (k == "shared.down") return MAT(L.down_sh, c.dim, s.ff_shared);
+    }
     if (k == "router") return F32(&L.router, E, c.dim);
     if (k == "correction" && s.ff_router == DSK_ROUTER_SIGMOID) return F32(&L.correction, E, 0);
     if (k == "router.b" && s.ff_router == DSK_ROUTER_TOP_SOFTMAX) return F32(&L.router_b, E, 0);
@@ -800,6 +899,7 @@ static int finalize(dsk_model* m) {
   };
   CK(cudaDeviceSynchronize());
   if (c.loop_times >= 1 && c.loop_stop > c.loop_start && !M->loop_step) return fail(-5, "missing tensor loop.step");
+  if (c.loop_in && c.loop_times >= 1 && c.loop_stop > c.loop_start && !M->loop_in.present) return fail(-5, "missing tensor loop.in");
   for (int i = 0; i < c.n_layers; i++) {
     HLayer& L = M->L[i];
     const dsk_layer_spec& s = L.sp;
@@ -823,7 +923,15 @@ static int finalize(dsk_model* m) {
     }
     if (c.block == DSK_BLOCK_SANDWICH && (!L.norm1b || (s.ff_kind != DSK_FF_NONE && (!L.norm2 || !L.norm2b))))
       return fail(-5, "layer %d: missing norm tensors (norm1b, norm2, norm2b)", i);
+    if (c.block == DSK_BLOCK_SANDWICH) {   // closing norm weights, times the layer scales
+      const bool ff = s.ff_kind != DSK_FF_NONE;
+      if (c.layer_scale && (!L.ls1 || (ff && !L.ls2))) return fail(-5, "layer %d: missing layer scale tensors (ls1, ls2)", i);
+      if (fold(L.norm1b, 1.f, L.ls1, &L.close1) || (ff && fold(L.norm2b, 1.f, L.ls2, &L.close2))) return -2;
+    }
     if (s.mixer == DSK_MIX_GDN) {
+    } else if (s.mixer == DSK_MIX_MLSTM) {
+      L.lin_in.present = L.have_lin[0] && L.have_lin[1] && L.have_lin[2] && L.have_lin[3] && L.have_gate[0] && L.have_gate[1];
+      if (!L.lin_in.present || !L.have_gateb[0] || !L.have_gateb[1] || !L.mnorm || !L.o.present) return fail(-5, "layer %d: missing matrix-memory tensors (mix.q, k, v, g, i, i.b, f, f.b, norm, o)", i);
     } else if (s.mixer == DSK_MIX_LIGHTNING) {
       L.lin_in.present = L.have_lin[0] && L.have_lin[1] && L.have_lin[2] && L.have_lin[3];
       if (!L.lin_in.present || !L.mnorm || !L.o.present) return fail(-5, "layer %d: missing lightning-attention tensors (mix.q, k, v, g, norm, o)", i);
@@ -842,6 +950,7 @@ static int finalize(dsk_model* m) {
       } else if (!L.q.present || !L.kproj.present) return fail(-5, "layer %d: missing attention tensors (mix.q, k)", i);
       if (!L.o.present || (s.att_qk_norm != DSK_QKNORM_HEAD && (!L.q_norm || !L.k_norm)) || (s.att_talk && !L.talk))
         return fail(-5, "layer %d: missing attention tensors (mix.q.norm, k.norm, talk, o)", i);
+      if (s.att_conv > 0 && !(L.have_conv[0] && L.have_conv[1] && L.have_conv[2])) return fail(-5, "layer %d: missing convolution taps (mix.q.conv, k.conv, v.conv)", i);
       if ((s.att_sink && !L.sink) || (s.att_rel_max > 0 && !L.rel) || (s.att_vmix && !L.have_vmix && i != M->vmix_first))
         return fail(-5, "layer %d: missing attention tensors (mix.sink, rel, vmix)", i);
       if (s.att_rel_max > 0) {   // distance -> bucket, in double: below half the buckets one distance each, then logarithmic steps up to att_rel_max
@@ -855,8 +964,8 @@ static int finalize(dsk_model* m) {
       }
     } else if (s.mixer == DSK_MIX_MLA) {
       L.in2.present = L.have_in2[0] && L.have_in2[1];
-      if (!L.in2.present || !L.dq_norm || !L.dkv_norm || !L.uq.present || !L.ukT.present || !L.uk.present || !L.uv.present || !L.o.present || (s.att_out_gate && !L.gmat.present))
-        return fail(-5, "layer %d: missing latent-attention tensors (mix.dq, dq.norm, uq, dkv, dkv.norm, uk, uv, g, o)", i);
+      if (!L.in2.present || !L.dq_norm || !L.dkv_norm || !L.uq.present || !L.ukT.present || !L.uk.present || !L.uv.present || !L.o.present || (s.att_out_gate && !L.gmat.present) || (s.att_sink && !L.sink))
+        return fail(-5, "layer %d: missing latent-attention tensors (mix.dq, dq.norm, uq, dkv, dkv.norm, uk, uv, sink, g, o)", i);
     } else if (is_ssd(s)) {
       if (!L.in.present || !L.o.present || !L.conv_w || !L.conv_b || !L.dt_bias || !L.A_log || !L.D || !L.mnorm)
         return fail(-5, "layer %d: missing state-space mixer tensors (mix.in, conv, conv.b, dt_bias, A_log, D, norm, o)", i);
@@ -869,7 +978,9 @@ static int finalize(dsk_model* m) {
     } else if (s.ff_kind == DSK_FF_DENSE && (!L.up.present || !L.down.present || !L.up_b || !L.down_b || !L.act))
       return fail(-5, "layer %d: missing feed-forward tensors (mlp.up, up.b, down, down.b, act)", i);
     if (s.ff_kind == DSK_FF_MOE) {
-      if (!L.router || (s.ff_router == DSK_ROUTER_SIGMOID ? !L.correction : !L.router_b)) return fail(-5, "layer %d: missing mlp.router / mlp.correction / mlp.router.b", i);
+      if (s.ff_shared > 0 && (!L.have_router[0] || !L.have_router[1] || !L.gate_sh.present || !L.up_sh.present || !L.down_sh.present))
+        return fail(-5, "layer %d: missing mlp.router or shared expert tensors (mlp.shared.gate, up, down, sg)", i);
+      if (!L.router || (s.ff_router == DSK_ROUTER_SIGMOID && !L.correction) || (s.ff_router == DSK_ROUTER_TOP_SOFTMAX && !L.router_b)) return fail(-5, "layer %d: missing mlp.router / mlp.correction / mlp.router.b", i);
       for (size_t k = s.ff_expert == DSK_EXPERT_RELU2 ? (size_t)s.ff_experts : 0; k < L.have.size(); k++)
         if (!L.have[k]) return fail(-5, "layer %d: missing expert tensor mlp.e%zu.%s", i, k % s.ff_experts, k / s.ff_experts == 0 ? "gate" : k / s.ff_experts == 1 ? "up" : "down");
     }
@@ -889,7 +1000,7 @@ static double active_bytes(const dsk_model* m) {
     const HLayer& L = M->L[R.layer];
     const dsk_layer_spec& s = L.sp;
     double mat = 0, f32 = W;
-    if (R.pass >= 0) f32 += W;
+    if (R.pass >= 0) { f32 += W; if (c.loop_in) mat += 2 * W * W; }
     if (c.block == DSK_BLOCK_PRE && s.ff_kind != DSK_FF_NONE) f32 += W;
     if (has_gdn(s)) {
       const double KD = (double)gdn_qk(s), RV = (double)gdn_v(s);
@@ -905,6 +1016,10 @@ static double active_bytes(const dsk_model* m) {
     if (c.token_shift) f32 += W;
     if (c.norm_bias) f32 += W * (s.ff_kind != DSK_FF_NONE ? 2 : 1);
     if (s.mixer == DSK_MIX_GDN) {
+    } else if (s.mixer == DSK_MIX_MLSTM) {
+      const double H = s.lin_heads, HN = H * s.lin_dim, HP = H * s.lin_vdim;
+      mat += (2 * HN + 2 * HP + 2 * H) * W + W * HP;
+      f32 += HP + 2 * H;
     } else if (s.mixer == DSK_MIX_LIGHTNING) {
       const double HN = (double)s.lin_heads * s.lin_dim, HP = (double)s.lin_heads * s.lin_vdim;
       mat += (2 * HN + 2 * HP) * W + W * HP;
@@ -917,17 +1032,17 @@ static double active_bytes(const dsk_model* m) {
       const bool reads = s.att_kv_from >= 0;
       const double HD = (double)s.att_heads * s.att_dim, GD = reads ? 0.0 : (double)s.att_kv_heads * s.att_dim, GV = s.att_value_proj && !reads ? (double)s.att_kv_heads * s.att_vdim : 0.0;
       mat += (HD + GD + GV) * W + W * s.att_heads * s.att_vdim + W * (double)att_layout(s).gate_rows;
-      f32 += (s.att_qk_norm == DSK_QKNORM_WHOLE ? HD + GD : s.att_qk_norm == DSK_QKNORM_HEAD_WEIGHT ? 2.0 * s.att_dim : 0.0) + (s.att_talk ? (double)s.att_heads * s.att_heads : 0.0) + (s.att_bias ? HD + GD + GV : 0.0) + (s.att_sink ? s.att_heads : 0);
+      f32 += (s.att_qk_norm == DSK_QKNORM_WHOLE ? HD + GD : s.att_qk_norm == DSK_QKNORM_HEAD_WEIGHT ? 2.0 * s.att_dim : 0.0) + (s.att_talk ? (double)s.att_heads * s.att_heads : 0.0) + (s.att_bias ? HD + GD + GV : 0.0) + (s.att_sink == DSK_SINK_HEAD ? s.att_heads : 0) + (HD + GD + GV) * s.att_conv;
     } else if (s.mixer == DSK_MIX_MLA) {
       const double H = s.att_heads, DK = s.att_dim + s.att_rot_dim, Rr = s.att_kv_rank, Q = s.att_q_rank;
       mat += (Q + Rr + s.att_rot_dim) * W + H * DK * Q + H * (s.att_dim + s.att_vdim) * Rr + (s.att_out_gate ? H * s.att_vdim * W : 0.0) + W * H * s.att_vdim;
-      f32 += Q + Rr;
+      f32 += Q + Rr + (s.att_sink == DSK_SINK_HEAD ? H : 0.0);
     } else if (is_ssd(s)) { mat += (double)ssd_proj(s) * W + W * ssd_inner(s); f32 += (double)ssd_channels(s) * (s.ssm_conv + 1) + 3.0 * s.ssm_heads + ssd_inner(s); }
     else {
       mat += (double)s.att_heads * s.att_dim * W + (double)s.att_heads * (s.att_dim + s.att_vdim) * s.att_kv_rank + W * s.att_heads * s.att_vdim;
       if (s.att_kv_from < 0) { mat += (double)s.att_kv_rank * W; f32 += s.att_kv_rank; }
     }
-    if (s.ff_kind == DSK_FF_MOE) { mat += (s.ff_expert == DSK_EXPERT_RELU2 ? 2.0 : 3.0) * s.ff_top * s.ff_hidden * W; f32 += (double)s.ff_experts * (W + 1); }
+    if (s.ff_kind == DSK_FF_MOE) { mat += (s.ff_expert == DSK_EXPERT_RELU2 ? 2.0 : 3.0) * s.ff_top * s.ff_hidden * W; f32 += (double)s.ff_experts * (W + 1); if (s.ff_shared > 0) { mat += 3.0 * s.ff_shared * W; f32 += W; } }
     if (s.ff_kind == DSK_FF_DENSE && s.ff_act != DSK_ACT_XIELU) mat += 3.0 * s.ff_hidden * W;
     else if (s.ff_kind == DSK_FF_DENSE) { mat += 2.0 * s.ff_hidden * W; f32 += s.ff_hidden + W; }
     if (c.side_dim > 0) { mat += 2.0 * c.side_dim * W + c.side_dim; f32 += W; }
@@ -944,6 +1059,7 @@ static bool lin_decode_fits(int N, int P) {
 
 // kernels one decoded token launches (embedding + layers + final norm + LM head + arg-max)
 static bool fused_norms(const dsk_hybrid_config& c);
+static bool rms_fused(const dsk_hybrid_config& c);
 static int launches_per_token(const dsk_model* m) {
   const Model* M = m->hy;
   int n = fused_norms(M->c) ? 3 : 4;
@@ -961,12 +1077,14 @@ static int launches_per_token(const dsk_model* m) {
     if (M->c.block == DSK_BLOCK_PRE && R.pass >= 0) n -= 1;   // the pass vector is added by the opening norm
     if (has_gdn(s)) n += lin_decode_fits(s.gdn_dim, s.gdn_vdim) ? 1 : 3 + (s.gdn_conv > 1 ? 1 : 0);
     if (s.mixer == DSK_MIX_GDN) n += 2;     // stacked projection, o
+    else if (s.mixer == DSK_MIX_MLSTM) n += lin_decode_fits(s.lin_dim, s.lin_vdim) ? 3 : 6;   // stacked projection, (gates, records,) recurrence, (norm,) o
     else if (s.mixer == DSK_MIX_LIGHTNING) n += lin_decode_fits(s.lin_dim, s.lin_vdim) ? 4 : 5;   // stacked projection, (records,) recurrence, norm, o
     else if (s.mixer == DSK_MIX_HGRN2) n += 4;   // stacked projection, recurrence, head norm, o
     else if (s.mixer == DSK_MIX_GQA) n += s.att_value_proj ? 5 : 6;   // q, k (or one stacked q / k / v (/ gate) product), norm + rotation, attention, merge, o
     else if (s.mixer == DSK_MIX_MLA) n += 10 + (s.att_out_gate ? 1 : 0);   // down-projections, query norm, query up, latent preparation, absorbed query, attention, merge, value up, (gate,) o
     else n += is_ssd(s) ? 5 + (s.ssm_conv > 1 ? 1 : 0) : 5 + (s.att_kv_from < 0 ? 2 : 0);
-    if (s.ff_kind == DSK_FF_MOE) n += post && M->c.norm_kind == DSK_NORM_LAYER && !M->c.res_gate && M->c.dim <= 256 * kLnRegs ? 4 : 5;
+    if (s.ff_kind == DSK_FF_MOE) n += (post && M->c.norm_kind == DSK_NORM_LAYER && !M->c.res_gate && M->c.dim <= 256 * kLnRegs && s.ff_shared == 0) || rms_fused(M->c) ? 4 : 5;
+    if (R.pass >= 0 && M->c.loop_in) n += 1 + (&R != &M->runs[0] && fused_norms(M->c) ? 1 : 0);   // product, its norm
     if (s.ff_kind == DSK_FF_DENSE) n += 2;
     if (M->c.side_dim > 0) n += 3;
   }
@@ -1025,7 +1143,7 @@ static dsk_state* state_create(dsk_model* m) {
   size_t mx0 = c.dim, mx1 = c.dim, mx2 = c.dim, mx3 = c.dim, mxE = 1, mxTop = 1;
   S->L.resize(M->runs.size());   // one state per layer run
   bool any_talk = false;
-  size_t mxLQ = 0, mxLV = 0, mxLH = 0;
+  size_t mxLQ = 0, mxLV = 0, mxLH = 0, mxMH = 0, mxShared = 0;
   size_t mxGV = 0;
   for (size_t r = 0; r < M->runs.size(); r++) {
     const int i = M->runs[r].layer;
@@ -1050,6 +1168,12 @@ static dsk_state* state_create(dsk_model* m) {
       mx3 = std::max<size_t>(mx3, RV + (sp.mixer2 ? (size_t)sp.att_heads * sp.att_vdim : 0));
     }
     if (sp.mixer == DSK_MIX_GDN) {
+    } else if (sp.mixer == DSK_MIX_MLSTM) {
+      const size_t H = sp.lin_heads, HN = H * sp.lin_dim, HP = H * sp.lin_vdim;
+      ls.lin_bytes = (HN * sp.lin_vdim + HN + H) * 4;   // S, n, m
+      if (salloc(S, (void**)&ls.lin, ls.lin_bytes)) return nullptr;
+      mx0 = std::max<size_t>(mx0, mlstm_layout(sp).total); mx3 = std::max<size_t>(mx3, HP);
+      mxLV = std::max(mxLV, HP); mxLH = std::max(mxLH, H); mxMH = std::max(mxMH, H);
     } else if (sp.mixer == DSK_MIX_LIGHTNING) {
       const size_t HN = (size_t)sp.lin_heads * sp.lin_dim, HP = (size_t)sp.lin_heads * sp.lin_vdim;
       ls.lin_bytes = HN * sp.lin_vdim * 4;
@@ -1072,6 +1196,10 @@ static dsk_state* state_create(dsk_model* m) {
       mx0 = std::max<size_t>(mx0, (sp.att_value_proj ? HD + GD + GV : HD) + (sp.att_out_gate ? (size_t)sp.att_heads * sp.att_vdim : 0)); mx1 = std::max<size_t>(mx1, GD); mx2 = std::max<size_t>(mx2, HD);
       mx3 = std::max<size_t>(mx3, (size_t)sp.att_heads * sp.att_vdim);
       any_talk |= sp.att_talk != 0;
+      if (sp.att_conv > 1) {
+        ls.hist_bytes = (size_t)(sp.att_conv - 1 + kConvSpare) * (HD + GD + GV) * 4;
+        if (salloc(S, (void**)&ls.hist, ls.hist_bytes)) return nullptr;
+      }
       if (sp.att_vmix) mxGV = std::max(mxGV, GV);
     } else if (sp.mixer == DSK_MIX_MLA) {
       const size_t H = sp.att_heads, RW = (size_t)sp.att_kv_rank + sp.att_rot_dim;
@@ -1099,8 +1227,9 @@ static dsk_state* state_create(dsk_model* m) {
     }
     if (sp.ff_kind == DSK_FF_MOE) {
       mxE = std::max<size_t>(mxE, sp.ff_experts); mxTop = std::max<size_t>(mxTop, sp.ff_top);
-      mx0 = std::max<size_t>(mx0, sp.ff_experts);
-      mx2 = std::max<size_t>(mx2, (size_t)sp.ff_top * sp.ff_hidden); mx3 = std::max<size_t>(mx3, (size_t)sp.ff_top * c.dim);
+      const size_t sh = sp.ff_shared > 0 ? 1 : 0;    // a shared expert's rows stand behind the routed ones'
+      mx0 = std::max<size_t>(mx0, sp.ff_experts + sh); mxShared = std::max(mxShared, sh);
+      mx2 = std::max<size_t>(mx2, (size_t)sp.ff_top * sp.ff_hidden + sp.ff_shared); mx3 = std::max<size_t>(mx3, (size_t)(sp.ff_top + sh) * c.dim);
     }
     if (sp.ff_kind == DSK_FF_DENSE) mx2 = std::max<size_t>(mx2, sp.ff_hidden);
     mx1 = std::max<size_t>(mx1, c.side_dim);
@@ -1121,7 +1250,7 @@ static dsk_state* state_create(dsk_model* m) {
     size_t keys = 0, hd = 0, hv = 0, heads = 0, pack_es = 0;
     bool latent = false;
     for (const HLayer& L : M->L) {
-      if (L.sp.mixer == DSK_MIX_SSD || L.sp.mixer == DSK_MIX_HGRN2 || L.sp.mixer == DSK_MIX_GDN || L.sp.mixer == DSK_MIX_LIGHTNING) continue;
+      if (!has_attn(L.sp)) continue;
       const size_t kh = L.sp.mixer == DSK_MIX_GQA ? L.sp.att_kv_heads : L.sp.att_heads;
       latent |= L.sp.mixer == DSK_MIX_LATENT_SWA || L.sp.mixer == DSK_MIX_MLA;
       if (L.sp.mixer == DSK_MIX_LATENT_SWA) pack_es = std::max(pack_es, M->wsize);
@@ -1146,6 +1275,9 @@ static dsk_state* state_create(dsk_model* m) {
   for (const HLayer& L : M->L)
     if (L.sp.mixer2 && !S->side && (cudaStreamCreateWithFlags(&S->side, cudaStreamNonBlocking) != cudaSuccess || cudaEventCreateWithFlags(&S->ev_fork, cudaEventDisableTiming) != cudaSuccess ||
                                     cudaEventCreateWithFlags(&S->ev_join, cudaEventDisableTiming) != cudaSuccess)) { fail(-2, "stream creation failed"); return nullptr; }
+  if (c.loop_in && c.loop_times >= 1) rc |= salloc(S, (void**)&S->xin, Tc * 2 * c.dim * 4);
+  if (mxMH) rc |= salloc(S, (void**)&S->lgate, 3 * (Tc + 1) * mxMH * 4) | salloc(S, (void**)&S->lden, Tc * mxMH * 4);
+  if (mxShared) rc |= salloc(S, (void**)&S->wsh, Tc * 4);
   if (mxLQ) rc |= salloc(S, (void**)&S->lq, Tc * mxLQ * 4) | salloc(S, (void**)&S->lk, Tc * mxLQ * 4) | salloc(S, (void**)&S->lv, Tc * mxLV * 4);
   if (c.block == DSK_BLOCK_SANDWICH || c.block == DSK_BLOCK_POST) rc |= salloc(S, (void**)&S->y, Tc * c.dim * 4);
   if (c.token_shift) rc |= salloc(S, (void**)&S->hs, Tc * c.dim * 4);
@@ -1222,6 +1354,7 @@ static void launch_gemm_mma(int epi, const GemmP& P, int Z, int tile_cap, cudaSt
     case HEPI_LINGATE: gemm_mma<HEPI_LINGATE><<<grid, 256, kMmaSmem, st>>>(P); break;
     case HEPI_SILU_SIG: gemm_mma<HEPI_SILU_SIG><<<grid, 256, kMmaSmem, st>>>(P); break;
     case HEPI_SOFTCAP: gemm_mma<HEPI_SOFTCAP><<<grid, 256, kMmaSmem, st>>>(P); break;
+    case HEPI_SWIGLU: gemm_mma<HEPI_SWIGLU><<<grid, 256, kMmaSmem, st>>>(P); break;
     default: gemm_mma<HEPI_GELU_MUL><<<grid, 256, kMmaSmem, st>>>(P); break;
   }
 }
@@ -1229,7 +1362,7 @@ static void launch_gemm_mma(int epi, const GemmP& P, int Z, int tile_cap, cudaSt
 template <typename WT>
 static void launch_gemm_t(int epi, const GemmP& P, int Z, bool small, int tile_cap, cudaStream_t st) {
   if (small) {
-    const dim3 grid((unsigned)std::max(1, std::min((P.N + 7) / 8, 148 * 8)), (unsigned)Z);
+    const dim3 grid((unsigned)std::max(1, std::min((std::max(P.N, P.n_shared > 0 ? P.sN : 0) + 7) / 8, 148 * 8)), (unsigned)Z);
     switch (epi) {
       case HEPI_STORE: gemv_rows<WT, HEPI_STORE><<<grid, 256, 0, st>>>(P); break;
       case HEPI_ADD: gemv_rows<WT, HEPI_ADD><<<grid, 256, 0, st>>>(P); break;
@@ -1241,6 +1374,7 @@ static void launch_gemm_t(int epi, const GemmP& P, int Z, bool small, int tile_c
       case HEPI_LINGATE: gemv_rows<WT, HEPI_LINGATE><<<grid, 256, 0, st>>>(P); break;
       case HEPI_SILU_SIG: gemv_rows<WT, HEPI_SILU_SIG><<<grid, 256, 0, st>>>(P); break;
       case HEPI_SOFTCAP: gemv_rows<WT, HEPI_SOFTCAP><<<grid, 256, 0, st>>>(P); break;
+      case HEPI_SWIGLU: gemv_rows<WT, HEPI_SWIGLU><<<grid, 256, 0, st>>>(P); break;
       default: gemv_rows<WT, HEPI_GELU_MUL><<<grid, 256, 0, st>>>(P); break;
     }
   } else {
@@ -1256,6 +1390,7 @@ static void launch_gemm_t(int epi, const GemmP& P, int Z, bool small, int tile_c
       case HEPI_LINGATE: gemm_tiled<WT, HEPI_LINGATE><<<grid, 256, 0, st>>>(P); break;
       case HEPI_SILU_SIG: gemm_tiled<WT, HEPI_SILU_SIG><<<grid, 256, 0, st>>>(P); break;
       case HEPI_SOFTCAP: gemm_tiled<WT, HEPI_SOFTCAP><<<grid, 256, 0, st>>>(P); break;
+      case HEPI_SWIGLU: gemm_tiled<WT, HEPI_SWIGLU><<<grid, 256, 0, st>>>(P); break;
       default: gemm_tiled<WT, HEPI_GELU_MUL><<<grid, 256, 0, st>>>(P); break;
     }
   }
@@ -1325,7 +1460,7 @@ static void launch_hgrn2(const dsk_layer_spec& sp, const float* proj, int ld, fl
 
 // the walk over the blocks of a step (lin_scan): lanes per channel group by the key size, warps per CTA by how many CTAs there are
 static void launch_lin_scan(bool delta, const float* q, const float* k, int ldq, int hs, int rep, const float* v, int ldv, const float* rec, float* state,
-                            float* out, int ldo, int T, int H, int N, int P, cudaStream_t st) {
+                            float* out, int ldo, int T, int H, int N, int P, cudaStream_t st, float* nst = nullptr, float* den = nullptr) {
   const int TPC = N <= 32 ? 8 : N <= 64 ? 16 : 32, RQ = N <= 128 ? 1 : 2;
   int CPT = N > 128 ? 4 : 2;          // value channels per lane
   if (const char* e = getenv("DSK_LIN_CPT")) CPT = atoi(e) == 4 || N > 128 ? 4 : 2;   // A/B switch
@@ -1334,9 +1469,9 @@ static void launch_lin_scan(bool delta, const float* q, const float* k, int ldq,
   while (warps > 2 && H * ((P + warps * CW - 1) / (warps * CW)) < 148) warps = (warps + 1) / 2;
   if (const char* e = getenv("DSK_LIN_WARPS")) warps = std::max(1, std::min(8, atoi(e)));   // A/B switch
   const int PB = warps * CW;
-  const dim3 grid((unsigned)H, (unsigned)((P + PB - 1) / PB));
+  const dim3 grid((unsigned)H, (unsigned)((P + (nst ? 1 : 0) + PB - 1) / PB));
   const size_t smem = lin_scan_smem(4 * TPC * RQ, PB, warps, CW);
-#define DSK_LSCAN(D, A, B, C) lin_scan<D, A, B, C><<<grid, 32 * (warps + kLinStage), smem, st>>>(q, k, ldq, hs, rep, v, ldv, rec, state, out, ldo, T, H, N, P, PB)
+#define DSK_LSCAN(D, A, B, C) lin_scan<D, A, B, C><<<grid, 32 * (warps + kLinStage), smem, st>>>(q, k, ldq, hs, rep, v, ldv, rec, state, out, ldo, T, H, N, P, PB, nst, den)
 #define DSK_LSCANS(D) do { if (N > 128) DSK_LSCAN(D, 32, 2, 4); else if (CPT == 2) { if (N <= 32) DSK_LSCAN(D, 8, 1, 2); else if (N <= 64) DSK_LSCAN(D, 16, 1, 2); else DSK_LSCAN(D, 32, 1, 2); } \
   else { if (N <= 32) DSK_LSCAN(D, 8, 1, 4); else if (N <= 64) DSK_LSCAN(D, 16, 1, 4); else DSK_LSCAN(D, 32, 1, 4); } } while (0)
   if (delta) DSK_LSCANS(true); else DSK_LSCANS(false);
@@ -1344,13 +1479,13 @@ static void launch_lin_scan(bool delta, const float* q, const float* k, int ldq,
 #undef DSK_LSCAN
 }
 
-static void launch_lin_decode(bool delta, const GdnP& D, const float* decay, float* state, const float* norm_w, float eps, int gate_off, float alpha,
-                              float* out, int ldo, cudaStream_t st) {
+static void launch_lin_decode(int mode, const GdnP& D, const float* decay, float* state, const float* norm_w, float eps, int gate_off, float alpha,
+                              float* out, int ldo, cudaStream_t st, const MlstmP& memory = MlstmP{1.f, nullptr, nullptr}) {
   const int NG = std::min(kLinDecodeThreads / ((D.P + 3) / 4), D.N), need = (D.N + NG - 1) / NG;
   const size_t smem = lin_decode_smem(D.N, D.P);
-#define DSK_LDEC(X, R) lin_decode<X, R><<<D.H, kLinDecodeThreads, smem, st>>>(D, decay, state, norm_w, eps, gate_off, alpha, out, ldo)
+#define DSK_LDEC(X, R) lin_decode<X, R><<<D.H, kLinDecodeThreads, smem, st>>>(D, decay, state, norm_w, eps, gate_off, alpha, out, ldo, memory)
 #define DSK_LDECS(X) do { if (need <= 1) DSK_LDEC(X, 1); else if (need <= 2) DSK_LDEC(X, 2); else if (need <= 4) DSK_LDEC(X, 4); else if (need <= 8) DSK_LDEC(X, 8); else DSK_LDEC(X, 16); } while (0)
-  if (delta) DSK_LDECS(true); else DSK_LDECS(false);
+  if (mode == LIN_DELTA) DSK_LDECS(LIN_DELTA); else if (mode == LIN_MLSTM) DSK_LDECS(LIN_MLSTM); else DSK_LDECS(LIN_PLAIN);
 #undef DSK_LDECS
 #undef DSK_LDEC
 }
@@ -1361,7 +1496,7 @@ static void gdn_forward(State* S, const HLayer& L, LayerState& ls, int ldp, cons
   const int H = sp.gdn_heads, G = sp.gdn_kv_heads, N = sp.gdn_dim, P = sp.gdn_vdim, RV = H * P, NP = (N + 3) & ~3, CH = 2 * G * N + RV;
   const GdnP D{S->b0, ldp, (int)a.dq, (int)a.db, (int)a.da, L.gdn_conv_w, L.A_log, L.dt_bias, ls.hist, sp.gdn_conv - 1 + kConvSpare, sp.gdn_conv, T, H, G, N, P, S->d_ctl};
   if (T <= kLinDecodeTokens && lin_decode_fits(N, P)) {
-    launch_lin_decode(true, D, nullptr, ls.lin, L.lin_norm, eps, (int)a.dg, alpha, out, ldo, st);
+    launch_lin_decode(LIN_DELTA, D, nullptr, ls.lin, L.lin_norm, eps, (int)a.dg, alpha, out, ldo, st);
     S->launches++;
     return;
   }
@@ -1380,7 +1515,7 @@ static void lightning_forward(State* S, const HLayer& L, LayerState& ls, int ldp
   const int H = sp.lin_heads, N = sp.lin_dim, P = sp.lin_vdim, HN = H * N, HP = H * P;
   if (T <= kLinDecodeTokens && lin_decode_fits(N, P)) {
     const GdnP D{S->b0, ldp, 0, 0, 0, nullptr, nullptr, nullptr, nullptr, 1, 1, T, H, H, N, P, S->d_ctl};
-    launch_lin_decode(false, D, L.decay, ls.lin, nullptr, 0.f, 0, 1.f, S->lout, HP, st);
+    launch_lin_decode(LIN_PLAIN, D, L.decay, ls.lin, nullptr, 0.f, 0, 1.f, S->lout, HP, st);
     S->launches++;
     return;
   }
@@ -1389,10 +1524,29 @@ static void lightning_forward(State* S, const HLayer& L, LayerState& ls, int ldp
   S->launches += 2;
 }
 
+// mLSTM of T tokens from the stacked projection in S->b0 (columns of mlstm_layout) -> normed and gated heads in out [T][H P]
+static void mlstm_forward(State* S, const HLayer& L, LayerState& ls, int ldp, const MlstmLayout& a, float* out, float eps, int T, cudaStream_t st) {
+  const dsk_layer_spec& sp = L.sp;
+  const int H = sp.lin_heads, N = sp.lin_dim, P = sp.lin_vdim, HN = H * N, HP = H * P;
+  float *nst = ls.lin + (size_t)HN * P, *mst = nst + HN;
+  if (T <= kLinDecodeTokens && lin_decode_fits(N, P)) {
+    const GdnP D{S->b0, ldp, 0, (int)a.i, (int)a.f, nullptr, nullptr, nullptr, nullptr, 1, 1, T, H, H, N, P, S->d_ctl};
+    launch_lin_decode(LIN_MLSTM, D, nullptr, ls.lin, L.mnorm, eps, (int)a.g, 1.f, out, HP, st, MlstmP{sp.lin_gate_cap, nst, mst});
+    S->launches++;
+    return;
+  }
+  float *gi = S->lgate, *gf = gi + (size_t)H * T, *gm = gf + (size_t)H * T;
+  mlstm_gates<<<H, 256, 0, st>>>(S->b0, ldp, (int)a.i, (int)a.f, sp.lin_gate_cap, T, H, gi, gf, gm, mst);
+  mlstm_gram<<<dim3((unsigned)((T + kLinBlk - 1) / kLinBlk), (unsigned)H), 256, (size_t)2 * kLinBlk * (((N + 3) & ~3) + 4) * 4, st>>>(S->b0, S->b0 + HN, ldp, gi, gf, gm, T, H, N, S->lrec);
+  launch_lin_scan(false, S->b0, S->b0 + HN, ldp, N, 1, S->b0 + 2 * HN, ldp, S->lrec, ls.lin, S->lout, HP, T, H, N, P, st, nst, S->lden);
+  head_rmsnorm<<<(unsigned)(((long long)T * H + 7) / 8), 256, 0, st>>>(S->lout, HP, L.mnorm, out, HP, T, H, P, eps, S->b0 + a.g, ldp, 1.f, P, 1, S->lden, gm);
+  S->launches += 4;
+}
+
 static int R0(const Model* M, size_t ri) { return M->runs[ri].owner_run; }
 
 static void launch_attn(const float* qa, const float* cache, float* out, int T, int H, int R, const int* ctl, int mask, int window, int ring,
-                        float scale, float* part, cudaStream_t st) {
+                        float scale, float* part, cudaStream_t st, const float* sink = nullptr) {
   const int TQ = T >= 8 ? 8 : T >= 4 ? 4 : T >= 2 ? 2 : 1, HB = 8 / TQ;
   int NS = 1;
   if (T <= kAttnSplitTokens) {   // the widest key range a CTA can meet is window + TQ - 1 keys
@@ -1401,10 +1555,10 @@ static void launch_attn(const float* qa, const float* cache, float* out, int T, 
   }
   const dim3 grid((unsigned)((T + TQ - 1) / TQ), (unsigned)((H + HB - 1) / HB), (unsigned)NS);
   const size_t smem = ((size_t)8 * R + (size_t)32 * (R + 1)) * 4;
-  if (R <= 128) latent_swa_attn<float, 4><<<grid, 256, smem, st>>>(qa, cache, out, T, H, R, ctl, mask, window, ring, scale, TQ, NS, part);
-  else if (R <= 256) latent_swa_attn<float, 8><<<grid, 256, smem, st>>>(qa, cache, out, T, H, R, ctl, mask, window, ring, scale, TQ, NS, part);
-  else if (R <= 512) latent_swa_attn<float, 16><<<grid, 256, smem, st>>>(qa, cache, out, T, H, R, ctl, mask, window, ring, scale, TQ, NS, part);
-  else latent_swa_attn<float, 32><<<grid, 256, smem, st>>>(qa, cache, out, T, H, R, ctl, mask, window, ring, scale, TQ, NS, part);
+  if (R <= 128) latent_swa_attn<float, 4><<<grid, 256, smem, st>>>(qa, cache, out, T, H, R, ctl, mask, window, ring, scale, TQ, NS, part, sink);
+  else if (R <= 256) latent_swa_attn<float, 8><<<grid, 256, smem, st>>>(qa, cache, out, T, H, R, ctl, mask, window, ring, scale, TQ, NS, part, sink);
+  else if (R <= 512) latent_swa_attn<float, 16><<<grid, 256, smem, st>>>(qa, cache, out, T, H, R, ctl, mask, window, ring, scale, TQ, NS, part, sink);
+  else latent_swa_attn<float, 32><<<grid, 256, smem, st>>>(qa, cache, out, T, H, R, ctl, mask, window, ring, scale, TQ, NS, part, sink);
   if (NS > 1) latent_swa_merge<<<dim3((unsigned)(T * H), (unsigned)((R + 127) / 128)), 128, 0, st>>>(part, out, R, NS);
 }
 
@@ -1426,8 +1580,9 @@ static void norm_rows(const dsk_hybrid_config& c, State* S, const float* in, con
 }
 
 static bool fused_norms(const dsk_hybrid_config& c) {
-  return c.block == DSK_BLOCK_SANDWICH && c.norm_kind == DSK_NORM_LAYER && c.dim <= 256 * kLnRegs && c.side_dim == 0;
+  return c.block == DSK_BLOCK_SANDWICH && (c.norm_kind == DSK_NORM_LAYER || c.norm_groups == 1) && c.dim <= 256 * kLnRegs && c.side_dim == 0;
 }
+static bool rms_fused(const dsk_hybrid_config& c) { return fused_norms(c) && c.norm_kind == DSK_NORM_RMS; }
 
 // where a sublayer's last product goes: added into the residual stream (parallel blocks), or stored for the closing norm
 struct Sink { int epi; float* C; float alpha; };
@@ -1447,10 +1602,12 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
   const float mult = c.residual_mult;
   const float es = c.embed_scale != 0.f ? c.embed_scale : 1.f;
   const int nb = c.bigram_buckets;
+  float* keep_emb = S->xin ? S->xin + W : S->emb;   // the embedding output again, for a layer loop
+  const int ld_keep = S->xin ? 2 * W : W;
   if (bf) embed_rows<__nv_bfloat16><<<T, 256, 0, st>>>(S->d_tok, (const __nv_bfloat16*)M->embed.p, W, S->x, es, nb > 0 ? (const __nv_bfloat16*)M->bigram.p : nullptr,
-                                                       nb, c.bigram_mul_prev, c.bigram_mul_cur, S->d_ctl, S->d_prev, S->emb);
+                                                       nb, c.bigram_mul_prev, c.bigram_mul_cur, S->d_ctl, S->d_prev, keep_emb, ld_keep);
   else embed_rows<float><<<T, 256, 0, st>>>(S->d_tok, (const float*)M->embed.p, W, S->x, es, nb > 0 ? (const float*)M->bigram.p : nullptr, nb, c.bigram_mul_prev,
-                                            c.bigram_mul_cur, S->d_ctl, S->d_prev, S->emb);
+                                            c.bigram_mul_cur, S->d_ctl, S->d_prev, keep_emb, ld_keep);
   S->launches++;
   if (nb > 0) { carry_token<<<1, 1, 0, st>>>(S->d_tok, T, S->d_prev); S->launches++; }   // the next step's first token pairs with this step's last
   if (pos0 < 0) S->tl_used = 0;   // a captured step records no events
@@ -1458,8 +1615,9 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
   auto MK = [&](const char* label) { if (tl) mark(S, label, st); };
   MK("embed");
   const Sink to_x{HEPI_ADD, S->x, mult}, to_y{HEPI_STORE, S->y, 1.f};
-  // sandwich blocks of layer norms: "x += ln(y); h = ln(x)" runs as one kernel (not while the residual stream is being recorded)
-  const bool fuse = fused_norms(c) && !trace;
+  // sandwich blocks: "x += norm(y); h = norm(x)" runs as one kernel (not while the residual stream is being recorded)
+  const bool fuse = fused_norms(c) && !trace, frms = fuse && rms_fused(c);
+  bool xin_ready = false; // the stream already stands in S->xin (the coming run opens a loop pass with a product)
   bool h_ready = false;   // S->h already holds the norm that opens the coming run (or the final norm)
   bool hs_ready = false;  // S->hs already holds the token-shifted input of the coming run's mixer
   for (size_t ri = 0; ri < M->runs.size(); ri++) {
@@ -1508,7 +1666,14 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       rms_open<<<T, 256, 0, st>>>(S->x, again ? S->emb : nullptr, run.pass >= 0 ? M->loop_step + (size_t)run.pass * W : nullptr, L.norm1, S->h, W, c.norm_eps);
       S->launches++;
     } else if (!h_ready) {
-      if (run.pass >= 0) {   // a pass of the layer loop opens with its own vector added to the residual stream
+      if (run.pass >= 0 && c.loop_in) {   // a pass of the layer loop opens with a product over [stream | embedding], its vector as the bias
+        if (!xin_ready) { copy_rows<<<T, 256, 0, st>>>(S->x, W, S->xin, 2 * W, W); S->launches++; }
+        xin_ready = false;
+        GemmP In = gp(S->xin, 2 * W, M->loop_in.p, 2 * W, S->x, W, T, W, 2 * W);
+        In.bias = M->loop_step + (size_t)run.pass * W;
+        linear(S, bf, HEPI_STORE, In, 1, st);
+        MK("loop.in");
+      } else if (run.pass >= 0) {   // a pass of the layer loop opens with its own vector added to the residual stream
         add_row<<<T, 256, 0, st>>>(S->x, W, M->loop_step + (size_t)run.pass * W, W);
         S->launches++;
       }
@@ -1525,9 +1690,20 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       hin = S->hs;
     }
     // the closing norm of this run's last sublayer, fused with what opens the next run (its pass vector and first norm) or the head
-    auto close_run = [&](const float* wb) {
+    auto close_run = [&](const float* wb, int routed = 0) {   // routed > 0: the sublayer's output is the weighted sum of the routed rows in S->b3
       if (!fuse) { norm_rows(c, S, S->y, wb, nullptr, S->x, T, 1, mult, st); return; }
       const Run* next = ri + 1 < M->runs.size() ? &M->runs[ri + 1] : nullptr;
+      if (frms) {
+        const bool to_xin = next && next->pass >= 0;   // the pass opens with a product: its norm follows that
+        const bool product = to_xin && c.loop_in;
+        const bool shared = routed && sp.ff_shared > 0;
+        rms_add_norm<<<T, 256, 0, st>>>(routed ? S->b3 : S->y, routed ? S->wgt : nullptr, routed, shared ? S->b3 + (size_t)T * routed * W : nullptr, S->wsh, wb, S->x,
+                                        product ? S->xin : S->x, product ? 2 * W : W, to_xin ? nullptr : next ? M->L[next->layer].norm1 : M->final_norm, S->h, W, c.norm_eps, mult);
+        S->launches++;
+        xin_ready = product;
+        h_ready = !to_xin;
+        return;
+      }
       const float* row = next && next->pass >= 0 ? M->loop_step + (size_t)next->pass * W : nullptr;
       layer_norm_add_norm<<<T, 256, 0, st>>>(S->y, wb, S->x, row, next ? M->L[next->layer].norm1 : M->final_norm, S->h, W, c.norm_eps, mult);
       S->launches++;
@@ -1535,7 +1711,7 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
     };
     const Sink sink = (sandwich || post) ? to_y : to_x;
     // a routed feed-forward that closes with a layer norm and no gate: no separate pass for the weighted sum of the experts' outputs
-    const bool combine_in_norm = post && sp.ff_kind == DSK_FF_MOE && c.norm_kind == DSK_NORM_LAYER && !c.res_gate && W <= 256 * kLnRegs;
+    const bool combine_in_norm = post && sp.ff_kind == DSK_FF_MOE && c.norm_kind == DSK_NORM_LAYER && !c.res_gate && W <= 256 * kLnRegs && sp.ff_shared == 0;
     if (sp.mixer == DSK_MIX_GQA) {
       const int H = sp.att_heads, G = sp.att_kv_heads, D = sp.att_dim, V = sp.att_vdim, HD = H * D, GD = G * D, GV = G * V, rep = H / G;
       const int keep = sp.att_keep_first;
@@ -1557,7 +1733,7 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
         linear(S, bf, HEPI_STORE, gp(hin, W, L.qkv.p, W, S->b0, ldp, T, ldp, W), 1, st);
         MK("att.qk");
         qk_norm_rope<<<qk_grid, 256, 0, st>>>(S->b0, S->b2, HD, nullptr, nullptr, GD, GV, ldp, 0, 0, L.q_norm, nullptr, c.norm_eps, D, sp.rot_dims, L.rot_freq,
-                                        L.rot_mag, S->d_ctl, nullptr, nullptr, ring, keep, nullptr, 0.f, nullptr, sp.rot_layout, sp.att_qk_norm);
+                                        L.rot_mag, S->d_ctl, nullptr, nullptr, ring, keep, nullptr, 0.f, nullptr, sp.rot_layout, sp.att_qk_norm, ConvP{nullptr, nullptr, 0, 1, 0});
       } else if (sp.att_value_proj) {   // one product for the stacked q / k / v rows; the first value-mixing layer keeps its values for the later ones
         const int ld = ldp;
         GemmP P = gp(hin, W, L.qkv.p, W, S->b0, ld, T, ld, W);
@@ -1571,15 +1747,21 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
           CKL(cudaEventRecord(S->ev_join, S->side));
         }
         const bool blend = sp.att_vmix && li != M->vmix_first;
-        qk_norm_rope<<<qk_grid, 256, 0, st>>>(S->b0, S->b2, HD, S->b0 + HD, S->b0 + HD + GD, GD, GV, ld, ld, ld, L.q_norm, L.k_norm, c.norm_eps, D, sp.rot_dims,
+        ConvP cv{nullptr, nullptr, 0, 1, 0};
+        if (sp.att_conv > 0) cv = ConvP{L.conv_w, ls.hist, sp.att_conv, sp.att_conv - 1 + kConvSpare, sp.att_conv > 1 && T <= kConvSpare};
+        qk_norm_rope<<<qk_grid, 256, cv.w ? (size_t)8 * D * 4 : 0, st>>>(S->b0, S->b2, HD, S->b0 + HD, S->b0 + HD + GD, GD, GV, ld, ld, ld, L.q_norm, L.k_norm, c.norm_eps, D, sp.rot_dims,
                                         L.rot_freq, L.rot_mag, S->d_ctl, kc, vc, ring, keep, blend ? S->vfirst : nullptr, L.vmix,
-                                        sp.att_vmix && li == M->vmix_first ? S->vfirst : nullptr, sp.rot_layout, sp.att_qk_norm);
+                                        sp.att_vmix && li == M->vmix_first ? S->vfirst : nullptr, sp.rot_layout, sp.att_qk_norm, cv);
+        if (sp.att_conv > 1 && !cv.store) {   // a long step stores its last inputs after its convolutions
+          conv_ring_store<<<(HD + GD + GV + 127) / 128, 128, 0, st>>>(S->b0, ld, 0, ls.hist, cv.ring, T, HD + GD + GV, sp.att_conv, S->d_ctl);
+          S->launches++;
+        }
       } else {
         linear(S, bf, HEPI_STORE, gp(hin, W, L.q.p, W, S->b0, HD, T, HD, W), 1, st);
         linear(S, bf, HEPI_STORE, gp(hin, W, L.kproj.p, W, S->b1, GD, T, GD, W), 1, st);
         MK("att.qk");
         qk_norm_rope<<<qk_grid, 256, 0, st>>>(S->b0, S->b2, HD, S->b1, nullptr, GD, GV, HD, GD, GD, L.q_norm, L.k_norm, c.norm_eps, D, sp.rot_dims, L.rot_freq,
-                                        L.rot_mag, S->d_ctl, kc, vc, ring, keep, nullptr, 0.f, nullptr, sp.rot_layout, sp.att_qk_norm);
+                                        L.rot_mag, S->d_ctl, kc, vc, ring, keep, nullptr, 0.f, nullptr, sp.rot_layout, sp.att_qk_norm, ConvP{nullptr, nullptr, 0, 1, 0});
       }
       S->launches++;
       MK("att.norm+rot");
@@ -1614,11 +1796,8 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       } else {
         int NS = 1;
         if (T <= kAttnSplitTokens) NS = std::max(1, std::min((std::min(sp.att_window, ring) + keep + 31) / 32, kAttnSplitMax));
-        // without score mixing the key heads are dealt over CTAs, as few per CTA as keep four query heads (half the warps) busy
-        int GL = G;
-        if (!sp.att_talk)
-          for (int d = G; d >= 1; d--) if (G % d == 0 && d * rep >= 4) GL = d;
-        gqa_attn<<<dim3((unsigned)T, (unsigned)NS, (unsigned)(G / GL)), 256, gqa_attn_smem_floats(H, G, D, V) * 4, st>>>(
+        const int GL = gqa_key_heads(H, G, sp.att_talk != 0);   // without score mixing the key heads are dealt over CTAs
+        gqa_attn<<<dim3((unsigned)T, (unsigned)NS, (unsigned)(G / GL)), 256, gqa_attn_smem_floats(GL * rep, GL, D, V, sp.att_talk != 0) * 4, st>>>(
             S->b2, kc, vc, S->b3, sp.att_talk ? L.talk : nullptr, T, H, G, D, V, S->d_ctl, sp.att_mask, sp.att_window, ring, sp.att_scale, NS, S->part, sm,
             NS > 1 ? nullptr : gate, ldp, gate_head, ldo, lscale);
         if (NS > 1) latent_swa_merge<<<dim3((unsigned)(T * H), (unsigned)((V + 127) / 128)), 128, 0, st>>>(S->part, S->b3, V, NS, gate, ldp, H, gate_head, ldo, lscale);
@@ -1645,10 +1824,12 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       linear(S, bf, HEPI_STORE, gp(S->b2, Q, L.uq.p, Q, S->b0, H * DK, T, H * DK, Q), 1, st);       // q [T][H][D | Rd]
       const bool portion = pos0 >= 0 && T >= kPrefillMin && S->prefill_keys > 0;
       mla_prepare<<<T, 256, 0, st>>>(S->b1 + Q, ldi, L.dkv_norm, c.norm_eps, S->b0, portion ? nullptr : S->b2, H, D, Rd, R, sp.rot_dims, L.rot_freq,
-                                     S->d_ctl, cache, L.ring);
+                                     L.rot_mag, sp.rot_layout, S->d_ctl, cache, L.ring);
       S->launches++;
       MK("att.q+latent");
       float* ov = S->b3;   // [T][H*V] heads' outputs
+      ScoreMods sm{};
+      sm.sink = sp.att_sink ? L.sink : nullptr;
       if (portion) {
         // blocks of kPrefillQ queries: plain keys and values up-projected from the visible latents, the rotated key part appended to every
         // head's keys; scores, softmax and the value product in fp32
@@ -1669,7 +1850,7 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
           Sc.sA = DK; Sc.sW = (long long)Lk * DK; Sc.sC = (long long)Tq * Lk; Sc.alpha = sp.att_scale;
           linear(S, false, HEPI_STORE, Sc, H, st);
           MK("att.scores");
-          softmax_band<<<dim3((unsigned)Tq, (unsigned)H), 128, 0, st>>>(S->sc, Tq, Lk, first, qpos0, sp.att_mask, sp.att_window, 0, ScoreMods{});
+          softmax_band<<<dim3((unsigned)Tq, (unsigned)H), 128, 0, st>>>(S->sc, Tq, Lk, first, qpos0, sp.att_mask, sp.att_window, 0, sm);
           MK("att.softmax");
           GemmP Ov = gp(S->sc, Lk, S->vt, Lk, S->b3 + (size_t)t0 * H * V, H * V, Tq, V, Lk);
           Ov.sA = (long long)Tq * Lk; Ov.sW = (long long)V * Lk; Ov.sC = V;
@@ -1683,7 +1864,7 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
           P.sA = DK; P.sW = (long long)R * D; P.sC = RW;
           linear(S, bf, HEPI_STORE, P, H, st);
         }
-        launch_attn(S->b2, cache, S->b3, T, H, RW, S->d_ctl, sp.att_mask, sp.att_window, L.ring, sp.att_scale, S->part, st);
+        launch_attn(S->b2, cache, S->b3, T, H, RW, S->d_ctl, sp.att_mask, sp.att_window, L.ring, sp.att_scale, S->part, st, sm.sink);
         S->launches++;
         {  // value up-projection per head from the first R entries of the weighted cache rows
           GemmP P = gp(S->b3, H * RW, L.uv.p, R, S->b0, H * V, T, V, R);
@@ -1710,6 +1891,20 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       P.alpha = sink.alpha;
       linear(S, bf, sink.epi, P, 1, st);
       MK("gdn.o");
+    } else if (sp.mixer == DSK_MIX_MLSTM) {
+      const MlstmLayout lay = mlstm_layout(sp);
+      const int HP = sp.lin_heads * sp.lin_vdim, pw = (int)lay.total;
+      MK("norm");
+      GemmP In = gp(hin, W, L.lin_in.p, W, S->b0, pw, T, pw, W);
+      In.bias = L.lin_bias;
+      linear(S, bf, HEPI_STORE, In, 1, st);
+      MK("lin.in");
+      mlstm_forward(S, L, ls, pw, lay, S->b3, c.norm_eps, T, st);
+      MK("lin.scan");
+      GemmP P = gp(S->b3, HP, L.o.p, HP, sink.C, W, T, W, HP);
+      P.alpha = sink.alpha;
+      linear(S, bf, sink.epi, P, 1, st);
+      MK("lin.o");
     } else if (sp.mixer == DSK_MIX_LIGHTNING) {
       const int HN = sp.lin_heads * sp.lin_dim, HP = sp.lin_heads * sp.lin_vdim, pw = 2 * HN + 2 * HP;
       MK("norm");
@@ -1832,12 +2027,15 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       MK("norm");
     }
     if (sandwich) {   // x += norm1b(mixer output); the feed-forward then reads norm2 of the new x
-      if (sp.ff_kind == DSK_FF_NONE) close_run(L.norm1b);
-      else if (fuse) {
-        layer_norm_add_norm<<<T, 256, 0, st>>>(S->y, L.norm1b, S->x, nullptr, L.norm2, S->h, W, c.norm_eps, mult);
+      if (sp.ff_kind == DSK_FF_NONE) close_run(L.close1);
+      else if (frms) {
+        rms_add_norm<<<T, 256, 0, st>>>(S->y, nullptr, 0, nullptr, nullptr, L.close1, S->x, S->x, W, L.norm2, S->h, W, c.norm_eps, mult);
+        S->launches++;
+      } else if (fuse) {
+        layer_norm_add_norm<<<T, 256, 0, st>>>(S->y, L.close1, S->x, nullptr, L.norm2, S->h, W, c.norm_eps, mult);
         S->launches++;
       } else {
-        norm_rows(c, S, S->y, L.norm1b, nullptr, S->x, T, 1, mult, st);
+        norm_rows(c, S, S->y, L.close1, nullptr, S->x, T, 1, mult, st);
         norm_rows(c, S, S->x, L.norm2, nullptr, S->h, T, 0, 0.f, st);
       }
       MK("norm");
@@ -1852,7 +2050,7 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
       const int ff = sp.ff_hidden;
       GemmP U = gp(hin, W, L.gate_d.p, W, S->b2, ff, T, ff, W);
       U.W2 = L.up.p; U.lim = sp.ff_limit;
-      linear(S, bf, sp.ff_act == DSK_ACT_GLU_CLAMPED ? HEPI_GLU : HEPI_GEGLU, U, 1, st);
+      linear(S, bf, sp.ff_act == DSK_ACT_GLU_CLAMPED ? HEPI_GLU : sp.ff_act == DSK_ACT_SWIGLU ? HEPI_SWIGLU : HEPI_GEGLU, U, 1, st);
       MK("ff.up");
       GemmP Dn = gp(S->b2, ff, L.down.p, ff, sink.C, W, T, W, ff);
       Dn.alpha = sink.alpha;
@@ -1871,24 +2069,32 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
     }
     if (sp.ff_kind == DSK_FF_MOE) {
       const int E = sp.ff_experts, top = sp.ff_top, ff = sp.ff_hidden, pairs = T * top;
-      GemmP Rt = gp(hin, W, L.router, W, S->b0, E, T, E, W);   // router: fp32 weights in every mode
+      const bool shared = sp.ff_shared > 0;
+      const int ffs = sp.ff_shared, ldz = E + (shared ? 1 : 0), groups = std::max(1, sp.ff_groups);
+      GemmP Rt = gp(hin, W, L.router, W, S->b0, ldz, T, ldz, W);   // router: fp32 weights in every mode (and the shared expert's weight)
       Rt.bias = sp.ff_router == DSK_ROUTER_TOP_SOFTMAX ? L.router_b : nullptr;
       linear(S, false, HEPI_STORE, Rt, 1, st);
-      moe_route<<<T, 128, (size_t)(2 * E + top) * 4, st>>>(S->b0, sp.ff_router == DSK_ROUTER_SIGMOID ? L.correction : nullptr, E, top, sp.ff_router_scale, S->d_idx,
-                                                           S->wgt, sp.ff_router == DSK_ROUTER_TOP_SOFTMAX ? 1 : 0);
+      moe_route<<<T, 128, (size_t)(2 * E + top + groups) * 4, st>>>(S->b0, ldz, sp.ff_router == DSK_ROUTER_SIGMOID ? L.correction : nullptr, E, top, sp.ff_router_scale,
+                                                                    S->d_idx, S->wgt, sp.ff_router == DSK_ROUTER_SOFTMAX_GROUPS ? 2 : sp.ff_router == DSK_ROUTER_TOP_SOFTMAX ? 1 : 0,
+                                                                    groups, sp.ff_groups > 0 ? sp.ff_groups_keep : 1, shared ? S->wsh : nullptr);
       S->launches++;
       MK("moe.router");
       const bool relu2 = sp.ff_expert == DSK_EXPERT_RELU2;   // one up matrix per expert instead of a gated pair
-      const int epi_up = relu2 ? HEPI_RELU2 : HEPI_GLU;
+      const int epi_up = relu2 ? HEPI_RELU2 : sp.ff_expert == DSK_EXPERT_SWIGLU ? HEPI_SWIGLU : HEPI_GLU;
       GemmP G = gp(hin, W, relu2 ? L.up_s.p : L.gate_s.p, W, S->b2, ff, pairs, ff, W);
       G.W2 = relu2 ? nullptr : L.up_s.p; G.sW = (long long)ff * W; G.lim = sp.ff_limit;
       GemmP Dn = gp(S->b2, ff, L.down_s.p, ff, S->b3, W, pairs, W, ff);
       Dn.sW = (long long)ff * W;
+      float *hsh = S->b2 + (size_t)pairs * ff, *ysh = S->b3 + (size_t)pairs * W;   // the shared expert's hidden rows and outputs, behind the routed ones'
       if (T <= 4) {
         G.z_expert = S->d_idx; G.z_adiv = top; Dn.z_expert = S->d_idx; Dn.z_adiv = 1;
-        linear(S, bf, epi_up, G, pairs, st);
+        if (shared) {   // its rows ride in the same launches
+          G.z_shared = pairs; G.n_shared = T; G.sN = ffs; G.sK = W; G.s_lda = W; G.s_ldc = ffs; G.sW1 = L.gate_sh.p; G.sW2 = L.up_sh.p; G.As = hin; G.Cs = hsh;
+          Dn.z_shared = pairs; Dn.n_shared = T; Dn.sN = W; Dn.sK = ffs; Dn.s_lda = ffs; Dn.s_ldc = W; Dn.sW1 = L.down_sh.p; Dn.As = hsh; Dn.Cs = ysh;
+        }
+        linear(S, bf, epi_up, G, pairs + (shared ? T : 0), st);
         MK("moe.glu");
-        linear(S, bf, HEPI_STORE, Dn, pairs, st);
+        linear(S, bf, HEPI_STORE, Dn, pairs + (shared ? T : 0), st);
         MK("moe.down");
       } else {
         const int bm = bf ? 128 : 64;   // rows per tile of the product kernel that follows (gemm_mma / gemm_tiled)
@@ -1902,15 +2108,25 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
         MK("moe.glu");
         linear(S, bf, HEPI_STORE, Dn, 1, st, cap);
         MK("moe.down");
+        if (shared) {
+          GemmP Us = gp(hin, W, L.gate_sh.p, W, hsh, ffs, T, ffs, W);
+          Us.W2 = L.up_sh.p; Us.lim = sp.ff_limit;
+          linear(S, bf, epi_up, Us, 1, st);
+          linear(S, bf, HEPI_STORE, gp(hsh, ffs, L.down_sh.p, ffs, ysh, W, T, W, ffs), 1, st);
+          MK("moe.shared");
+        }
       }
       if (combine_in_norm) {   // x += ln(sum_k w_k y_k): the weighted sum of the experts' outputs is taken by the closing layer norm as it reads its row
         layer_norm<<<T, 256, 0, st>>>(S->b3, W, L.close2, L.norm2_bias, S->x, W, W, c.norm_eps, 1, mult, S->wgt, top);
-      } else moe_combine<<<T, 256, 0, st>>>(sink.C, W, S->b3, S->wgt, top, W, sink.alpha, sink.epi == HEPI_ADD ? 1 : 0);
-      S->launches++;
+        S->launches++;
+      } else if (!frms) {   // (sandwich blocks of RMS norms combine as they close)
+        moe_combine<<<T, 256, 0, st>>>(sink.C, W, S->b3, S->wgt, top, W, sink.alpha, sink.epi == HEPI_ADD ? 1 : 0, shared ? ysh : nullptr, S->wsh);
+        S->launches++;
+      }
       MK("moe.combine");
     }
     if (sandwich && sp.ff_kind != DSK_FF_NONE) {
-      close_run(L.norm2b);
+      close_run(L.close2, frms && sp.ff_kind == DSK_FF_MOE ? sp.ff_top : 0);
       MK("norm");
     }
     if (post && sp.ff_kind != DSK_FF_NONE && !combine_in_norm) {

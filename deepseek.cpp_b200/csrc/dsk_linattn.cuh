@@ -1,6 +1,8 @@
-// dsk_linattn.cuh — linear attention with a decayed matrix state per head, in two forms that share their kernels:
+// dsk_linattn.cuh — linear attention with a decayed matrix state per head, in three forms that share their kernels:
 //   delta rule (DELTA):  S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q      (g, beta per token and head)
 //   plain:               S <- g S + k v^T;  o = S^T q                                       (g fixed per head)
+//   mLSTM:               m' = max(f + m, i);  S <- e^(f + m - m') S + e^(i - m') k v^T;  n likewise with k alone (n is one more value
+//                        channel whose value is 1);  o = S^T q / (max(|n . q|, e^-m') + 1e-6)         (log gates f, i per token and head)
 //
 // Portions run it over blocks of kLinBlk tokens (a re-association of the same fp32 sums, no reduced precision).  With S0 the
 // state ahead of a block, G_j the product of the decays up to and including token j, and R(j, i) = G_j / G_i:
@@ -8,7 +10,7 @@
 //   U = (I + A)^-1 W,   w_j = beta_j (v_j - G_j S0^T k_j)            (plain: U = V)
 //   o_j = G_j S0^T q_j + sum_i M_ji u_i,    S <- G_end S0 + sum_j R(end, j) k_j u_j^T
 // The part that does not depend on the state (A, its inverse, M, the decays) is computed for all blocks of a step at once
-// (gdn_prepare / lin_gram); lin_scan then walks the blocks with the state in registers.  Decay ratios are exponentials of
+// (gdn_prepare / lin_gram / mlstm_gates + mlstm_gram); lin_scan then walks the blocks with the state in registers.  Decay ratios are exponentials of
 // sums of the logarithms between the two tokens, so a decay that underflows gives 0 and never 0 / 0, and nothing cancels.
 // Steps of up to kLinDecodeTokens tokens run token by token in lin_decode, for the delta rule together with its convolutions,
 // unit norms, gates, head norm and output gate.
@@ -183,6 +185,79 @@ __global__ void __launch_bounds__(256) lin_gram(const float* __restrict__ q, con
   if (tid == 0) R[kRecEnd] = expf(ld1 * (float)nt);
 }
 
+// mLSTM, the gates of a step, one CTA per head: log gates  i = cap tanh(raw / cap),  f = log sigmoid(cap tanh(raw / cap))  of every
+// token to gi / gf [H][T], and the running maximum to gm [H][T + 1]: gm[h][0] is the one carried in, m[h] then becomes the last.
+// The recurrence m' = max(f + m, i) is a scan of pairs (F, B): m -> max(F + m, B); a thread owns consecutive tokens.
+__device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+__global__ void __launch_bounds__(256) mlstm_gates(const float* __restrict__ proj, int ld, int i_off, int f_off, float cap, int T, int H,
+                                                   float* __restrict__ gi, float* __restrict__ gf, float* __restrict__ gm, float* __restrict__ m) {
+  __shared__ float sF[256], sB[256];
+  const int h = blockIdx.x, tid = threadIdx.x, per = (T + 255) / 256, t0 = min(T, tid * per), t1 = min(T, t0 + per);
+  float F = 0.f, B = -INFINITY;
+  for (int t = t0; t < t1; t++) {
+    const float a = cap * tanhf(proj[(size_t)t * ld + i_off + h] / cap), f = log_sigmoid_f(cap * tanhf(proj[(size_t)t * ld + f_off + h] / cap));
+    gi[(size_t)h * T + t] = a;
+    gf[(size_t)h * T + t] = f;
+    B = fmaxf(B + f, a);
+    F += f;
+  }
+  sF[tid] = F; sB[tid] = B;
+  __syncthreads();
+  for (int o = 1; o < 256; o <<= 1) {
+    const float pF = tid >= o ? sF[tid - o] : 0.f, pB = tid >= o ? sB[tid - o] : -INFINITY;
+    __syncthreads();
+    sB[tid] = fmaxf(pB + sF[tid], sB[tid]);
+    sF[tid] = pF + sF[tid];
+    __syncthreads();
+  }
+  const float m0 = m[h];
+  float cur = tid ? fmaxf(sF[tid - 1] + m0, sB[tid - 1]) : m0;
+  __syncthreads();   // every thread has read m[h]
+  float* out = gm + (size_t)h * (T + 1);
+  if (tid == 0) out[0] = m0;
+  for (int t = t0; t < t1; t++) { cur = fmaxf(gf[(size_t)h * T + t] + cur, gi[(size_t)h * T + t]); out[t + 1] = cur; }
+  if (t1 == T && t0 < T) m[h] = cur;
+}
+
+// mLSTM: the records of a step from q and k as they are (q is scaled by 1 / sqrt(N) here) and the gates above.  Grid (blocks, heads).
+__global__ void __launch_bounds__(256) mlstm_gram(const float* __restrict__ q, const float* __restrict__ k, int ld, const float* __restrict__ gi,
+                                                  const float* __restrict__ gf, const float* __restrict__ gm, int T, int H, int N, float* __restrict__ rec) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float sf[kLinBlk], si[kLinBlk], sx[kLinBlk + 1];
+  const int pitch = ((N + 3) & ~3) + 4, tid = threadIdx.x, t0 = blockIdx.x * kLinBlk, nt = min(kLinBlk, T - t0), h = blockIdx.y;
+  float* sq = sm;
+  float* sk = sq + kLinBlk * pitch;
+  for (int e = tid; e < kLinBlk * pitch; e += 256) {
+    const int t = e / pitch, n = e - t * pitch;
+    const bool ok = t < nt && n < N;
+    sq[e] = ok ? q[(size_t)(t0 + t) * ld + h * N + n] : 0.f;
+    sk[e] = ok ? k[(size_t)(t0 + t) * ld + h * N + n] : 0.f;
+  }
+  if (tid < kLinBlk) {
+    sf[tid] = tid < nt ? gf[(size_t)h * T + t0 + tid] : 0.f;
+    si[tid] = tid < nt ? gi[(size_t)h * T + t0 + tid] : 0.f;
+  }
+  if (tid <= kLinBlk) sx[tid] = gm[(size_t)h * (T + 1) + t0 + min(tid, nt)];   // sx[j + 1]: maximum behind token j
+  __syncthreads();
+  float kk, qk;
+  block_gram(sq, sk, pitch, (N + 3) >> 2, kk, qk);
+  const float qs = 1.f / sqrtf((float)N);
+  const int j = tid >> 4, i = tid & 15;
+  float* R = rec + ((size_t)blockIdx.x * H + h) * kRecFloats;
+  float lr = si[i] - sx[j + 1];               // logarithm of what token i's write is worth at token j
+  for (int l = i + 1; l <= j; l++) lr += sf[l];
+  R[kRecM + tid] = i <= j && j < nt ? expf(lr) * (qk * qs) : 0.f;
+  if (tid < kLinBlk) {
+    float lg = sx[0], le = si[tid] - sx[nt];
+    for (int l = 0; l <= tid; l++) lg += sf[l];
+    for (int l = tid + 1; l < nt; l++) le += sf[l];
+    R[kRecG + tid] = tid < nt ? expf(lg - sx[tid + 1]) * qs : 0.f;
+    R[kRecB + tid] = 1.f;
+    R[kRecE + tid] = tid < nt ? expf(le) : 0.f;
+    if (tid == nt - 1) R[kRecEnd] = expf(lg - sx[nt]);
+  }
+}
+
 // sums of 32 accumulators over TPC neighbouring lanes, scattered: afterwards a[0 .. 32 / TPC - 1] of a lane hold the totals of
 // the entries red_index(..) .. + 32 / TPC - 1
 template <int TPC>
@@ -213,12 +288,13 @@ __device__ __forceinline__ int reduce_index(int s) {
 // they bring the blocks' q, k, v and records through three buffers, two blocks ahead (16-byte asynchronous copies where the rows
 // allow it, plain loads otherwise), so a block costs the computing warps one barrier.
 // q, k: head stride hs (rows of N entries), v: head stride P; head h reads q / k head h / rep.
+// nst non-null: one more value channel (index P) whose value is 1 for every token, with its state in nst [H][N] and its output in den [T][H].
 // ---------------------------------------------------------------------------------------------------------------------
 constexpr int kLinStage = 2;           // staging warps of a CTA
 template <bool DELTA, int TPC, int RQ, int CPT>
 __global__ void __launch_bounds__(320) lin_scan(const float* __restrict__ q, const float* __restrict__ k, int ldq, int hs, int rep,
                                                 const float* __restrict__ v, int ldv, const float* __restrict__ rec, float* __restrict__ state,
-                                                float* __restrict__ out, int ldo, int T, int H, int N, int P, int PB) {
+                                                float* __restrict__ out, int ldo, int T, int H, int N, int P, int PB, float* __restrict__ nst, float* __restrict__ den) {
   extern __shared__ __align__(16) float sm[];
   constexpr int C = kLinBlk, PITCH = 4 * TPC * RQ, CW = CPT * (32 / TPC), VB = 32 / CPT;
   const int per = 2 * C * PITCH + C * PB + kRecFloats;     // one buffer: k [C][PITCH], q [C][PITCH], v [C][PB], record
@@ -235,7 +311,10 @@ __global__ void __launch_bounds__(320) lin_scan(const float* __restrict__ q, con
     for (int i = 0; i < 4; i++) {
       const int n = 4 * (s + TPC * r) + i;
 #pragma unroll
-      for (int c = 0; c < CPT; c++) S[r][i][c] = (n < N && pc + c < P && cw + grp * CPT + c < PB) ? state[((size_t)h * N + n) * P + pc + c] : 0.f;
+      for (int c = 0; c < CPT; c++) {
+        S[r][i][c] = (n < N && pc + c < P && cw + grp * CPT + c < PB) ? state[((size_t)h * N + n) * P + pc + c] : 0.f;
+        if (nst && n < N && pc + c == P && cw + grp * CPT + c < PB) S[r][i][c] = nst[(size_t)h * N + n];
+      }
     }
   const bool vec = (N & 3) == 0 && (ldq & 3) == 0 && (hs & 3) == 0 && ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k)) & 15) == 0;
   const bool vecv = (P & 3) == 0 && (PB & 3) == 0 && (ldv & 3) == 0 && (reinterpret_cast<uintptr_t>(v) & 15) == 0 && p0 + PB <= P;
@@ -277,7 +356,7 @@ __global__ void __launch_bounds__(320) lin_scan(const float* __restrict__ q, con
     } else {
       for (int e = stid; e < C * PB; e += ST) {
         const int t = e / PB, c = e - t * PB;
-        bv[e] = t < nt && p0 + c < P ? vs[(size_t)t * ldv + c] : 0.f;
+        bv[e] = t < nt && p0 + c < P ? vs[(size_t)t * ldv + c] : nst && t < nt && p0 + c == P ? 1.f : 0.f;
       }
     }
     const float* rs = rec + ((size_t)(t0 / C) * H + h) * kRecFloats;
@@ -372,6 +451,7 @@ __global__ void __launch_bounds__(320) lin_scan(const float* __restrict__ q, con
         s0 = fmaf(mm.z, Xw[(i + 2) * CW + c], s0); s1 = fmaf(mm.w, Xw[(i + 3) * CW + c], s1);
       }
       if (j < nt && cw + c < PB && p0 + cw + c < P) out[(size_t)(t0 + j) * ldo + (size_t)h * P + p0 + cw + c] = s0 + s1;
+      else if (nst && j < nt && cw + c < PB && p0 + cw + c == P) den[(size_t)(t0 + j) * H + h] = s0 + s1;
     }
     __syncwarp();
     const float ge = br[kRecEnd];
@@ -404,7 +484,10 @@ __global__ void __launch_bounds__(320) lin_scan(const float* __restrict__ q, con
     for (int i = 0; i < 4; i++) {
       const int n = 4 * (s + TPC * r) + i;
 #pragma unroll
-      for (int c = 0; c < CPT; c++) if (n < N && pc + c < P && cw + grp * CPT + c < PB) state[((size_t)h * N + n) * P + pc + c] = S[r][i][c];
+      for (int c = 0; c < CPT; c++) {
+        if (n < N && pc + c < P && cw + grp * CPT + c < PB) state[((size_t)h * N + n) * P + pc + c] = S[r][i][c];
+        if (nst && n < N && pc + c == P && cw + grp * CPT + c < PB) nst[(size_t)h * N + n] = S[r][i][c];
+      }
     }
 }
 inline size_t lin_scan_smem(int pitch, int PB, int warps, int cw) { return ((size_t)3 * (2 * kLinBlk * pitch + kLinBlk * PB + kRecFloats) + (size_t)warps * 4 * kLinBlk * cw) * 4; }
@@ -417,14 +500,19 @@ inline size_t lin_scan_smem(int pitch, int PB, int warps, int cw) { return ((siz
 // CTA of the step reads), silu, unit norms, step size and decay, head norm, output gate and factor are applied here:
 //   out[t][h P + p] = alpha rms(o)_p norm_w[p] silu(gate[t][h P + p]).
 // Plain form: q, k, v rows of proj (q_off, k and v behind it) as they are, decay[h]; out = o.
+// mLSTM: q, k, v likewise, raw gates in columns a_off (forget) and b_off (input), n and m carried in X; head norm with weights [H P], gate:
+//   out[t][h P + p] = rms(o)_p norm_w[h P + p] sigmoid(gate[t][h P + p]).
 // ---------------------------------------------------------------------------------------------------------------------
 constexpr int kLinDecodeThreads = 512;
-template <bool DELTA, int RN>
+enum { LIN_PLAIN = 0, LIN_DELTA = 1, LIN_MLSTM = 2 };
+struct MlstmP { float cap; float *n, *m; };   // n [H][N], m [H]
+template <int MODE, int RN>
 __global__ void __launch_bounds__(kLinDecodeThreads) lin_decode(const GdnP D, const float* __restrict__ decay, float* __restrict__ state,
                                                                 const float* __restrict__ norm_w, float eps, int gate_off, float alpha,
-                                                                float* __restrict__ out, int ldo) {
+                                                                float* __restrict__ out, int ldo, const MlstmP X) {
+  constexpr bool DELTA = MODE == LIN_DELTA, MLSTM = MODE == LIN_MLSTM;
   extern __shared__ __align__(16) float sm[];
-  __shared__ float red[33], gb[4];
+  __shared__ float red[33], gb[5];
   const int N = D.N, P = D.P, h = blockIdx.x, rep = D.H / D.G, g = h / rep, tid = threadIdx.x;
   const int PL = (P + 3) >> 2, NG = min(kLinDecodeThreads / PL, N), pl = tid % PL, ng = tid / PL;
   const bool on = ng < NG;
@@ -434,7 +522,12 @@ __global__ void __launch_bounds__(kLinDecodeThreads) lin_decode(const GdnP D, co
   float* so = sv + P;                // [P]
   float* part = so + P + ((4 - ((2 * N + 2 * P) & 3)) & 3);   // [2][NG][4 PL]
   float S[RN][4];
+  float* sn = part + 2 * (size_t)NG * 4 * PL;   // [N]  (mLSTM)
   const bool vec = (P & 3) == 0;
+  if (MLSTM) {
+    for (int n = tid; n < N; n += kLinDecodeThreads) sn[n] = X.n[(size_t)h * N + n];
+    if (tid == 0) gb[3] = X.m[h];
+  }
 #pragma unroll
   for (int r = 0; r < RN; r++) {
     const int n = ng + NG * r;
@@ -460,19 +553,23 @@ __global__ void __launch_bounds__(kLinDecodeThreads) lin_decode(const GdnP D, co
     }
     __syncthreads();
     const int lane = tid & 31, w = tid >> 5;
-    if (w < 3) {                     // sums of q^2, k^2 and q k
+    if (w < 3) {                     // sums of q^2 (mLSTM: n q), k^2 and q k
       float a = 0.f;
-      for (int n = lane; n < N; n += 32) { const float x = w == 1 ? sk[n] : sq[n], y = w == 0 ? sq[n] : sk[n]; a = fmaf(x, y, a); }
+      for (int n = lane; n < N; n += 32) { const float x = w == 1 ? sk[n] : sq[n], y = w == 0 ? (MLSTM ? sn[n] : sq[n]) : sk[n]; a = fmaf(x, y, a); }
       a = warp_sum(a);
       if (lane == 0) red[w] = a;
     } else if (w == 3 && lane == 0) {
       if (DELTA) { gb[0] = expf(gdn_log_decay(pr[D.a_off + h], D.A_log[h], D.dt_bias[h])); gb[1] = sigmoid_f(pr[D.b_off + h]); }
-      else { gb[0] = decay[h]; gb[1] = 1.f; }
+      else if (MLSTM) {
+        const float i = X.cap * tanhf(pr[D.b_off + h] / X.cap), f = log_sigmoid_f(X.cap * tanhf(pr[D.a_off + h] / X.cap)), m = fmaxf(f + gb[3], i);
+        gb[0] = expf(f + gb[3] - m); gb[1] = expf(i - m); gb[2] = expf(-m); gb[3] = m;
+      } else { gb[0] = decay[h]; gb[1] = 1.f; }
     }
     __syncthreads();
     // unit norms as factors on the dot products
-    const float fq = DELTA ? 1.f / (sqrtf(red[0] + 1e-6f) * sqrtf((float)N)) : 1.f, fk = DELTA ? 1.f / sqrtf(red[1] + 1e-6f) : 1.f, kq = red[2] * fq * fk;
+    const float fq = DELTA ? 1.f / (sqrtf(red[0] + 1e-6f) * sqrtf((float)N)) : MLSTM ? 1.f / sqrtf((float)N) : 1.f, fk = DELTA ? 1.f / sqrtf(red[1] + 1e-6f) : 1.f, kq = red[2] * fq * fk;
     const float gd = gb[0], beta = gb[1];
+    const float inv = MLSTM ? 1.f / (fmaxf(fabsf(fmaf(gd * fq, red[0], beta * kq)), gb[2]) + 1e-6f) : 1.f;
     float ak[4] = {0.f, 0.f, 0.f, 0.f}, aq[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
     for (int r = 0; r < RN; r++) {
@@ -495,8 +592,8 @@ __global__ void __launch_bounds__(kLinDecodeThreads) lin_decode(const GdnP D, co
         if (DELTA) rk += part[(size_t)i * 4 * PL + p];
         rq += part[(size_t)(NG + i) * 4 * PL + p];
       }
-      const float u = DELTA ? beta * fmaf(-gd * fk, rk, sv[p]) : sv[p];
-      so[p] = fmaf(gd * fq, rq, kq * u);
+      const float u = DELTA ? beta * fmaf(-gd * fk, rk, sv[p]) : MLSTM ? beta * sv[p] : sv[p];
+      so[p] = fmaf(gd * fq, rq, kq * u) * inv;
       sv[p] = u * fk;                 // the update below multiplies the unscaled k
     }
     __syncthreads();
@@ -512,14 +609,22 @@ __global__ void __launch_bounds__(kLinDecodeThreads) lin_decode(const GdnP D, co
         for (int c = 0; c < 4; c++) S[r][c] = fmaf(x, uu[c], gd * S[r][c]);
       }
     }
-    if (DELTA) {
+    if (MLSTM) for (int n = tid; n < N; n += kLinDecodeThreads) sn[n] = fmaf(beta, sk[n], gd * sn[n]);
+    if (DELTA || MLSTM) {
       float ss = 0.f;
       for (int p = tid; p < P; p += kLinDecodeThreads) ss = fmaf(so[p], so[p], ss);
       const float sc = alpha / sqrtf(block_sum(ss, red) / (float)P + eps);
-      for (int p = tid; p < P; p += kLinDecodeThreads) out[(size_t)t * ldo + (size_t)h * P + p] = so[p] * sc * norm_w[p] * silu_f(pr[gate_off + h * P + p]);
+      for (int p = tid; p < P; p += kLinDecodeThreads) {
+        const float gt = pr[gate_off + h * P + p];
+        out[(size_t)t * ldo + (size_t)h * P + p] = MLSTM ? so[p] * sc * norm_w[(size_t)h * P + p] * sigmoid_f(gt) : so[p] * sc * norm_w[p] * silu_f(gt);
+      }
     } else
       for (int p = tid; p < P; p += kLinDecodeThreads) out[(size_t)t * ldo + (size_t)h * P + p] = so[p];
     __syncthreads();
+  }
+  if (MLSTM) {
+    for (int n = tid; n < N; n += kLinDecodeThreads) X.n[(size_t)h * N + n] = sn[n];
+    if (tid == 0) X.m[h] = gb[3];
   }
 #pragma unroll
   for (int r = 0; r < RN; r++) {
@@ -534,7 +639,7 @@ __global__ void __launch_bounds__(kLinDecodeThreads) lin_decode(const GdnP D, co
 }
 inline size_t lin_decode_smem(int N, int P) {
   const int PL = (P + 3) / 4, NG = kLinDecodeThreads / PL < N ? kLinDecodeThreads / PL : N;
-  return ((size_t)2 * N + 2 * P + 4 + (size_t)2 * NG * 4 * PL) * 4;
+  return ((size_t)3 * N + 2 * P + 4 + (size_t)2 * NG * 4 * PL) * 4;
 }
 
 }  // namespace hy

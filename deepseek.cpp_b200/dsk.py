@@ -23,18 +23,19 @@ sys.path.insert(0, HERE)
 import dseek  # noqa: E402
 
 QUANT_IDS = {"fp32": 0, "fp16": 1, "f8e5m2": 2, "q2_k": 3, "q3_k": 4, "bf16": 5}
-MIX_SSD, MIX_LATENT_SWA, MIX_GQA, MIX_MLA, MIX_HGRN2, MIX_GDN, MIX_LIGHTNING = 0, 1, 2, 3, 4, 5, 6
+MIX_SSD, MIX_LATENT_SWA, MIX_GQA, MIX_MLA, MIX_HGRN2, MIX_GDN, MIX_LIGHTNING, MIX_MLSTM = 0, 1, 2, 3, 4, 5, 6, 7
 FF_NONE, FF_MOE, FF_DENSE = 0, 1, 2
 MASK_WINDOW, MASK_CHUNK = 0, 1
-ACT_XIELU, ACT_GEGLU, ACT_GLU_CLAMPED = 0, 1, 2
+ACT_XIELU, ACT_GEGLU, ACT_GLU_CLAMPED, ACT_SWIGLU = 0, 1, 2, 3
 BLOCK_PARALLEL, BLOCK_SANDWICH, BLOCK_POST, BLOCK_PRE = 0, 1, 2, 3
 NORM_RMS, NORM_LAYER = 0, 1
 ROT_PAIRS, ROT_HALF = 0, 1
 ROTSCALE_YARN, ROTSCALE_BANDS = 0, 1
 QKNORM_WHOLE, QKNORM_HEAD, QKNORM_HEAD_WEIGHT = 0, 1, 2
 GATE_NONE, GATE_ENTRY, GATE_HEAD = 0, 1, 2
-ROUTER_SIGMOID, ROUTER_TOP_SOFTMAX = 0, 1
-EXPERT_GLU_CLAMPED, EXPERT_RELU2 = 0, 1
+ROUTER_SIGMOID, ROUTER_TOP_SOFTMAX, ROUTER_SOFTMAX_GROUPS = 0, 1, 2
+EXPERT_GLU_CLAMPED, EXPERT_RELU2, EXPERT_SWIGLU = 0, 1, 2
+SINK_NONE, SINK_HEAD, SINK_ONE = 0, 1, 2
 HYDRATE_KV_CACHE, OUTPUT_LOGITS = 0, 1
 
 f32p = C.POINTER(C.c_float)
@@ -106,7 +107,8 @@ class LayerSpec(C.Structure):
                [(n, C.c_int) for n in ("att_q_rank", "att_rot_dim", "att_out_gate", "rot_layout", "rot_scale", "att_qk_norm",
                                        "lin_heads", "lin_dim", "lin_vdim", "ff_router", "ff_expert", "mixer2")] + \
                [("mix_scale", C.c_float), ("mix2_scale", C.c_float)] + \
-               [(n, C.c_int) for n in ("gdn_heads", "gdn_kv_heads", "gdn_dim", "gdn_vdim", "gdn_conv")] + [("lin_decay", f32p)]
+               [(n, C.c_int) for n in ("gdn_heads", "gdn_kv_heads", "gdn_dim", "gdn_vdim", "gdn_conv")] + [("lin_decay", f32p), ("lin_gate_cap", C.c_float)] + \
+               [(n, C.c_int) for n in ("att_conv", "ff_groups", "ff_groups_keep", "ff_shared")]
 
 
 class HybridConfig(C.Structure):
@@ -117,7 +119,7 @@ class HybridConfig(C.Structure):
                [(n, C.c_int) for n in ("block", "norm_kind", "tie_head", "loop_start", "loop_stop", "loop_times")] + \
                [("embed_scale", C.c_float)] + \
                [(n, C.c_int) for n in ("bigram_buckets", "bigram_mul_prev", "bigram_mul_cur", "norm_scalar", "canon_taps", "res_gate", "layer_scale",
-                                       "norm_bias", "token_shift", "norm_one_plus", "loop_embed")] + [("logit_softcap", C.c_float)]
+                                       "norm_bias", "token_shift", "norm_one_plus", "loop_embed")] + [("logit_softcap", C.c_float), ("loop_in", C.c_int)]
 
 
 # mixer "type" strings of a layer-list config.json -> mixer kernel family.  Two names may map to one mechanism.
@@ -392,12 +394,78 @@ def zetivik_from_config(cfg: dict, quant: str = "bf16", max_seq_len: int = 0, ch
     return hc, specs
 
 
+def netusun_from_config(cfg: dict, quant: str = "bf16", max_seq_len: int = 0, chunk: int = 256):
+    """config.json of the Netusun design -> (HybridConfig, LayerSpec array): sandwich blocks of RMS norms with layer scales, a layer
+    loop whose passes open with a product over [stream; embedding], a tied head, and per layer grouped-query attention behind short
+    convolutions (weighted per-head query / key norm, score cap, window, a one in the softmax denominator), latent attention
+    (half-split rotation with YaRN scaling, a learned sink per head, output gate) or the mLSTM matrix memory; gated dense or routed
+    feed-forwards (softmax router over expert groups, shared expert).  Absent keys switch a part off."""
+    hc = HybridConfig()
+    layers = cfg["layers"]
+    hc.dim, hc.vocab_size, hc.n_layers = int(cfg["width"]), int(cfg["vocab"]), len(layers)
+    hc.quant, hc.chunk = QUANT_IDS[quant], int(chunk)
+    hc.max_seq_len = int(max_seq_len) if max_seq_len else 1 << 30
+    hc.norm_eps, hc.norm_groups = float(cfg["norm"]["eps"]), 1
+    hc.residual_mult, hc.logit_scale, hc.side_dim = 1.0, 1.0, 0
+    hc.block, hc.norm_kind, hc.tie_head, hc.layer_scale = BLOCK_SANDWICH, NORM_RMS, 1, 1
+    loop = cfg.get("loop")
+    if loop:            # a loop of one pass is still a loop: it opens with its product and vector
+        hc.loop_start, hc.loop_stop, hc.loop_times, hc.loop_in = int(loop["start"]), int(loop["stop"]), int(loop["times"]), 1
+    specs = (LayerSpec * len(layers))()
+    for i, lc in enumerate(layers):
+        sp, mx = specs[i], lc["mixer"]
+        sp.att_kv_from = -1
+        if lc["type"] == "attention":
+            sp.mixer = MIX_GQA
+            sp.att_heads, sp.att_kv_heads = int(mx["heads"]), int(mx.get("kv_heads") or mx["heads"])
+            sp.att_dim, sp.att_vdim, sp.att_scale = int(mx["dim"]), int(mx["vdim"]), float(mx["scale"])
+            mask = mx.get("mask") or {}
+            sp.att_mask = MASK_WINDOW
+            sp.att_window = int(mask["size"]) if mask.get("size") is not None else 1 << 30      # no window: every earlier token is visible
+            sp.att_value_proj, sp.att_qk_norm, sp.att_sink = 1, QKNORM_HEAD_WEIGHT, SINK_ONE
+            sp.att_softcap, sp.att_conv = float(mx.get("softcap") or 0.0), int(mx.get("conv") or 0)
+        elif lc["type"] == "latent_attention":
+            sp.mixer, sp.att_mask, sp.att_window = MIX_MLA, MASK_WINDOW, 1 << 30
+            sp.att_heads, sp.att_dim, sp.att_vdim, sp.att_scale = int(mx["heads"]), int(mx["dim"]), int(mx["vdim"]), float(mx["scale"])
+            sp.att_kv_rank, sp.att_q_rank, sp.att_rot_dim = int(mx["kv_rank"]), int(mx["q_rank"]), int(mx["rot_dim"])
+            sp.att_out_gate, sp.att_sink = GATE_ENTRY, SINK_HEAD
+            rot = mx.get("rot") or {}
+            sp.rot_dims, sp.rot_base, sp.rot_layout = int(rot.get("dims", 0)), float(rot.get("base", 10000.0)), ROT_HALF
+            sc = rot.get("scaling")
+            if sc:
+                sp.rot_scale, sp.rot_factor, sp.rot_original = ROTSCALE_YARN, float(sc["factor"]), int(sc["original"])
+                sp.rot_fast, sp.rot_slow = float(sc["fast"]), float(sc["slow"])
+                if not sp.rot_factor > 0:
+                    raise DskError(f"layer {i}: rotation scaling factor must be positive")
+        elif lc["type"] == "mlstm":
+            sp.mixer = MIX_MLSTM
+            sp.lin_heads, sp.lin_dim, sp.lin_vdim, sp.lin_gate_cap = int(mx["heads"]), int(mx["dim"]), int(mx["vdim"]), float(mx["gate_cap"])
+        else:
+            raise DskError(f"layer {i}: unknown mixer type {lc['type']!r}")
+        ff = lc.get("mlp")
+        if not ff:
+            sp.ff_kind = FF_NONE
+        elif ff.get("kind") == "dense":
+            sp.ff_kind, sp.ff_hidden, sp.ff_act = FF_DENSE, int(ff["ff"]), ACT_SWIGLU
+        elif ff.get("kind") == "moe":
+            r = ff["router"]
+            sp.ff_kind, sp.ff_router, sp.ff_expert = FF_MOE, ROUTER_SOFTMAX_GROUPS, EXPERT_SWIGLU
+            sp.ff_experts, sp.ff_top, sp.ff_hidden, sp.ff_router_scale = int(r["experts"]), int(r["top"]), int(ff["expert"]["ff"]), float(r.get("scale", 1.0))
+            gr = r.get("groups")
+            if gr:
+                sp.ff_groups, sp.ff_groups_keep = int(gr["count"]), int(gr["keep"])
+            sp.ff_shared = int((ff.get("shared") or {}).get("ff", 0))
+        else:
+            raise DskError(f"layer {i}: unknown feed-forward kind {ff.get('kind')!r}")
+    return hc, specs
+
+
 # config.json "architecture" -> builder of the C-ABI model description (the DeepSeek families come as .dseek metadata instead)
 ARCHITECTURES = {"Desarax": hybrid_from_config, "Rutulix": rutulix_from_config, "Sakusun": sakusun_from_config, "Nalizen": nalizen_from_config,
-                 "Zetivik": zetivik_from_config}
+                 "Zetivik": zetivik_from_config, "Netusun": netusun_from_config}
 
 _lib = None
-ABI_VERSION = 8   # DSK_ABI_VERSION (include/dsk.h)
+ABI_VERSION = 9   # DSK_ABI_VERSION (include/dsk.h)
 
 
 def build(force: bool = False) -> str:

@@ -20,7 +20,7 @@
 extern "C" {
 #endif
 
-#define DSK_ABI_VERSION 8
+#define DSK_ABI_VERSION 9
 
 /* Quant: src/codec.h:79-85 (same numbering) */
 enum { DSK_F32 = 0, DSK_F16 = 1, DSK_F8E5M2 = 2, DSK_Q2_K = 3, DSK_Q3_K = 4,
@@ -74,14 +74,19 @@ typedef struct dsk_config {
  * or DSK_ROUTER_TOP_SOFTMAX / DSK_EXPERT_RELU2 routed feed-forwards, a scaled and tied embedding and the per-layer token input; the
  * Zetivik design is DSK_BLOCK_PRE with RMS norms whose weight is stored around zero, layers of two mixers side by side (DSK_MIX_GQA
  * with half-split rotation, weighted per-head query / key norm, one output gate per head and a chunk mask, beside DSK_MIX_GDN) or of
- * DSK_MIX_LIGHTNING, clamped dense feed-forwards, a layer loop that adds the embedding again, a tied head and a logit cap.) */
+ * DSK_MIX_LIGHTNING, clamped dense feed-forwards, a layer loop that adds the embedding again, a tied head and a logit cap; the
+ * Netusun design is DSK_BLOCK_SANDWICH with RMS norms and layer scales, DSK_MIX_GQA mixers (short convolutions, weighted per-head
+ * query / key norm, score cap, window, DSK_SINK_ONE), DSK_MIX_MLA mixers (half-split rotation with YaRN scaling, DSK_SINK_HEAD, output
+ * gate) or DSK_MIX_MLSTM mixers, dense or DSK_ROUTER_SOFTMAX_GROUPS / DSK_EXPERT_SWIGLU feed-forwards with a shared expert, a layer
+ * loop whose passes open with a product over [stream; embedding], and a tied head.) */
 enum { DSK_MIX_SSD = 0, DSK_MIX_LATENT_SWA = 1, DSK_MIX_GQA = 2, DSK_MIX_MLA = 3, DSK_MIX_HGRN2 = 4,
-       DSK_MIX_GDN = 5, DSK_MIX_LIGHTNING = 6 };
+       DSK_MIX_GDN = 5, DSK_MIX_LIGHTNING = 6, DSK_MIX_MLSTM = 7 };
 enum { DSK_FF_NONE = 0, DSK_FF_MOE = 1, DSK_FF_DENSE = 2 };
 enum { DSK_MASK_WINDOW = 0,   /* position i sees j with 0 <= i - j < att_window */
        DSK_MASK_CHUNK = 1 };  /* position i sees j <= i with floor(i / att_window) == floor(j / att_window): borders at multiples of att_window in sequence positions */
 enum { DSK_ACT_XIELU = 0,      /* z > 0: softplus(p) z^2 + z/2;  z <= 0: (1/2 + softplus(q)) (e^z - 1 - z) + z/2;  (p, q) = tensor mlp.act */
        DSK_ACT_GEGLU = 1,      /* gated: down(gelu_tanh(gate h) * (up h)), tensors mlp.gate / mlp.up / mlp.down, no biases */
+       DSK_ACT_SWIGLU = 3,     /* gated: down(silu(gate h) * (up h)), the same tensors */
        DSK_ACT_GLU_CLAMPED = 2 };   /* gated: down(g sigmoid(1.702 g) (u + 1)), g = min(gate h, ff_limit), u = clamp(up h, +-ff_limit), the same tensors */
 enum { DSK_BLOCK_PARALLEL = 0,   /* h = norm1(x); x += residual_mult (mixer(h) + ff(h)) */
        DSK_BLOCK_SANDWICH = 1,   /* x += norm1b(mixer(norm1(x))); x += norm2b(ff(norm2(x))) */
@@ -102,21 +107,26 @@ enum { DSK_QKNORM_WHOLE = 0,     /* RMS norm with weights mix.q.norm / mix.k.nor
 enum { DSK_GATE_NONE = 0, DSK_GATE_ENTRY = 1,   /* att_out_gate: heads multiplied by sigmoid(g h), one number per entry of the concatenated heads (mix.g [heads * vdim]) */
        DSK_GATE_HEAD = 2 };      /* one number per head (mix.g [heads]); DSK_MIX_GQA */
 enum { DSK_ROUTER_SIGMOID = 0,   /* sigmoid scores, selection by score + mlp.correction, weights = chosen scores normalised x ff_router_scale */
-       DSK_ROUTER_TOP_SOFTMAX = 1 };   /* logits = router h + mlp.router.b; the ff_top largest logits; weights = softmax over the chosen logits */
+       DSK_ROUTER_TOP_SOFTMAX = 1,     /* logits = router h + mlp.router.b; the ff_top largest logits; weights = softmax over the chosen logits */
+       DSK_ROUTER_SOFTMAX_GROUPS = 2 };   /* s = softmax(router h) over all experts; ff_groups equal groups of neighbours, those of the ff_groups_keep
+                                             groups with the largest best score stay; the ff_top largest of them; weights = s x ff_router_scale */
+enum { DSK_SINK_NONE = 0, DSK_SINK_HEAD = 1,   /* att_sink: e^sink joins the softmax denominator, one number per head (mix.sink [heads]) */
+       DSK_SINK_ONE = 2 };             /* one joins it (a sink of score 0, no tensor) */
 enum { DSK_EXPERT_GLU_CLAMPED = 0,     /* down(g sigmoid(1.702 g) (u + 1)), g = min(gate h, limit), u = clamp(up h, +-limit) */
-       DSK_EXPERT_RELU2 = 1 };         /* down(max(up h, 0)^2), no gate matrix */
+       DSK_EXPERT_RELU2 = 1,           /* down(max(up h, 0)^2), no gate matrix */
+       DSK_EXPERT_SWIGLU = 2 };        /* down(silu(gate h) * (up h)) */
 /* DSK_MIX_GQA also has these switches (all off in the Rutulix design): att_value_proj (values = v matrix mix.v of att_vdim per
  * key head instead of the raw key projection), att_bias (biases mix.q.b / k.b / v.b added in the projections), att_softcap > 0
  * (score <- cap tanh(score / cap) after the scale), att_rel_max > 0 (a learned bias per distance bucket and head added after
  * the cap: tensor mix.rel [B][heads], bucket(n) = n below B/2, else min(B - 1, B/2 + floor(ln(n / (B/2)) / ln(att_rel_max / (B/2))
  * (B - B/2)))), att_keep_first (DSK_MASK_WINDOW only: the first positions of a sequence stay visible beyond the window, at their
- * true distance), att_sink (tensor mix.sink [heads]: e^sink joins the softmax denominator, with no key and no value), att_vmix (the
+ * true distance), att_sink (DSK_SINK_*: an extra term of the softmax denominator, with no key and no value), att_vmix (the
  * first such layer's values v1 of a token are kept for the step; every later such layer caches (1 - l) v + l v1, l = tensor mix.vmix).
  *   DSK_MIX_MLA         softmax attention over cached latents with a query latent and a rotated key part: c_q = rms(dq h) dq.norm,
  *                       q = uq c_q laid out per head as [att_dim plain | att_rot_dim rotated]; dkv h = [att_kv_rank latent, RMS-normed
  *                       with dkv.norm | att_rot_dim rotated key part shared by all heads]; per head key = uk c, value = uv c; score =
- *                       att_scale (q_plain . k + q_rot . k_rot); rotation of the pairs (2i, 2i + 1) of the first rot_dims entries of the
- *                       rotated part by pos * rot_base^(-2i / rot_dims); mask att_mask of size att_window; with att_out_gate the
+ *                       att_scale (q_plain . k + q_rot . k_rot); rotation (rot_layout) of the first rot_dims entries of the
+ *                       rotated part by pos * rot_base^(-2i / rot_dims), YaRN-scaled when rot_factor > 0; att_sink as in DSK_MIX_GQA; mask att_mask of size att_window; with att_out_gate the
  *                       concatenated heads are multiplied by sigmoid(g h) before the output projection.  Caches [latent | rotated key].
  *   DSK_MIX_GQA         softmax attention with att_heads query heads over att_kv_heads cached key heads (query head h reads key head
  *                       h / (att_heads / att_kv_heads)); a position's value vector is the raw output of its key matrix, taken ahead of the key norm and the rotation (no value matrix:
@@ -143,6 +153,15 @@ enum { DSK_EXPERT_GLU_CLAMPED = 0,     /* down(g sigmoid(1.702 g) (u + 1)), g = 
  *   DSK_MIX_LIGHTNING   linear attention with a fixed decay per head: q, k = silu(.) [lin_heads][lin_dim], v = silu(.) [lin_heads][lin_vdim];
  *                       S <- lin_decay[h] S + k v^T, o = S^T q; RMS norm with mix.norm over the concatenated heads, times sigmoid(mix.g h),
  *                       output projection mix.o.  Carries S in fp32.
+ *   DSK_MIX_MLSTM       matrix memory with exponential gates: q = mix.q h / sqrt(lin_dim), k = mix.k h [lin_heads][lin_dim], v = mix.v h [lin_heads][lin_vdim];
+ *                       per head, with cap = lin_gate_cap: i = cap tanh((mix.i h + mix.i.b) / cap), f = log sigmoid(cap tanh((mix.f h + mix.f.b) / cap)),
+ *                       m' = max(f + m, i) (m starts at 0); S <- e^(f + m - m') S + e^(i - m') k v^T, n likewise with k alone;
+ *                       o = S^T q / (max(|n . q|, e^-m') + 1e-6); every head's o divided by its RMS, times mix.norm [lin_heads * lin_vdim], times
+ *                       sigmoid(mix.g h); output projection mix.o.  Carries S, n and m in fp32.
+ *   att_conv > 0 (DSK_MIX_GQA with att_value_proj): the projected q, k and v rows first go through a causal per-channel convolution of att_conv taps
+ *                       (mix.q.conv / k.conv / v.conv [channels][taps], last tap on the current token, no bias, no activation).  Carries the last inputs.
+ *   ff_shared > 0 (DSK_FF_MOE): a shared expert of that hidden size (mlp.shared.*, the experts' form) runs for every token, its output times
+ *                       sigmoid(mlp.shared.sg h) is added.
  *   mixer2 = DSK_MIX_GDN runs beside a DSK_MIX_GQA mixer on the same input: x += residual_mult (mix_scale left + mix2_scale right), tensors
  *                       mix.left.* and mix.right.*.
  *   DSK_FF_DENSE        down(act(up h + b_up)) + b_down with activation ff_act. */
@@ -161,14 +180,17 @@ typedef struct dsk_layer_spec {
   int ff_act;                                                           /* DSK_FF_DENSE: DSK_ACT_*, hidden size ff_hidden */
   int att_value_proj, att_bias, att_keep_first, att_rel_max, att_sink, att_vmix;   /* DSK_MIX_GQA switches (above) */
   float att_softcap;
-  int att_q_rank, att_rot_dim, att_out_gate;                            /* DSK_MIX_MLA (with att_heads, att_dim, att_vdim, att_kv_rank, att_scale, att_mask, att_window, rot_dims, rot_base) */
+  int att_q_rank, att_rot_dim, att_out_gate;                            /* DSK_MIX_MLA (with att_heads, att_dim, att_vdim, att_kv_rank, att_scale, att_mask, att_window, att_sink, rot_*) */
   int rot_layout, rot_scale, att_qk_norm;                               /* DSK_MIX_GQA: DSK_ROT_*, DSK_ROTSCALE_*, DSK_QKNORM_* */
-  int lin_heads, lin_dim, lin_vdim;                                     /* DSK_MIX_HGRN2 */
+  int lin_heads, lin_dim, lin_vdim;                                     /* DSK_MIX_HGRN2, DSK_MIX_LIGHTNING, DSK_MIX_MLSTM */
   int ff_router, ff_expert;                                             /* DSK_FF_MOE: DSK_ROUTER_*, DSK_EXPERT_* */
   int mixer2;                                                           /* 0: one mixer; DSK_MIX_GDN: a second one beside it (above) */
   float mix_scale, mix2_scale;
   int gdn_heads, gdn_kv_heads, gdn_dim, gdn_vdim, gdn_conv;             /* DSK_MIX_GDN */
   const float* lin_decay;                                               /* DSK_MIX_LIGHTNING (with lin_heads, lin_dim, lin_vdim): lin_heads decays, read by dsk_model_create_hybrid */
+  float lin_gate_cap;                                                   /* DSK_MIX_MLSTM (with lin_heads, lin_dim, lin_vdim) */
+  int att_conv;                                                         /* DSK_MIX_GQA: taps of the convolutions behind the projections, 0: none */
+  int ff_groups, ff_groups_keep, ff_shared;                             /* DSK_FF_MOE: expert groups (0 reads as one group), hidden size of the shared expert (0: none) */
 } dsk_layer_spec;
 typedef struct dsk_hybrid_config {
   int dim, vocab_size, n_layers;
@@ -189,7 +211,7 @@ typedef struct dsk_hybrid_config {
   int bigram_buckets, bigram_mul_prev, bigram_mul_cur;   /* > 0 buckets: row (prev * mul_prev + token * mul_cur) mod buckets of tensor "bigram"
                                               [buckets + 1][dim] is added to the embedding; a sequence's first token takes the last row */
   int norm_scalar;           /* 1: the weights of the norms outside the mixers (norm1, norm2, final.norm) are single numbers */
-  int canon_taps, res_gate, layer_scale;   /* DSK_BLOCK_POST: taps of the causal per-channel input convolution (tensors canon1 / canon2 [dim][taps], last tap on
+  int canon_taps, res_gate, layer_scale;   /* DSK_BLOCK_POST (layer_scale: also DSK_BLOCK_SANDWICH): taps of the causal per-channel input convolution (tensors canon1 / canon2 [dim][taps], last tap on
                                               the current token; 0: none), gated sublayer results (rg1 / rg2 [dim][dim] + .b), per-channel scale after the norm (ls1 / ls2) */
   int norm_bias;             /* DSK_NORM_LAYER: every norm outside the mixers adds a bias, tensor "<norm>.b" */
   int token_shift;           /* 1: a mixer reads h + (h' - h) * shift (tensor l<i>.shift [dim]) instead of its input h, h' being the previous token's h
@@ -197,6 +219,7 @@ typedef struct dsk_hybrid_config {
   int norm_one_plus;         /* 1: the norms outside the mixers multiply by 1 + their stored weight */
   int loop_embed;            /* 1: ahead of every loop pass but the first, the embedding output is added to the residual stream */
   float logit_softcap;       /* > 0: logits <- cap tanh(logits / cap) */
+  int loop_in;               /* 1: every loop pass opens with x <- loop.in [x; embedding output] (tensor [dim][2 dim]) ahead of its loop.step row */
 } dsk_hybrid_config;
 
 typedef struct dsk_model dsk_model;
