@@ -11,6 +11,7 @@
 //                     epilogues (residual add, clamped GLU, GELU x per-token embedding) and row gather / scatter / expert tiles
 //   gemm_mma          the same interface on the tensor cores for bf16 weights (activations rounded to bf16 as they are staged)
 //   gemv_rows         the same interface for T <= 4 rows: one warp per weight row, 16-byte loads
+//   gemv_one          the same for one row (a decoded token): eight 16-byte weight loads in flight per lane
 //   causal_conv_silu  depthwise causal convolution over the chunk continuing from the carried (taps - 1) inputs, + SiLU
 //   ssd_scan          the state-space recurrence S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x, gated by silu(z)
 //   latent_swa_attn   softmax attention over a sliding window of cached latents with absorbed key up-projection
@@ -690,16 +691,24 @@ template <typename WT> struct WVec;
 template <> struct WVec<float> {
   static constexpr int N = 4;
   static __device__ __forceinline__ void load(const float* p, float (&o)[4]) { const float4 v = *reinterpret_cast<const float4*>(p); o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w; }
+  static __device__ __forceinline__ void decode(const uint4& v, float (&o)[4]) { o[0] = __uint_as_float(v.x); o[1] = __uint_as_float(v.y); o[2] = __uint_as_float(v.z); o[3] = __uint_as_float(v.w); }
 };
 template <> struct WVec<__nv_bfloat16> {
   static constexpr int N = 8;
   static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&o)[8]) {
-    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    decode(*reinterpret_cast<const uint4*>(p), o);
+  }
+  static __device__ __forceinline__ void decode(const uint4& v, float (&o)[8]) {
     const uint32_t w[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
     for (int i = 0; i < 4; i++) { o[2 * i] = __uint_as_float(w[i] << 16); o[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
   }
 };
+__device__ __forceinline__ uint4 ldg_stream(const void* p) {   // 16 read-only bytes that are used once
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
 
 // M <= 4 rows: one warp per weight row, lanes stride over K with 16-byte loads when pitches and bases allow it.
 template <typename WT, int EPI>
@@ -794,6 +803,94 @@ __global__ void __launch_bounds__(256) gemv_rows(const GemmP P) {
       }
     }
   }
+}
+
+// One activation row per batch (a decoded token, or a routed (token, slot) pair): the product is a stream of weights, so a warp takes R
+// rows of the matrix at a time and has eight 16-byte loads per lane in flight before the first multiplication; the weights bypass L1,
+// which holds the activation row.  Needs what gemv_rows calls `vec` (gemv_one_ok).
+template <typename WT, int EPI, int R>
+__global__ void __launch_bounds__(256) gemv_one(const GemmP P) {
+  constexpr bool DUAL = epi_dual(EPI);
+  constexpr int V = WVec<WT>::N, NM = DUAL ? 2 : 1, U = 8 / (R * NM);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, z = blockIdx.y;
+  int N = P.N, K = P.K, ldw = P.ldw, cr = 0;
+  const WT *W, *W2 = nullptr;
+  const float* A;
+  float* C;
+  if (P.z_expert && P.n_shared > 0 && z >= P.z_shared) {
+    N = P.sN; K = P.sK; ldw = P.sK;
+    W = reinterpret_cast<const WT*>(P.sW1); W2 = reinterpret_cast<const WT*>(P.sW2);
+    A = P.As + (size_t)(z - P.z_shared) * P.s_lda;
+    C = P.Cs + (size_t)(z - P.z_shared) * P.s_ldc;
+  } else {
+    const long long woff = P.z_expert ? (long long)P.z_expert[z] * P.sW : (long long)(z / P.z_wdiv) * P.sW;
+    W = reinterpret_cast<const WT*>(P.W) + woff;
+    if (DUAL) W2 = reinterpret_cast<const WT*>(P.W2) + woff;
+    if (P.z_expert) {
+      A = P.A + (size_t)(z / P.z_adiv) * P.lda;
+      C = P.C + (size_t)z * P.ldc;
+    } else {
+      cr = P.c_map ? P.c_map[0] : 0;
+      A = P.A + (long long)z * P.sA + (size_t)(P.a_map ? P.a_map[0] / P.a_div : 0) * P.lda;
+      C = P.C + (long long)z * P.sC + (size_t)cr * P.ldc;
+    }
+  }
+  for (int n0 = (blockIdx.x * 8 + warp) * R; n0 < N; n0 += gridDim.x * 8 * R) {
+    const WT* w[R][NM];
+    float acc[R][NM];
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+      const size_t row = (size_t)min(n0 + r, N - 1) * ldw;
+      w[r][0] = W + row;
+      if (DUAL) w[r][NM - 1] = W2 + row;
+#pragma unroll
+      for (int m = 0; m < NM; m++) acc[r][m] = 0.f;
+    }
+    for (int k0 = lane * V; k0 < K; k0 += 32 * V * U) {
+      uint4 raw[U][R][NM];
+#pragma unroll
+      for (int u = 0; u < U; u++)
+#pragma unroll
+        for (int r = 0; r < R; r++)
+#pragma unroll
+          for (int m = 0; m < NM; m++) raw[u][r][m] = k0 + u * 32 * V < K ? ldg_stream(w[r][m] + k0 + u * 32 * V) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+      for (int u = 0; u < U; u++) {
+        const int k = k0 + u * 32 * V;
+        if (k < K) {
+          float a[V];
+#pragma unroll
+          for (int q = 0; q < V; q += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(A + k + q);
+            a[q] = v.x; a[q + 1] = v.y; a[q + 2] = v.z; a[q + 3] = v.w;
+          }
+#pragma unroll
+          for (int r = 0; r < R; r++)
+#pragma unroll
+            for (int m = 0; m < NM; m++) {
+              float wv[V];
+              WVec<WT>::decode(raw[u][r][m], wv);
+#pragma unroll
+              for (int q = 0; q < V; q++) acc[r][m] = fmaf(a[q], wv[q], acc[r][m]);
+            }
+        }
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < R; r++) {
+      const float v = warp_sum(acc[r][0]);
+      const float v2 = DUAL ? warp_sum(acc[r][NM - 1]) : 0.f;
+      if (lane == 0 && n0 + r < N) gemm_epilogue<WT, EPI>(P, C, cr, n0 + r, v, v2);
+    }
+  }
+}
+// whether gemv_one's 16-byte loads are aligned for every batch
+template <typename WT>
+inline bool gemv_one_ok(const GemmP& P) {
+  constexpr int V = WVec<WT>::N;
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (P.z_rows > 0 || (!P.z_expert && P.M != 1) || P.K % V || P.ldw % V || P.lda % 4 || P.sW % V || P.sA % 4 || !al(P.A) || !al(P.W) || (P.W2 && !al(P.W2))) return false;
+  return P.n_shared <= 0 || (P.sK % V == 0 && P.s_lda % 4 == 0 && al(P.As) && al(P.sW1) && (!P.sW2 || al(P.sW2)));
 }
 
 // ---------------------------------------------------------------------------------------------------------------------
@@ -1215,22 +1312,23 @@ __global__ void __launch_bounds__(256) latent_swa_attn(const float* __restrict__
 __global__ void __launch_bounds__(128) latent_swa_merge(const float* __restrict__ part, float* __restrict__ out, int R, int NS,
                                                         const float* __restrict__ gate = nullptr, int ld_gate = 0, int H = 1,
                                                         int gate_head = 0, int ld_out = 0, float alpha = 1.f) {
-  __shared__ float wts[64], ms[64];   // NS <= 64 (kAttnSplitMax)
+  __shared__ float wts[64], ms[64], ls[64];   // NS <= 64 (kAttnSplitMax)
   const size_t th = blockIdx.x;
   const float* pp = part + th * NS * (R + 2);
-  if ((int)threadIdx.x < NS) ms[threadIdx.x] = pp[(size_t)threadIdx.x * (R + 2)];
+  if ((int)threadIdx.x < NS) { ms[threadIdx.x] = pp[(size_t)threadIdx.x * (R + 2)]; ls[threadIdx.x] = pp[(size_t)threadIdx.x * (R + 2) + 1]; }
   __syncthreads();
   float m = -1e30f;
   for (int s = 0; s < NS; s++) m = fmaxf(m, ms[s]);
   if ((int)threadIdx.x < NS) wts[threadIdx.x] = expf(ms[threadIdx.x] - m);
   __syncthreads();
   float l = 0.f;
-  for (int s = 0; s < NS; s++) l = fmaf(wts[s], pp[(size_t)s * (R + 2) + 1], l);
+  for (int s = 0; s < NS; s++) l = fmaf(wts[s], ls[s], l);
   const float inv = 1.f / l;
   const int r = blockIdx.y * 128 + threadIdx.x;
   if (r >= R) return;
   float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
   int s = 0;
+#pragma unroll 4
   for (; s + 4 <= NS; s += 4) {
     const float v0 = pp[(size_t)s * (R + 2) + 2 + r], v1 = pp[(size_t)(s + 1) * (R + 2) + 2 + r];
     const float v2 = pp[(size_t)(s + 2) * (R + 2) + 2 + r], v3 = pp[(size_t)(s + 3) * (R + 2) + 2 + r];
@@ -1429,45 +1527,56 @@ __global__ void __launch_bounds__(256) rms_open(float* __restrict__ x, const flo
 //   x' = x + alpha rms(y) wy  -> xo (row pitch ldxo; the stream itself, or the input rows of the product that opens a loop pass);
 //   h = rms(x') wh            (wh nullable: no norm follows here).
 // wgt non-null: y_t = sum_k wgt[t][k] y[t * top + k] (+ wsh[t] ysh[t], nullable): routed experts' outputs and the shared one's.
-__global__ void __launch_bounds__(256) rms_add_norm(const float* __restrict__ y, const float* __restrict__ wgt, int top, const float* __restrict__ ysh,
+// NT threads per row: 256, or 1024 when a step has so few rows that the latency of one row counts.
+template <int NT>
+__global__ void __launch_bounds__(NT) rms_add_norm(const float* __restrict__ y, const float* __restrict__ wgt, int top, const float* __restrict__ ysh,
                                                     const float* __restrict__ wsh, const float* __restrict__ wy, const float* x, float* xo, int ldxo,
                                                     const float* __restrict__ wh, float* __restrict__ h, int n,
                                                     float eps, float alpha) {
   __shared__ float red[33];
   const size_t t = blockIdx.x;
-  float v[kLnRegs], u[kLnRegs], ss = 0.f;
+  constexpr int KR = NT * kLnRegs / NT;
+  float v[KR], u[KR], ss = 0.f;
 #pragma unroll
-  for (int k = 0; k < kLnRegs; k++) {
-    const int i = threadIdx.x + 256 * k;
+  for (int k = 0; k < KR; k++) {
+    const int i = threadIdx.x + NT * k;
     v[k] = i < n && !wgt ? y[t * n + i] : 0.f;
     u[k] = i < n ? x[t * n + i] : 0.f;
   }
   if (wgt) {
-    for (int e = 0; e < top; e++) {
-      const float we = wgt[t * top + e];
-      const float* yr = y + (t * top + e) * n;
+    constexpr int EB = KR >= 16 ? 1 : 16 / KR;   // rows whose loads are in flight together
+    for (int e0 = 0; e0 < top; e0 += EB) {
+      float r[EB][KR];
 #pragma unroll
-      for (int k = 0; k < kLnRegs; k++) { const int i = threadIdx.x + 256 * k; if (i < n) v[k] = fmaf(we, yr[i], v[k]); }
+      for (int e = 0; e < EB; e++)
+#pragma unroll
+        for (int k = 0; k < KR; k++) { const int i = threadIdx.x + NT * k; r[e][k] = e0 + e < top && i < n ? y[(t * top + e0 + e) * n + i] : 0.f; }
+#pragma unroll
+      for (int e = 0; e < EB; e++) {
+        const float we = e0 + e < top ? wgt[t * top + e0 + e] : 0.f;
+#pragma unroll
+        for (int k = 0; k < KR; k++) v[k] = fmaf(we, r[e][k], v[k]);
+      }
     }
     if (ysh) {
       const float we = wsh[t];
 #pragma unroll
-      for (int k = 0; k < kLnRegs; k++) { const int i = threadIdx.x + 256 * k; if (i < n) v[k] = fmaf(we, ysh[t * n + i], v[k]); }
+      for (int k = 0; k < KR; k++) { const int i = threadIdx.x + NT * k; if (i < n) v[k] = fmaf(we, ysh[t * n + i], v[k]); }
     }
   }
 #pragma unroll
-  for (int k = 0; k < kLnRegs; k++) ss = fmaf(v[k], v[k], ss);
+  for (int k = 0; k < KR; k++) ss = fmaf(v[k], v[k], ss);
   float sc = alpha / sqrtf(block_sum(ss, red) / (float)n + eps);
   ss = 0.f;
 #pragma unroll
-  for (int k = 0; k < kLnRegs; k++) {
-    const int i = threadIdx.x + 256 * k;
+  for (int k = 0; k < KR; k++) {
+    const int i = threadIdx.x + NT * k;
     if (i < n) { u[k] = fmaf(v[k] * sc, wy[i], u[k]); xo[t * ldxo + i] = u[k]; ss = fmaf(u[k], u[k], ss); }
   }
   if (!wh) return;
   sc = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
 #pragma unroll
-  for (int k = 0; k < kLnRegs; k++) { const int i = threadIdx.x + 256 * k; if (i < n) h[t * n + i] = u[k] * sc * wh[i]; }
+  for (int k = 0; k < KR; k++) { const int i = threadIdx.x + NT * k; if (i < n) h[t * n + i] = u[k] * sc * wh[i]; }
 }
 
 // the T rows of a step (pitch ls) copied to rows of pitch ld
@@ -1539,24 +1648,43 @@ __device__ __forceinline__ float rot_entry(const float* __restrict__ src, int c,
   }
   return v;
 }
-// A causal convolution of the [q | k | v] channels: w [channels][taps], last tap on the current token; hist: ring over positions of `ring`
-// rows of inputs.  A step of at most ring - (taps - 1) tokens stores its inputs in rows that it does not read.
+// A causal convolution of the [q | k | v] channels, last tap on the current token: w holds three blocks [taps][channels of q, k, v];
+// hist: ring over positions of `ring` rows of inputs.  A step of at most ring - (taps - 1) tokens stores its inputs in rows that it does
+// not read.
 struct ConvP {
   const float* w;
   float* hist;
   int taps, ring, store;
 };
-__device__ __forceinline__ float conv_at(const ConvP& cv, const float* __restrict__ rows, int ld, int c, int ch, int pos0, int t) {
-  float acc = 0.f;
-  for (int j = 0; j < cv.taps; j++) {
-    const int tau = t - (cv.taps - 1) + j;
-    float v = 0.f;
-    if (tau >= 0) v = rows[(size_t)tau * ld + c];
-    else if (pos0 + tau >= 0) v = cv.hist[(size_t)((pos0 + tau) % cv.ring) * ch + c];
-    acc = fmaf(cv.w[(size_t)c * cv.taps + j], v, acc);
+// channels c0 + i, i = first, first + stride, .. < n (at most four of them go into acc) of token t; w: taps of channel c0, ldw apart
+__device__ __forceinline__ void conv4(const ConvP& cv, const float* __restrict__ w, int ldw, const float* __restrict__ rows, int ld, int c0, int first, int stride,
+                                      int n, int ch, int pos0, int t, float (&acc)[4]) {
+#pragma unroll
+  for (int e = 0; e < 4; e++) acc[e] = 0.f;
+  for (int j0 = 0; j0 < cv.taps; j0 += 4) {   // sixteen inputs and taps in flight
+    float x[4][4], wt[4][4];
+#pragma unroll
+    for (int jj = 0; jj < 4; jj++) {
+      const int j = j0 + jj, tau = t - (cv.taps - 1) + j;
+      const bool on = j < cv.taps && pos0 + tau >= 0;
+      const float* src = tau >= 0 ? rows + (size_t)tau * ld : on ? cv.hist + (size_t)((pos0 + tau) % cv.ring) * ch : rows;
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const int i = first + stride * e;
+        x[jj][e] = on && i < n ? src[c0 + i] : 0.f;
+        wt[jj][e] = on && i < n ? w[(size_t)j * ldw + i] : 0.f;
+      }
+    }
+#pragma unroll
+    for (int jj = 0; jj < 4; jj++)
+#pragma unroll
+      for (int e = 0; e < 4; e++) acc[e] = fmaf(wt[jj][e], x[jj][e], acc[e]);
   }
-  if (cv.store) cv.hist[(size_t)((pos0 + t) % cv.ring) * ch + c] = rows[(size_t)t * ld + c];
-  return acc;
+  if (cv.store) {
+    float* dst = cv.hist + (size_t)((pos0 + t) % cv.ring) * ch + c0;
+#pragma unroll
+    for (int e = 0; e < 4; e++) { const int i = first + stride * e; if (i < n) dst[i] = rows[(size_t)t * ld + c0 + i]; }
+  }
 }
 __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q, float* __restrict__ q_out, int HD,
                                                     const float* __restrict__ k, const float* __restrict__ v_src, int GD, int GV, int ld_q, int ld_k, int ld_v,
@@ -1581,7 +1709,13 @@ __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q,
       const float* src = isq ? qr : kr;
       if (cv.w) {
         float* row_s = cs + w * D;
-        for (int d = lane; d < D; d += 32) row_s[d] = conv_at(cv, q, ld_q, hh * D + d, HD + GD + GV, ctl[0], t);
+        const float* wt = isq ? cv.w + c0 : cv.w + (size_t)HD * cv.taps + c0;
+        for (int d0 = lane; d0 < D; d0 += 128) {
+          float acc[4];
+          conv4(cv, wt, isq ? HD : GD, q, ld_q, hh * D, d0, 32, D, HD + GD + GV, pos - t, t, acc);
+#pragma unroll
+          for (int e = 0; e < 4; e++) if (d0 + 32 * e < D) row_s[d0 + 32 * e] = acc[e];
+        }
         __syncwarp();
         src = row_s - c0;
       }
@@ -1618,7 +1752,13 @@ __global__ void __launch_bounds__(256) qk_norm_rope(const float* __restrict__ q,
   }
   if (!k) return;
   if (cv.w) {   // the value channels are dealt over the CTAs of the token too
-    for (int e = threadIdx.x + 256 * (int)blockIdx.y; e < GV; e += 256 * (int)gridDim.y) vcache[row * GV + e] = conv_at(cv, q, ld_q, HD + GD + e, HD + GD + GV, ctl[0], t);
+    const int step = 256 * (int)gridDim.y;
+    for (int e0 = threadIdx.x + 256 * (int)blockIdx.y; e0 < GV; e0 += 4 * step) {
+      float acc[4];
+      conv4(cv, cv.w + (size_t)(HD + GD) * cv.taps, GV, q, ld_q, HD + GD, e0, step, GV, HD + GD + GV, pos - t, t, acc);
+#pragma unroll
+      for (int e = 0; e < 4; e++) if (e0 + step * e < GV) vcache[row * GV + e0 + step * e] = acc[e];
+    }
     return;
   }
   if (blockIdx.y > 0) return;

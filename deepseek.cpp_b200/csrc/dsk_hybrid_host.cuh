@@ -96,7 +96,7 @@ struct HLayer {
   // gated delta rule: its projections ride in qkv (att_layout), convolution taps of the [q | k | v] channels in one array; A_log, dt_bias
   // and lin_norm as above.  Side by side with attention, o holds both output matrices column by column: [left | right]
   float* gdn_conv_w = nullptr;
-  // attention behind short convolutions: taps of the [q | k | v] channels in conv_w, have_conv as below.  mLSTM: lin_in [q | k | v | g | i | f],
+  // attention behind short convolutions: taps of the q, k and v channels in conv_w, three blocks [taps][channels], have_conv as below.  mLSTM: lin_in [q | k | v | g | i | f],
   // padded to a multiple of 8 rows, lin_bias with the gates' biases, mnorm
   char have_gate[2] = {0, 0}, have_gateb[2] = {0, 0};
   char have_gdn[6] = {0, 0, 0, 0, 0, 0}, have_conv[3] = {0, 0, 0}, have_o[2] = {0, 0};
@@ -770,11 +770,11 @@ static int upload(dsk_model* m, const char* name, int dtype, const int64_t shape
       }
       if (s.att_conv > 0)
         for (int n = 0; n < 3; n++)
-          if (k == std::string(1, "qkv"[n]) + ".conv") {   // taps of the stacked [q | k | v] channels
+          if (k == std::string(1, "qkv"[n]) + ".conv") {
             if (L.have_conv[n]) return fail(-4, "tensor %s uploaded twice", name);
             if (!L.conv_w && dmalloc(m, (void**)&L.conv_w, (size_t)(HD + GD + GV) * s.att_conv * 4)) return -2;
             L.have_conv[n] = 1;
-            return put(name, dtype, shape, data, nbytes, on_dev, n == 0 ? HD : n == 1 ? GD : GV, s.att_conv, L.conv_w + (size_t)(n == 0 ? 0 : n == 1 ? HD : HD + GD) * s.att_conv, false, 0);
+            return put(name, dtype, shape, data, nbytes, on_dev, n == 0 ? HD : n == 1 ? GD : GV, s.att_conv, L.conv_w + (size_t)(n == 0 ? 0 : n == 1 ? HD : HD + GD) * s.att_conv, false, (int)(n == 0 ? HD : n == 1 ? GD : GV));   // stored [taps][channels]
           }
       if (k == "rel" && s.att_rel_max > 0) {   // the number of distance buckets is the tensor's first size
         if (shape[0] < 2 || shape[0] > (1 << 20)) return fail(-4, "tensor %s: %lld distance buckets", name, (long long)shape[0]);
@@ -1081,7 +1081,7 @@ static int launches_per_token(const dsk_model* m) {
     else if (s.mixer == DSK_MIX_LIGHTNING) n += lin_decode_fits(s.lin_dim, s.lin_vdim) ? 4 : 5;   // stacked projection, (records,) recurrence, norm, o
     else if (s.mixer == DSK_MIX_HGRN2) n += 4;   // stacked projection, recurrence, head norm, o
     else if (s.mixer == DSK_MIX_GQA) n += s.att_value_proj ? 5 : 6;   // q, k (or one stacked q / k / v (/ gate) product), norm + rotation, attention, merge, o
-    else if (s.mixer == DSK_MIX_MLA) n += 10 + (s.att_out_gate ? 1 : 0);   // down-projections, query norm, query up, latent preparation, absorbed query, attention, merge, value up, (gate,) o
+    else if (s.mixer == DSK_MIX_MLA) n += 9 + (s.att_out_gate ? 1 : 0);   // down-projections, query norm, query up, latent preparation, absorbed query, attention, merge, value up, (gate,) o
     else n += is_ssd(s) ? 5 + (s.ssm_conv > 1 ? 1 : 0) : 5 + (s.att_kv_from < 0 ? 2 : 0);
     if (s.ff_kind == DSK_FF_MOE) n += (post && M->c.norm_kind == DSK_NORM_LAYER && !M->c.res_gate && M->c.dim <= 256 * kLnRegs && s.ff_shared == 0) || rms_fused(M->c) ? 4 : 5;
     if (R.pass >= 0 && M->c.loop_in) n += 1 + (&R != &M->runs[0] && fused_norms(M->c) ? 1 : 0);   // product, its norm
@@ -1361,7 +1361,27 @@ static void launch_gemm_mma(int epi, const GemmP& P, int Z, int tile_cap, cudaSt
 
 template <typename WT>
 static void launch_gemm_t(int epi, const GemmP& P, int Z, bool small, int tile_cap, cudaStream_t st) {
-  if (small) {
+  if (small && gemv_one_ok<WT>(P)) {
+    const int n = std::max(P.N, P.n_shared > 0 ? P.sN : 0);
+    const int R = (long long)n * Z >= 16384 && Z == 1 ? 2 : 1;   // rows per warp
+    const dim3 grid((unsigned)std::max(1, std::min((n + 8 * R - 1) / (8 * R), 148 * 8)), (unsigned)Z);
+#define DSK_GEMV1(E) do { if (R == 2) gemv_one<WT, E, 2><<<grid, 256, 0, st>>>(P); else gemv_one<WT, E, 1><<<grid, 256, 0, st>>>(P); } while (0)
+    switch (epi) {
+      case HEPI_STORE: DSK_GEMV1(HEPI_STORE); break;
+      case HEPI_ADD: DSK_GEMV1(HEPI_ADD); break;
+      case HEPI_GLU: DSK_GEMV1(HEPI_GLU); break;
+      case HEPI_XIELU: DSK_GEMV1(HEPI_XIELU); break;
+      case HEPI_GEGLU: DSK_GEMV1(HEPI_GEGLU); break;
+      case HEPI_SIGMUL: DSK_GEMV1(HEPI_SIGMUL); break;
+      case HEPI_RELU2: DSK_GEMV1(HEPI_RELU2); break;
+      case HEPI_LINGATE: DSK_GEMV1(HEPI_LINGATE); break;
+      case HEPI_SILU_SIG: DSK_GEMV1(HEPI_SILU_SIG); break;
+      case HEPI_SOFTCAP: DSK_GEMV1(HEPI_SOFTCAP); break;
+      case HEPI_SWIGLU: DSK_GEMV1(HEPI_SWIGLU); break;
+      default: DSK_GEMV1(HEPI_GELU_MUL); break;
+    }
+#undef DSK_GEMV1
+  } else if (small) {
     const dim3 grid((unsigned)std::max(1, std::min((std::max(P.N, P.n_shared > 0 ? P.sN : 0) + 7) / 8, 148 * 8)), (unsigned)Z);
     switch (epi) {
       case HEPI_STORE: gemv_rows<WT, HEPI_STORE><<<grid, 256, 0, st>>>(P); break;
@@ -1398,7 +1418,7 @@ static void launch_gemm_t(int epi, const GemmP& P, int Z, bool small, int tile_c
 // C = A W^T (+ epilogue).  Z > 1: per-head batches or (gemv) one batch per routed (token, slot) pair.
 static void linear(State* S, bool bf16, int epi, const GemmP& P, int Z, cudaStream_t st, int tile_cap = 0) {
   const bool small = P.z_expert != nullptr || (!P.tiles && P.M <= 4);
-  if (!small && !P.tiles && Z == 1 && P.N <= 64) {   // narrow output (router, token-input gate): warp-per-row products over batches of 4 rows
+  if (!small && !P.tiles && Z == 1 && P.N <= 96) {   // narrow output (router, token-input gate): warp-per-row products over batches of 4 rows
     GemmP Q = P;
     Q.z_rows = P.M;
     const int zb = (P.M + 3) / 4;
@@ -1575,8 +1595,15 @@ static void enqueue_head(dsk_model* m, dsk_state* s, int first, int count, cudaS
 // the model's norm over the T rows of `in` (width values each): stored into `out`, or added into it times alpha (mode 1)
 static void norm_rows(const dsk_hybrid_config& c, State* S, const float* in, const float* w, const float* b, float* out, int T, int mode, float alpha, cudaStream_t st) {
   if (c.norm_kind == DSK_NORM_LAYER) layer_norm<<<T, 256, 0, st>>>(in, c.dim, w, b, out, c.dim, c.dim, c.norm_eps, mode, alpha, nullptr, 0);
+  else if (mode == 0 && c.norm_groups == 1) rms_open<<<T, 256, 0, st>>>(const_cast<float*>(in), nullptr, nullptr, w, out, c.dim, c.norm_eps);   // (adds nothing: the row is only read)
   else group_rmsnorm<float><<<T, 256, 0, st>>>(in, c.dim, w, out, c.dim, c.dim, c.norm_groups, c.norm_eps, mode, alpha, nullptr, 0);
   S->launches++;
+}
+
+template <typename... A>
+static void launch_rms_add_norm(int T, cudaStream_t st, A... a) {
+  if (T <= kAttnSplitTokens) rms_add_norm<1024><<<T, 1024, 0, st>>>(a...);
+  else rms_add_norm<256><<<T, 256, 0, st>>>(a...);
 }
 
 static bool fused_norms(const dsk_hybrid_config& c) {
@@ -1697,7 +1724,7 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
         const bool to_xin = next && next->pass >= 0;   // the pass opens with a product: its norm follows that
         const bool product = to_xin && c.loop_in;
         const bool shared = routed && sp.ff_shared > 0;
-        rms_add_norm<<<T, 256, 0, st>>>(routed ? S->b3 : S->y, routed ? S->wgt : nullptr, routed, shared ? S->b3 + (size_t)T * routed * W : nullptr, S->wsh, wb, S->x,
+        launch_rms_add_norm(T, st, routed ? S->b3 : S->y, routed ? S->wgt : nullptr, routed, shared ? S->b3 + (size_t)T * routed * W : nullptr, S->wsh, wb, S->x,
                                         product ? S->xin : S->x, product ? 2 * W : W, to_xin ? nullptr : next ? M->L[next->layer].norm1 : M->final_norm, S->h, W, c.norm_eps, mult);
         S->launches++;
         xin_ready = product;
@@ -2029,7 +2056,7 @@ static int enqueue_chunk(dsk_model* m, dsk_state* s, int T, int n_want, float* t
     if (sandwich) {   // x += norm1b(mixer output); the feed-forward then reads norm2 of the new x
       if (sp.ff_kind == DSK_FF_NONE) close_run(L.close1);
       else if (frms) {
-        rms_add_norm<<<T, 256, 0, st>>>(S->y, nullptr, 0, nullptr, nullptr, L.close1, S->x, S->x, W, L.norm2, S->h, W, c.norm_eps, mult);
+        launch_rms_add_norm(T, st, S->y, nullptr, 0, nullptr, nullptr, L.close1, S->x, S->x, W, L.norm2, S->h, W, c.norm_eps, mult);
         S->launches++;
       } else if (fuse) {
         layer_norm_add_norm<<<T, 256, 0, st>>>(S->y, L.close1, S->x, nullptr, L.norm2, S->h, W, c.norm_eps, mult);

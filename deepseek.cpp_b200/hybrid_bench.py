@@ -6,7 +6,9 @@ attention-only design with dense feed-forwards) at equal width, depth, heads, wi
 Nalizen sizes run beside a Desarax model (the framework's other design with a recurrence, shared attention caches, routed
 feed-forwards and the per-layer token input) at equal width, depth, layer pattern, heads, window and active matrix elements; the
 Zetivik sizes run beside a Nalizen model (the framework's other design of attention with an output gate, a gated linear recurrence
-and gated dense feed-forwards), one Nalizen layer per mixer of every layer run, at equal width, heads, sizes and feed-forwards.
+and gated dense feed-forwards), one Nalizen layer per mixer of every layer run, at equal width, heads, sizes and feed-forwards; the
+Netusun sizes run beside a Nalizen model (the framework's other design of windowed attention, a gated recurrence and routed
+feed-forwards), one Nalizen layer per layer run, at equal width, heads, windows and active feed-forward elements.
 
 Used by `bench.py --hybrid`.  Random weights generated on the GPU (bf16), uploaded through dsk_upload_tensor(src_on_device).
 Decode is the device-side greedy loop (CUDA events around the captured step graph); prefill is dsk_forward_chunk over a prompt
@@ -47,7 +49,155 @@ SIZES = {
                           lin_heads=16, lin_kv_heads=8, lin_dim=64, lin_vdim=64, conv=4, ff=2816),
     "zetivik_large": dict(design="Zetivik", width=2048, vocab=102400, pattern="plpplppl", loop=(3, 5, 2), att_heads=16, kv_heads=4, att_dim=128, window=1024,
                           lin_heads=16, lin_kv_heads=8, lin_dim=128, lin_vdim=128, conv=4, ff=5632),
+    # Netusun: layers of windowed attention (a), latent attention over everything (l) and the matrix memory (m); the first layer's feed-forward
+    # is dense, the others are routed with a shared expert; layers loop[0] .. loop[1]-1 run loop[2] times
+    "netusun_small": dict(design="Netusun", width=1024, vocab=32000, pattern="amalma", loop=(1, 4, 2), att_heads=16, kv_heads=4, att_dim=64, window=512, conv=4,
+                          lin_heads=16, lin_dim=64, lin_vdim=64, lat_dim=64, rot=32, kv_rank=256, q_rank=384, ff=1536, experts=16, groups=4, keep=2, top=2,
+                          eff=512, shared=512),
+    "netusun_large": dict(design="Netusun", width=2048, vocab=102400, pattern="amalmaml", loop=(2, 5, 2), att_heads=16, kv_heads=4, att_dim=128, window=1024,
+                          conv=4, lin_heads=16, lin_dim=128, lin_vdim=128, lat_dim=128, rot=64, kv_rank=512, q_rank=768, ff=10944, experts=64, groups=8, keep=4,
+                          top=6, eff=1408, shared=2816),
 }
+
+
+def netusun_config(z):
+    layers = []
+    for i, ch in enumerate(z["pattern"]):
+        if ch == "a":
+            mx = {"heads": z["att_heads"], "kv_heads": z["kv_heads"], "dim": z["att_dim"], "vdim": z["att_dim"], "scale": z["att_dim"] ** -0.5, "softcap": 50.0,
+                  "mask": {"size": z["window"]}, "conv": z["conv"]}
+        elif ch == "l":
+            mx = {"heads": z["att_heads"], "dim": z["lat_dim"], "rot_dim": z["rot"], "vdim": z["lat_dim"], "kv_rank": z["kv_rank"], "q_rank": z["q_rank"],
+                  "scale": (z["lat_dim"] + z["rot"]) ** -0.5,
+                  "rot": {"dims": z["rot"], "base": 500000.0, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        else:
+            mx = {"heads": z["lin_heads"], "dim": z["lin_dim"], "vdim": z["lin_vdim"], "gate_cap": 15.0}
+        ff = {"kind": "dense", "ff": z["ff"]} if i == 0 else \
+             {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"], "scale": 2.5, "groups": {"count": z["groups"], "keep": z["keep"]}},
+              "expert": {"ff": z["eff"]}, "shared": {"ff": z["shared"]}}
+        layers.append({"type": {"a": "attention", "l": "latent_attention", "m": "mlstm"}[ch], "mixer": mx, "mlp": ff})
+    a, b, t = z["loop"]
+    return {"architecture": "Netusun", "vocab": z["vocab"], "width": z["width"], "layers": layers, "norm": {"eps": 1e-5}, "loop": {"start": a, "stop": b, "times": t}}
+
+
+def closest_nalizen_of_netusun(z):
+    """Nalizen layers at a Netusun size, one per layer run: attention for both kinds of attention (the latent one without a window),
+    the recurrence for the matrix memory; routed feed-forwards of two-matrix experts with as many active matrix elements."""
+    layers = []
+    moe = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": 3 * (z["top"] * z["eff"] + z["shared"]) // (2 * z["top"])}}
+    for i, ch in enumerate(zetivik_runs(z)):
+        mlp = {"kind": "dense", "ff": z["ff"]} if i == 0 else moe
+        if ch == "m":
+            layers.append({"type": "hgrn2", "mixer": {"heads": z["lin_heads"], "dim": z["lin_dim"], "vdim": z["lin_vdim"]}, "mlp": mlp})
+            continue
+        mx = {"heads": z["att_heads"], "kv_heads": z["kv_heads"], "dim": z["att_dim"], "vdim": z["att_dim"], "scale": z["att_dim"] ** -0.5,
+              "rot": {"dims": z["att_dim"], "base": 500000.0}}
+        if ch == "a":
+            mx["mask"] = {"size": z["window"]}
+        layers.append({"type": "attention", "mixer": mx, "mlp": mlp})
+    return {"architecture": "Nalizen", "vocab": z["vocab"], "width": z["width"], "layers": layers, "norm": {"eps": 1e-5}}
+
+
+def mint_netusun(dsk, torch, cfg, quant, chunk, context, device=0):
+    import hashlib
+    hc, specs = dsk.netusun_from_config(cfg, quant=quant, max_seq_len=context, chunk=chunk)
+    m = dsk.Model(hc, 0, 1, device, layers=specs)
+    dev = torch.device("cuda", device)
+    W, V = cfg["width"], cfg["vocab"]
+
+    def up(name, shape, kind="mat"):
+        torch.manual_seed(int(hashlib.md5(name.encode()).hexdigest()[:8], 16))
+        if kind == "mat":
+            t = torch.randn(*shape, device=dev) * (shape[-1] ** -0.5)
+        elif kind == "embed":
+            t = torch.randn(*shape, device=dev)
+        elif kind == "norm":
+            t = 1.0 + 0.1 * torch.randn(*shape, device=dev)
+        elif kind == "gate":
+            t = torch.empty(*shape, device=dev).uniform_(1.0, 6.0)
+        else:
+            t = 0.1 * torch.randn(*shape, device=dev)
+        t = t.to(torch.bfloat16).contiguous()
+        m.upload_device(name, "BF16", shape, t.data_ptr(), t.numel() * 2)
+        torch.cuda.synchronize()
+
+    def glu(q, f):
+        up(q + "gate", (f, W)); up(q + "up", (f, W)); up(q + "down", (W, f))
+
+    up("embed", (V, W), "embed"); up("final.norm", (W,), "norm"); up("loop.in", (W, 2 * W)); up("loop.step", (cfg["loop"]["times"], W), "small")
+    for i, lc in enumerate(cfg["layers"]):
+        p, mx, ff = f"l{i}.", lc["mixer"], lc["mlp"]
+        q = p + "mix."
+        for n in ("norm1", "norm1b", "norm2", "norm2b", "ls1", "ls2"):
+            up(p + n, (W,), "norm")
+        H, D, P = mx["heads"], mx["dim"], mx["vdim"]
+        if lc["type"] == "attention":
+            G = mx["kv_heads"]
+            for t, n in (("q", H * D), ("k", G * D), ("v", G * P)):
+                up(q + t, (n, W)); up(q + t + ".conv", (n, mx["conv"]))
+            up(q + "q.norm", (D,), "norm"); up(q + "k.norm", (D,), "norm")
+        elif lc["type"] == "latent_attention":
+            R, Q, Rd = mx["kv_rank"], mx["q_rank"], mx["rot_dim"]
+            up(q + "dq", (Q, W)); up(q + "dq.norm", (Q,), "norm"); up(q + "uq", (H * (D + Rd), Q)); up(q + "dkv", (R + Rd, W)); up(q + "dkv.norm", (R,), "norm")
+            up(q + "uk", (H * D, R)); up(q + "uv", (H * P, R)); up(q + "sink", (H,), "small"); up(q + "g", (H * P, W))
+        else:
+            for t, n in (("q", H * D), ("k", H * D), ("v", H * P), ("g", H * P), ("i", H), ("f", H)):
+                up(q + t, (n, W))
+            up(q + "i.b", (H,), "small"); up(q + "f.b", (H,), "gate"); up(q + "norm", (H * P,), "norm")
+        up(q + "o", (W, H * P))
+        if ff["kind"] == "dense":
+            glu(p + "mlp.", ff["ff"])
+        else:
+            up(p + "mlp.router", (ff["router"]["experts"], W)); up(p + "mlp.shared.sg", (1, W)); glu(p + "mlp.shared.", ff["shared"]["ff"])
+            for e in range(ff["router"]["experts"]):
+                glu(f"{p}mlp.e{e}.", ff["expert"]["ff"])
+    m.finalize()
+    return m
+
+
+def netusun_matrix_elements(cfg, z, prompt_len):
+    """Matrix elements one token multiplies with over all layer runs (projections, gates, feed-forward, loop products, head), and the
+    attention's own multiply-adds per token at the mean number of visible keys (half the window, half the prompt)."""
+    W, att = cfg["width"], 0.0
+    n = W * cfg["vocab"] + 2 * W * W * z["loop"][2]
+    a, b, t = z["loop"]
+    order = list(range(a)) + list(range(a, b)) * t + list(range(b, len(z["pattern"])))
+    for i in order:
+        mx, ff = cfg["layers"][i]["mixer"], cfg["layers"][i]["mlp"]
+        H, D, P = mx["heads"], mx["dim"], mx["vdim"]
+        if z["pattern"][i] == "a":
+            n += H * (D + P) * W + mx["kv_heads"] * (D + P) * W
+            att += H * (D + P) * (z["window"] / 2.0)
+        elif z["pattern"][i] == "l":
+            R, Q, Rd = mx["kv_rank"], mx["q_rank"], mx["rot_dim"]
+            n += (Q + R + Rd) * W + H * (D + Rd) * Q + H * (D + P) * R + 2 * H * P * W
+            att += H * (D + Rd + P) * (prompt_len / 2.0)
+        else:
+            n += (2 * H * D + 3 * H * P + 2 * H) * W
+        n += 3 * ff["ff"] * W if ff["kind"] == "dense" else 3 * (ff["router"]["top"] * ff["expert"]["ff"] + ff["shared"]["ff"]) * W + (ff["router"]["experts"] + 1) * W
+    return n, att
+
+
+def run_netusun(dsk, torch, name, hbm, tfl, prompt_len, gen, chunk, log):
+    """A Netusun size and the closest layer-list model (Nalizen) at equal size."""
+    z = SIZES[name]
+    cfg = netusun_config(z)
+    t0 = time.time()
+    m = mint_netusun(dsk, torch, cfg, "bf16", chunk, prompt_len + gen + 8)
+    log(f"hybrid/{name}/bf16: minted {m.resident_bytes() / 1e9:.2f} GB in {time.time() - t0:.1f} s")
+    mat, att = netusun_matrix_elements(cfg, z, prompt_len)
+    res = [measure_layer_list(m, f"Netusun {name}", z["vocab"], 2.0 * mat, hbm, tfl, prompt_len, gen, chunk, log,
+                              {"layer_runs": len(zetivik_runs(z)), "width": z["width"], "attention_flops_per_token_fp32": 2.0 * att})]
+    m.close()
+    cfgn = closest_nalizen_of_netusun(z)
+    t0 = time.time()
+    m = mint_nalizen(dsk, torch, cfgn, "bf16", chunk, prompt_len + gen + 8)
+    log(f"hybrid/{name}/closest Nalizen/bf16: minted {m.resident_bytes() / 1e9:.2f} GB in {time.time() - t0:.1f} s")
+    matn, attn = nalizen_matrix_elements(cfgn, z)
+    res.append(measure_layer_list(m, f"Nalizen layers at {name}", z["vocab"], 2.0 * matn, hbm, tfl, prompt_len, gen, chunk, log,
+                                  {"layers": len(cfgn["layers"]), "width": z["width"]}))
+    m.close()
+    return res
 
 
 def zetivik_config(z):
@@ -639,6 +789,9 @@ def run(dsk, torch, repo, bench_module, sizes=("small", "v2lite_like"), prompt_l
             continue
         if z.get("design") == "Zetivik":
             out["results"] += run_zetivik(dsk, torch, name, hbm, tfl, prompt_len, gen, chunk, log)
+            continue
+        if z.get("design") == "Netusun":
+            out["results"] += run_netusun(dsk, torch, name, hbm, tfl, prompt_len, gen, chunk, log)
             continue
         cfg = desarax_config(z)
         for quant in ("bf16",):

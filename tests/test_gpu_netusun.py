@@ -630,7 +630,7 @@ def test_launch_count_of_a_decoded_token(full):
     cfg, m, W, toks, exp, _ = full
     import dsk
     n = dsk.lib().dsk_launches_per_forward(m.h, dsk.OUTPUT_LOGITS)
-    att, mem, lat, moe, dense = 5, 3, 11, 4, 2            # launches of a mixer / feed-forward without the norms around it
+    att, mem, lat, moe, dense = 5, 3, 10, 4, 2            # launches of a mixer / feed-forward without the norms around it
     runs = [(att, moe)] + [(mem, dense), (lat, moe), (att, moe)] * 3 + [(mem, moe), (lat, None)]
     want = 3 + 1 + sum(a + 1 + ((f + 1) if f else 0) for a, f in runs) + 3 * 2     # embed, head, arg-max; first norm; passes: product and norm
     assert n == want

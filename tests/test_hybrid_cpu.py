@@ -331,3 +331,90 @@ def test_zetivik_oracle_invariants(zo):
     y = zo.clamped_glu({"f." + k: v for k, v in Wf.items()}, "f.", np.array([1.0]), 2.0)[0]
     assert abs(y - 2.0 / (1.0 + np.exp(-3.404)) * (-1.0)) < 1e-12
     assert abs(zo.soft_cap(np.array([1e9]), 4.0)[0] - 4.0) < 1e-9 and zo.soft_cap(np.array([3.0]), 0)[0] == 3.0
+
+
+# ---- the Netusun design ----------------------------------------------------------------------------------------------------------
+@pytest.fixture(scope="module")
+def nu():
+    import netusun_oracle
+    return netusun_oracle
+
+
+def test_netusun_config_to_layer_specs(nu):
+    import dsk
+    cfg = nu.small_config()
+    hc, specs = dsk.ARCHITECTURES[cfg["architecture"]](cfg, quant="fp32", max_seq_len=77, chunk=16)
+    assert (hc.dim, hc.vocab_size, hc.n_layers, hc.max_seq_len, hc.chunk, hc.quant) == (44, 61, 6, 77, 16, dsk.QUANT_IDS["fp32"])
+    assert (hc.block, hc.norm_kind, hc.layer_scale, hc.tie_head, hc.loop_start, hc.loop_stop, hc.loop_times, hc.loop_in, hc.loop_embed) == \
+        (dsk.BLOCK_SANDWICH, dsk.NORM_RMS, 1, 1, 1, 4, 3, 1, 0)
+    assert abs(hc.norm_eps - 1e-5) < 1e-12 and (hc.norm_bias, hc.token_shift, hc.norm_scalar, hc.side_dim, hc.norm_one_plus) == (0, 0, 0, 0, 0)
+    a, m, l, b = specs[0], specs[1], specs[2], specs[3]
+    assert (a.mixer, a.att_heads, a.att_kv_heads, a.att_dim, a.att_vdim, a.att_mask, a.att_window, a.att_kv_from) == (dsk.MIX_GQA, 6, 2, 10, 6, dsk.MASK_WINDOW, 7, -1)
+    assert (a.att_value_proj, a.att_bias, a.att_out_gate, a.att_qk_norm, a.att_talk, a.att_sink, a.rot_dims, a.att_conv) == \
+        (1, 0, 0, dsk.QKNORM_HEAD_WEIGHT, 0, dsk.SINK_ONE, 0, 3) and abs(a.att_softcap - 4.0) < 1e-7 and abs(a.att_scale - 0.6) < 1e-7
+    assert (a.ff_kind, a.ff_experts, a.ff_top, a.ff_hidden, a.ff_groups, a.ff_groups_keep, a.ff_shared, a.ff_router, a.ff_expert) == \
+        (dsk.FF_MOE, 9, 3, 14, 3, 2, 11, dsk.ROUTER_SOFTMAX_GROUPS, dsk.EXPERT_SWIGLU) and abs(a.ff_router_scale - 1.7) < 1e-7
+    assert (m.mixer, m.lin_heads, m.lin_dim, m.lin_vdim, m.ff_kind, m.ff_act, m.ff_hidden) == (dsk.MIX_MLSTM, 3, 5, 9, dsk.FF_DENSE, dsk.ACT_SWIGLU, 28)
+    assert m.lin_gate_cap == 4.0
+    assert (l.mixer, l.att_heads, l.att_dim, l.att_rot_dim, l.att_vdim, l.att_kv_rank, l.att_q_rank, l.att_sink, l.att_out_gate, l.att_window) == \
+        (dsk.MIX_MLA, 4, 9, 6, 7, 13, 18, dsk.SINK_HEAD, dsk.GATE_ENTRY, 1 << 30)
+    assert (l.rot_dims, l.rot_layout, l.rot_scale, l.rot_original, l.rot_factor, l.rot_fast, l.rot_slow) == (6, dsk.ROT_HALF, dsk.ROTSCALE_YARN, 40, 3.0, 6.0, 0.5)
+    assert (l.ff_groups, l.ff_shared) == (0, 0) and (b.att_conv, b.ff_groups, b.ff_groups_keep) == (5, 4, 1) and specs[5].ff_kind == dsk.FF_NONE
+    mx = cfg["layers"][0]["mixer"]
+    del mx["mask"], mx["softcap"], mx["kv_heads"], cfg["layers"][2]["mixer"]["rot"]["scaling"], cfg["loop"]
+    hc, specs = dsk.netusun_from_config(cfg)
+    assert (specs[0].att_window, specs[0].att_softcap, specs[0].att_kv_heads, specs[2].rot_factor, hc.loop_times, hc.loop_in) == (1 << 30, 0.0, 6, 0.0, 0, 0)
+    for where, key, value in (("layers", "type", "hgrn2"), ("mlp", "kind", "sparse")):
+        bad = nu.small_config()
+        (bad["layers"][1] if where == "layers" else bad["layers"][1]["mlp"])[key] = value
+        with pytest.raises(dsk.DskError):
+            dsk.netusun_from_config(bad)
+
+
+def test_netusun_oracle_invariants(nu):
+    """(1) a sequence fed token by token equals the whole; (2) the order of layer runs; (3) window starts; (4) the softmax with an
+    extra term; (5) the convolution pairs its last tap with the current input; (6) the memory: two writes under one key, weighted by
+    their gates, and the floor of the normaliser; (7) a memory shifted by a constant input gate and its own maximum reads the same;
+    (8) groups; (9) the YaRN table's two ends and its magnitude; (10) the cap."""
+    cfg = nu.small_config()
+    W = nu.random_weights(cfg, 5)
+    toks = np.arange(20) % 61
+    whole = nu.run(cfg, W, toks)[0]
+    seq = nu.Sequence(cfg, W)
+    assert np.allclose(np.array([seq.feed(int(t)) for t in toks]), whole, rtol=0, atol=1e-12)
+    assert nu.layer_runs(cfg) == [(0, None), (1, 0), (2, None), (3, None), (1, 1), (2, None), (3, None), (1, 2), (2, None), (3, None), (4, None), (5, None)]
+    assert [nu.window_first(4, p) for p in (0, 3, 4, 9)] == [0, 0, 1, 6] and nu.window_first(None, 9) == 0
+    assert np.allclose(nu.softmax_with(np.array([0.0, 0.0]), 0.0), 1.0 / 3.0) and np.allclose(nu.softmax_with(np.array([900.0]), 0.0), 1.0)
+    w = np.array([[1.0, 10.0, 100.0]])
+    assert nu.short_conv(w, [np.array([2.0]), np.array([3.0])], np.array([4.0]))[0] == 432.0 and nu.short_conv(w, [], np.array([4.0]))[0] == 400.0
+    mx = {"heads": 1, "dim": 1, "vdim": 2, "gate_cap": 1e6}
+
+    def weights(i_bias, f_bias):
+        Wm = {"q": np.array([[1.0, 0.0, 0.0]]), "k": np.array([[1.0, 0.0, 0.0]]), "v": np.eye(3)[1:], "g": np.full((2, 3), 0.0), "i": np.zeros((1, 3)),
+              "f": np.zeros((1, 3)), "i.b": np.array([i_bias]), "f.b": np.array([f_bias]), "norm": np.array([2.0, 2.0]), "o": np.eye(2)}
+        return {"m." + k: v for k, v in Wm.items()}
+
+    def fresh():
+        return {"S": np.zeros((1, 1, 2)), "n": np.zeros((1, 1)), "m": np.zeros(1)}
+    st = fresh()
+    nu.mlstm_step(weights(0.0, 40.0), "m.", mx, np.array([1.0, 2.0, 0.0]), st, 1e-12)
+    nu.mlstm_step(weights(np.log(3.0), 40.0), "m.", mx, np.array([1.0, 0.0, 4.0]), st, 1e-12)
+    assert np.allclose(st["S"][0, 0] / st["n"][0, 0], [0.5, 3.0]) and np.allclose(st["m"], np.log(3.0))
+    a, b = fresh(), fresh()
+    for h in ([1.0, 2.0, 0.5], [0.3, 1.0, 4.0], [2.0, -1.0, 1.0]):
+        ya = nu.mlstm_step(weights(9.0, 1.0), "m.", mx, np.array(h), a, 1e-12)
+        yb = nu.mlstm_step(weights(5.0, 1.0), "m.", mx, np.array(h), b, 1e-12)
+        assert np.allclose(ya, yb, rtol=1e-6)                            # gates far above the start: only their differences matter
+    st = fresh()
+    nu.mlstm_step(weights(-50.0, 0.0), "m.", mx, np.array([1.0, 2.0, 0.0]), st, 1e-12)
+    assert np.allclose(st["m"], np.log(0.5)) and float(st["n"][0, 0]) < 1e-21      # the floor e^-m, not n . q, divides
+    z = np.array([1.0, 5.0, 2.0, 4.0, 4.5, 0.0])
+    r = {"top": 2, "scale": 2.0, "groups": {"count": 3, "keep": 1}}
+    p = np.exp(z) / np.exp(z).sum()
+    chosen, wt = nu.route(z, r)
+    assert chosen == [1, 0] and np.allclose(wt, 2.0 * p[[1, 0]])
+    assert nu.route(z, dict(r, groups={"count": 3, "keep": 2}))[0] == [1, 4] and nu.route(z, {"top": 3, "scale": 1.0})[0] == [1, 4, 3]
+    f, mag = nu.rotation_table({"dims": 16, "base": 10000.0, "scaling": {"factor": 4.0, "original": 64, "fast": 8.0, "slow": 0.25}})
+    f0 = 10000.0 ** (-np.arange(8) / 8.0)
+    assert f[0] == f0[0] and np.isclose(f[-1], f0[-1] / 4.0) and np.isclose(mag, 0.1 * np.log(4.0) + 1.0)
+    assert abs(nu.soft_cap(np.array([1e9]), 4.0)[0] - 4.0) < 1e-9 and nu.soft_cap(np.array([3.0]), None)[0] == 3.0
